@@ -5,6 +5,7 @@ from .qwen3 import Qwen3Config
 from .registry import architectures, config_class, read_config, register_architecture
 from .fusasun import FusasunConfig
 from .ninenex import NinenexConfig
+from .soputar import SoputarConfig
 from .tifapel import TifapelConfig
 from .voserax import VoseraxConfig
 from .spec import BlockSpec, LayerCall, ModelSpec, PartSpec, TensorSpec, default_schedule
@@ -14,8 +15,10 @@ register_architecture("Tifapel", TifapelConfig)
 register_architecture("Voserax", VoseraxConfig)
 register_architecture("Ninenex", NinenexConfig)
 register_architecture("Fusasun", FusasunConfig)
+register_architecture("Soputar", SoputarConfig)
 
 __all__ = [
-    "Qwen3Config", "FusasunConfig", "NinenexConfig", "TifapelConfig", "VoseraxConfig", "architectures", "config_class", "read_config", "register_architecture",
+    "Qwen3Config", "FusasunConfig", "NinenexConfig", "SoputarConfig", "TifapelConfig", "VoseraxConfig", "architectures",
+    "config_class", "read_config", "register_architecture",
     "BlockSpec", "LayerCall", "ModelSpec", "PartSpec", "TensorSpec", "default_schedule",
 ]

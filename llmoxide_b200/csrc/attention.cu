@@ -19,6 +19,8 @@
 // b*pool .. b*pool+pool-1, seen from p when b*pool+pool-1 <= p - window) is seen as one key and one value: row b of
 // a second store (pool_k, pool_v, with a block table of its own), taken first, in the same softmax.
 // With `gate` a head's output is multiplied by sigmoid(gate[t * gate_stride + hq]).
+// With `softcap` c > 0 a scaled score s becomes c * tanh(s / c) before the softmax.  With `sinks` (float32 [H]) the
+// denominator of head hq has exp(sinks[hq]) added: a learned score without key and value, neither scaled nor capped.
 //
 // One warp per (token, head).  Keys are taken 32 at a time starting at the
 // range's first key: lane j scores key lo + c*32 + j with a sequential dot over
@@ -40,7 +42,7 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
                                        float scale, float sink, int chunk, int pool,
                                        const TC* __restrict__ pool_k, const TC* __restrict__ pool_v,
                                        const int* __restrict__ pool_table, const float* __restrict__ gate,
-                                       size_t gate_stride) {
+                                       size_t gate_stride, float softcap, const float* __restrict__ sinks) {
   extern __shared__ float q_buf[];  // [ATT_WARPS][D]
   pdl_launch_dependents();
   pdl_wait();
@@ -87,6 +89,7 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
       float dot = 0.f;
       for (int i = 0; i < D; ++i) dot += qs[i] * to_f32(krow[i]);
       s = dot * scale;
+      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);  // exp(-inf) = 0 on the first chunk; lane 0 of a chunk is always live
@@ -109,7 +112,9 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
   }
   }
   // a sink: `sink` keys of score 0 that have no value; they only add to the denominator
-  float inv = 1.0f / (sink > 0.f ? l + sink * expf(-m) : l);
+  if (sink > 0.f) l += sink * expf(-m);
+  if (sinks) l += expf(sinks[hq] - m);
+  float inv = 1.0f / l;
   if (gate) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride + hq]));
   TA* orow = out + ((size_t)t * H + hq) * Dv;
 #pragma unroll
@@ -122,12 +127,14 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
 // pool > 0: pool_k / pool_v hold one row per block of `pool` positions, paged like the cache, with the block table
 // pool_table (as wide as block_table); needs a window and no kept first keys.  gate: null, or float32 with
 // gate[t * gate_stride + head] the logit of head's output gate.
-LLMX_API int llmx_attention_paged_pooled(const void* q, void* out, int act_dtype, const void* k_cache,
+// softcap <= 0: scores are not capped; sinks: null, or float32 [H].
+LLMX_API int llmx_attention_paged_capped(const void* q, void* out, int act_dtype, const void* k_cache,
                                   const void* v_cache, int cache_dtype, const int* block_table, int table_width,
                                   const int* token_seq, const int* token_pos, int n_tokens, int H, int G, int D,
                                   int Dv, long long q_stride, int window, int keep_first, float scale, float sink,
                                   int chunk, int pool, const void* pool_k, const void* pool_v, const int* pool_table,
-                                  const float* gate, long long gate_stride, cudaStream_t stream) {
+                                  const float* gate, long long gate_stride, float softcap, const float* sinks,
+                                  cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (chunk < 0 || (chunk > 0 && keep_first > 0)) return LLMX_REFUSED(1);
   if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || chunk > 0 || !pool_k || !pool_v || !pool_table)))
@@ -141,7 +148,7 @@ LLMX_API int llmx_attention_paged_pooled(const void* q, void* out, int act_dtype
   launch_pdl(attention_paged_kernel<TA, TC>, grid, dim3(ATT_WARPS * 32), smem, stream,                    \
       (const TA*)q, (TA*)out, (const TC*)k_cache, (const TC*)v_cache, block_table, table_width, token_seq, \
       token_pos, H, G, D, Dv, (size_t)q_stride, window, keep_first, scale, sink, chunk, pool, (const TC*)pool_k,  \
-      (const TC*)pool_v, pool_table, gate, (size_t)gate_stride)
+      (const TC*)pool_v, pool_table, gate, (size_t)gate_stride, softcap, sinks)
   if (act_dtype == LLMX_F32 && cache_dtype == LLMX_F32) CASE(float, float);
   else if (act_dtype == LLMX_BF16 && cache_dtype == LLMX_BF16) CASE(bf16, bf16);
   else if (act_dtype == LLMX_F32 && cache_dtype == LLMX_BF16) CASE(float, bf16);
@@ -149,6 +156,18 @@ LLMX_API int llmx_attention_paged_pooled(const void* q, void* out, int act_dtype
   else return LLMX_REFUSED(2);
 #undef CASE
   return LLMX_LAUNCH_STATUS();
+}
+
+LLMX_API int llmx_attention_paged_pooled(const void* q, void* out, int act_dtype, const void* k_cache,
+                                  const void* v_cache, int cache_dtype, const int* block_table, int table_width,
+                                  const int* token_seq, const int* token_pos, int n_tokens, int H, int G, int D,
+                                  int Dv, long long q_stride, int window, int keep_first, float scale, float sink,
+                                  int chunk, int pool, const void* pool_k, const void* pool_v, const int* pool_table,
+                                  const float* gate, long long gate_stride, cudaStream_t stream) {
+  return llmx_attention_paged_capped(q, out, act_dtype, k_cache, v_cache, cache_dtype, block_table, table_width,
+                                     token_seq, token_pos, n_tokens, H, G, D, Dv, q_stride, window, keep_first, scale,
+                                     sink, chunk, pool, pool_k, pool_v, pool_table, gate, gate_stride, 0.f, nullptr,
+                                     stream);
 }
 
 LLMX_API int llmx_attention_paged_chunked(const void* q, void* out, int act_dtype, const void* k_cache,

@@ -14,6 +14,9 @@
 // Shared memory holds the query tile and two stages of (K page, V page),
 // filled by cp.async in 16-byte chunks whose position in a row is XORed with
 // the row number so that ldmatrix reads are free of bank conflicts.
+//
+// Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own) every scaled score is capped (common.cuh).
+// `sinks` (float32 [H]): exp(sinks[h]) joins head h's denominator once.
 #include "common.cuh"
 
 #define PF_BQ 64          // query tokens per CTA (4 warps x 16 rows)
@@ -65,7 +68,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, con
                          const int* __restrict__ seq_start, const int* __restrict__ seq_past, int H, int G,
                          int window, int keep_first, int mask_chunk, float scale_log2, float sink, int pool_arg,
                          const bf16* __restrict__ pool_k, const bf16* __restrict__ pool_v,
-                         const int* __restrict__ pool_table) {
+                         const int* __restrict__ pool_table, const float* __restrict__ sinks, const ScoreCap cap) {
   const int pool = POOLED ? pool_arg : 0;
   constexpr int CHUNKS = D / 8;              // 16-byte chunks per row
   constexpr int KSTEPS = D / 16;             // k-steps of the score product
@@ -202,8 +205,13 @@ attention_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, con
         const int key = key0 + 8 * j + 2 * (lane & 3) + e;
         const bool v0 = pooled ? key < nb0 : ((key >= f0 || key < keep_first) && key <= p0);
         const bool v1 = pooled ? key < nb1 : ((key >= f1 || key < keep_first) && key <= p1);
+#if LLMX_SCORE_CAP
+        s[j][e] = v0 ? capped_score_log2(cap, s[j][e]) : -INFINITY;
+        s[j][2 + e] = v1 ? capped_score_log2(cap, s[j][2 + e]) : -INFINITY;
+#else
         s[j][e] = v0 ? s[j][e] * scale_log2 : -INFINITY;
         s[j][2 + e] = v1 ? s[j][2 + e] * scale_log2 : -INFINITY;
+#endif
         mx0 = fmaxf(mx0, s[j][e]);
         mx1 = fmaxf(mx1, s[j][2 + e]);
       }
@@ -264,6 +272,11 @@ attention_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, con
     l0 += sink * exp2f(-m0);
     l1 += sink * exp2f(-m1);
   }
+  if (sinks) {
+    const float sk = sinks[hq] * 1.4426950408889634f;
+    l0 += exp2f(sk - m0);
+    l1 += exp2f(sk - m1);
+  }
   const float inv0 = 1.0f / l0, inv1 = 1.0f / l1;
   const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
 #pragma unroll
@@ -282,7 +295,8 @@ template <int D, bool POOLED>
 static int launch_prefill_as(const void* q, void* out, const void* k_cache, const void* v_cache, const int* block_table,
                           int table_width, const int* seq_start, const int* seq_past, int B, int max_new, int H,
                           int G, int window, int keep_first, int mask_chunk, float scale, float sink, int pool,
-                          const void* pool_k, const void* pool_v, const int* pool_table, cudaStream_t stream) {
+                          const void* pool_k, const void* pool_v, const int* pool_table, const float* sinks,
+                          float softcap, cudaStream_t stream) {
   const size_t smem = (size_t)PF_BQ * D * 2 + 4 * (size_t)PF_BK * D * 2;
   auto kernel = attention_prefill_kernel<D, POOLED>;
   static bool attr_set = false;
@@ -295,13 +309,17 @@ static int launch_prefill_as(const void* q, void* out, const void* k_cache, cons
   launch_pdl(kernel, grid, dim3(PF_THREADS), smem, stream, (const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache,
                                              block_table, table_width, seq_start, seq_past, H, G, window,
                                              keep_first, mask_chunk, scale * 1.4426950408889634f, sink, pool,
-                                             (const bf16*)pool_k, (const bf16*)pool_v, pool_table);
+                                             (const bf16*)pool_k, (const bf16*)pool_v, pool_table, sinks,
+                                             make_score_cap(scale, softcap));
   return LLMX_LAUNCH_STATUS();
 }
 
 template <int D, typename... Args>
 static int launch_prefill(int pool, Args... args) {
-  return pool > 0 ? launch_prefill_as<D, true>(args...) : launch_prefill_as<D, false>(args...);
+#if !LLMX_SCORE_CAP            // (pooled blocks beside capped scores are not built)
+  if (pool > 0) return launch_prefill_as<D, true>(args...);
+#endif
+  return launch_prefill_as<D, false>(args...);
 }
 
 // q, out: bf16 [T, H*D], tokens packed sequence after sequence; seq_start [B+1] offsets into the packed
@@ -312,13 +330,15 @@ static int launch_prefill(int pool, Args... args) {
 // pool n > 0 (beside a window, without kept first keys or a chunked mask): every block of n positions that lies
 // wholly before a query's window is seen as row b of pool_k / pool_v, a second store paged like the cache with the
 // block table pool_table (as wide as block_table).
-LLMX_API int llmx_attention_prefill_pooled(const void* q, void* out, const void* k_cache, const void* v_cache,
+// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it.
+LLMX_API int llmx_attention_prefill_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
                                            const int* block_table, int table_width, const int* seq_start,
                                            const int* seq_past, int B, int max_new, int H, int G, int D, int window,
                                            int keep_first, int mask_chunk, float scale, float sink, int pool,
                                            const void* pool_k, const void* pool_v, const int* pool_table,
-                                           cudaStream_t stream) {
+                                           const float* sinks, float softcap, cudaStream_t stream) {
   if (B <= 0 || max_new <= 0) return 0;
+  if ((softcap > 0.f) != (LLMX_SCORE_CAP != 0) || (LLMX_SCORE_CAP && pool > 0)) return LLMX_REFUSED(1);
   if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || mask_chunk > 0 || !pool_k || !pool_v || !pool_table ||
                                 ((uintptr_t)pool_k & 15) || ((uintptr_t)pool_v & 15))))
     return LLMX_REFUSED(1);
@@ -329,12 +349,23 @@ LLMX_API int llmx_attention_prefill_pooled(const void* q, void* out, const void*
   if (D == 128)
     return launch_prefill<128>(pool, q, out, k_cache, v_cache, block_table, table_width, seq_start, seq_past, B, max_new,
                                H, G, window, window > 0 ? keep_first : 0, mask_chunk, scale, sink, pool, pool_k, pool_v,
-                               pool_table, stream);
+                               pool_table, sinks, softcap, stream);
   if (D == 64)
     return launch_prefill<64>(pool, q, out, k_cache, v_cache, block_table, table_width, seq_start, seq_past, B, max_new, H,
                               G, window, window > 0 ? keep_first : 0, mask_chunk, scale, sink, pool, pool_k, pool_v,
-                              pool_table, stream);
+                              pool_table, sinks, softcap, stream);
   return LLMX_REFUSED(1);
+}
+
+LLMX_API int llmx_attention_prefill_pooled(const void* q, void* out, const void* k_cache, const void* v_cache,
+                                           const int* block_table, int table_width, const int* seq_start,
+                                           const int* seq_past, int B, int max_new, int H, int G, int D, int window,
+                                           int keep_first, int mask_chunk, float scale, float sink, int pool,
+                                           const void* pool_k, const void* pool_v, const int* pool_table,
+                                           cudaStream_t stream) {
+  return llmx_attention_prefill_capped(q, out, k_cache, v_cache, block_table, table_width, seq_start, seq_past, B,
+                                       max_new, H, G, D, window, keep_first, mask_chunk, scale, sink, pool, pool_k, pool_v,
+                                       pool_table, nullptr, 0.f, stream);
 }
 
 LLMX_API int llmx_attention_prefill_masked(const void* q, void* out, const void* k_cache, const void* v_cache,

@@ -30,6 +30,9 @@
 // so two CTAs share it: while one's softmax warps wait for a tensor-memory load
 // or the special-function unit, the other's run.  Every mbarrier wait is
 // bounded; a wait that runs out sets the status word and the CTA winds down.
+//
+// Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own) every scaled score is capped (common.cuh).
+// `sinks` (float32 [H]): exp(sinks[h]) joins head h's denominator once.
 #include "tc_ptx.cuh"
 
 #define AT_ROWS 128        // query rows per CTA = MMA M
@@ -60,7 +63,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
                             const int* __restrict__ block_table, int table_width, const int* __restrict__ seq_start,
                             const int* __restrict__ seq_past, int H, int G, int window, int keep_first,
-                            int mask_chunk, float scale_log2, float sink) {
+                            int mask_chunk, float scale_log2_arg, float sink, const float* __restrict__ sinks,
+                            const ScoreCap cap) {
+#if LLMX_SCORE_CAP
+  constexpr float scale_log2 = 1.0f;           // the capped scores are base-2 logarithms already
+#else
+  const float scale_log2 = scale_log2_arg;
+#endif
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   pdl_launch_dependents();
   pdl_wait();
@@ -215,6 +224,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
       for (int c = 0; c < AT_KEYS; c += 32) tmem_ld32_nowait(tS + (uint32_t)c, sr + c);
       tmem_ld_wait();
+#if LLMX_SCORE_CAP
+#pragma unroll
+      for (int e = 0; e < AT_KEYS; ++e) {       // (as capped_score_log2, with the one-instruction exponential)
+        const float ex = ex2_approx(cap.mul * __uint_as_float(sr[e]));
+        sr[e] = __float_as_uint(cap.top - __fdividef(2.0f * cap.top, 1.0f + ex));
+      }
+#endif
       // Tiles that some row of this CTA sees only in part (the diagonal, a window's edge, rows past the
       // sequence's end) are masked; the others, which is most of them, skip the compares.
       const bool edge = (key0 + AT_KEYS - 1 > pos_lo) || (window > 0 && key0 < pos_hi - (window - 1)) ||
@@ -309,6 +325,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (ok) {
       tc_fence_after();
       // a sink: `sink` keys of score 0 without a value; they only add to the denominator (l is in units of 2^-m_used)
+      if (sinks && row_live) l += exp2f(sinks[hq] * 1.4426950408889634f - m_used);
       const float inv = 1.0f / ((sink > 0.f && row_live) ? l + sink * exp2f(-m_used) : l);
       bf16* orow = out + ((size_t)(tok0 + i0 + row) * H + hq) * AT_D;
 #pragma unroll 1
@@ -346,12 +363,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 // max_new = most new tokens of a sequence.
 // mask_chunk n > 0: a query sees only the keys of its own chunk of n positions, counted from the sequence's
 // position 0 (no kept first keys then).
-LLMX_API int llmx_attention_prefill_tc_masked(const void* q, void* out, const void* k_cache, const void* v_cache,
+// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it.
+LLMX_API int llmx_attention_prefill_tc_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
                                               long long n_pages, const int* block_table, int table_width,
                                               const int* seq_start, const int* seq_past, int B, int T, int max_new,
                                               int H, int G, int D, int window, int keep_first, int mask_chunk,
-                                              float scale, float sink, cudaStream_t stream) {
+                                              float scale, float sink, const float* sinks, float softcap,
+                                              cudaStream_t stream) {
   if (B <= 0 || max_new <= 0 || T <= 0) return 0;
+  if ((softcap > 0.f) != (LLMX_SCORE_CAP != 0)) return LLMX_REFUSED(1);
   if (window <= 0) keep_first = 0;
   if (mask_chunk < 0 || (mask_chunk > 0 && keep_first > 0)) return LLMX_REFUSED(1);
   if (D != AT_D || H <= 0 || G <= 0 || H % G || window < 0 || keep_first < 0 || B > 65535 || (max_new + AT_ROWS - 1) / AT_ROWS > 65535 || n_pages <= 0)
@@ -376,8 +396,19 @@ LLMX_API int llmx_attention_prefill_tc_masked(const void* q, void* out, const vo
   }
   dim3 grid(H, (max_new + AT_ROWS - 1) / AT_ROWS, B);
   launch_pdl(attention_prefill_tc_kernel, grid, dim3(AT_THREADS), smem, stream, mq, mk, mv, (bf16*)out, block_table,
-             table_width, seq_start, seq_past, H, G, window, keep_first, mask_chunk, scale * 1.4426950408889634f, sink);
+             table_width, seq_start, seq_past, H, G, window, keep_first, mask_chunk, scale * 1.4426950408889634f, sink,
+             sinks, make_score_cap(scale, softcap));
   return LLMX_LAUNCH_STATUS();
+}
+
+LLMX_API int llmx_attention_prefill_tc_masked(const void* q, void* out, const void* k_cache, const void* v_cache,
+                                              long long n_pages, const int* block_table, int table_width,
+                                              const int* seq_start, const int* seq_past, int B, int T, int max_new,
+                                              int H, int G, int D, int window, int keep_first, int mask_chunk,
+                                              float scale, float sink, cudaStream_t stream) {
+  return llmx_attention_prefill_tc_capped(q, out, k_cache, v_cache, n_pages, block_table, table_width, seq_start, seq_past,
+                                          B, T, max_new, H, G, D, window, keep_first, mask_chunk, scale, sink, nullptr,
+                                          0.f, stream);
 }
 
 LLMX_API int llmx_attention_prefill_tc(const void* q, void* out, const void* k_cache, const void* v_cache,

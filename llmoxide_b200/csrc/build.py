@@ -32,19 +32,25 @@ from ..errors import ExtensionMissing
 SRC_DIR = Path(__file__).resolve().parent
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC,-fvisibility=hidden", "-shared"]
-# library name -> (source files, extra link flags)
+# library name -> (source files, extra compiler flags)
 LIBRARIES = {
     "elementwise": (["elementwise.cu"], []),
     "attention": (["attention.cu"], []),
     "attention_decode": (["attention_decode.cu"], []),
     "attention_prefill": (["attention_prefill.cu"], []),
     "attention_prefill_tc": (["attention_prefill_tc.cu"], []),
+    # the tiled attention kernels once more, with every score capped
+    "attention_decode_capped": (["attention_decode.cu"], ["-DLLMX_SCORE_CAP=1"]),
+    "attention_prefill_capped": (["attention_prefill.cu"], ["-DLLMX_SCORE_CAP=1"]),
+    "attention_prefill_tc_capped": (["attention_prefill_tc.cu"], ["-DLLMX_SCORE_CAP=1"]),
+    "delta_rule": (["delta_rule.cu"], []),
     "gemm_fma": (["gemm_fma.cu"], []),
     "gemm_tc": (["gemm_tc.cu"], []),
     "linear_attention": (["linear_attention.cu"], []),
     "latent_attention": (["latent_attention.cu"], []),
     "moe": (["moe.cu"], []),
     "post_norm": (["post_norm.cu"], []),
+    "qk_row_norm": (["qk_row_norm.cu"], []),
     "moe_tc": (["moe_tc.cu"], []),
     "short_conv": (["short_conv.cu"], []),
     "stream_mix": (["stream_mix.cu"], []),

@@ -195,6 +195,29 @@ template <typename T> __device__ __forceinline__ T from_f32(float x);
 template <> __device__ __forceinline__ float from_f32<float>(float x) { return x; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float x) { return __float2bfloat16_rn(x); }
 
+// Capped attention scores.  The tiled attention kernels are compiled twice, with LLMX_SCORE_CAP 0 and 1; the second
+// library caps every scaled score s at c: c * tanh(s / c).  They keep scores in base-2 logarithms, where that is
+// top * tanh(z) = top - 2 top / (1 + 2^(mul * raw)) for the unscaled product `raw`, top = c log2(e) and
+// mul = 2 log2(e) scale / c: one exponential and one division, off by a few 1e-7 of top.  A product that overflows
+// the exponential gives the limits +-top.
+#ifndef LLMX_SCORE_CAP
+#define LLMX_SCORE_CAP 0
+#endif
+struct ScoreCap {
+  float mul, top;
+};
+__device__ __forceinline__ float capped_score_log2(const ScoreCap c, float raw) {
+  return c.top - __fdividef(2.0f * c.top, 1.0f + exp2f(c.mul * raw));
+}
+static inline ScoreCap make_score_cap(float scale, float softcap) {
+  ScoreCap c = {0.f, 0.f};
+  if (softcap > 0.f) {
+    c.mul = 2.0f * 1.4426950408889634f * scale / softcap;
+    c.top = softcap * 1.4426950408889634f;
+  }
+  return c;
+}
+
 // Gated activations of the feed-forwards, act(g) * f(u):
 //   SILU            g sigmoid(g) * u
 //   RELU            max(g, 0) * u

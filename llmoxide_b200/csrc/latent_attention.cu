@@ -5,7 +5,7 @@
 // part (R) | head gates (H) ], float32 or split float32 partials.
 //
 // latent_norms: cq = rms(down[:Rq]) * gq and c = rms(down[Rq : Rq+Rkv]) * gkv, x / sqrt(mean(x^2) + eps), float32
-// statistics, written in the compute dtype as the operands of the two up-projections.  One CTA of 128 threads per
+// statistics, written in the compute dtype as the operands of the two up-projections (Rq 0: only the second).  One CTA of 128 threads per
 // token; sums in an order fixed by the width alone.
 //
 // latent_rope_cache: per (token, head), from q [T, H, R + D] (up-projected queries, every head [rotated part |
@@ -33,7 +33,7 @@ __global__ void latent_norms_kernel(const TIN* __restrict__ down, int n_split, s
                                     TA* __restrict__ cq, TA* __restrict__ c, int Rq, int Rkv) {
   __shared__ float red[32];
   pdl_launch_dependents();
-  const int t = blockIdx.x, which = blockIdx.y;          // which: 0 the query latent, 1 the key/value latent
+  const int t = blockIdx.x, which = Rq > 0 ? blockIdx.y : 1;     // which: 0 the query latent, 1 the key/value latent
   const int n = which ? Rkv : Rq;
   const TIN* src = down + (size_t)t * row_stride + (which ? Rq : 0);
   const float* gain = which ? kv_gain : q_gain;
@@ -158,8 +158,9 @@ LLMX_API int llmx_latent_norms(const void* down, int in_dtype, int n_split, long
                                long long row_stride, const float* q_gain, const float* kv_gain, float eps, void* cq,
                                void* c, int act_dtype, int n_tokens, int Rq, int Rkv, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (Rq <= 0 || Rkv <= 0 || n_split < 1 || row_stride < Rq + Rkv || !q_gain || !kv_gain) return LLMX_REFUSED(1);
-  dim3 grid(n_tokens, 2);
+  if (Rq < 0 || Rkv <= 0 || n_split < 1 || row_stride < Rq + Rkv || (Rq > 0 && (!q_gain || !cq)) || !kv_gain)
+    return LLMX_REFUSED(1);
+  dim3 grid(n_tokens, Rq > 0 ? 2 : 1);
 #define CASE(TIN, TA)                                                                                          \
   launch_pdl(latent_norms_kernel<TIN, TA>, grid, dim3(128), 0, stream, (const TIN*)down, n_split,               \
              (size_t)split_stride, (size_t)row_stride, q_gain, kv_gain, eps, (TA*)cq, (TA*)c, Rq, Rkv)

@@ -8,7 +8,8 @@
 //   y = y * sigmoid(z[t,:] + zb)                      when a gate z is given (z: partials added in order like a group's)
 //   y = norm(y) * post_gain                           when post_gain is given (else y joins as it is)
 //   v = h[t,:] + y;  h[t,:] = v when write_h
-//   out[r,:] = norm(v) * gain                         when out is given
+//   out[r,:] = norm(v) * gain                         when out is given; without a gain out = v as it is (the next
+//                                                     sublayer reads the stream itself)
 // Either norm is a layer norm without bias, (x - mean) / sqrt(mean((x - mean)^2) + eps), or an RMS norm,
 // x / sqrt(mean(x^2) + eps); the two norms choose independently (`post_center`, `center`).  Everything is float32;
 // mean and variance are taken in two passes over the row, which is held in registers (rows of up to 8192 aligned
@@ -159,9 +160,13 @@ post_norm_add_norm_kernel(float* __restrict__ h, const PnGroup g0, const PnGroup
   }
   if (!out) return;
   __syncthreads();
+  TO* orow = out + (size_t)r * d;
+  if (!gain) {
+    for (int i = threadIdx.x; i < d; i += blockDim.x) orow[i] = from_f32<TO>(pn_row[i]);
+    return;
+  }
   float mean, rstd;
   pn_stats(pn_row, d, center != 0, eps, red, mean, rstd);
-  TO* orow = out + (size_t)r * d;
   if (VEC) {
     for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
       const float4 v = pn_load4(pn_row + i), g = pn_load4(gain + i);
@@ -263,9 +268,15 @@ post_norm_add_norm_reg_kernel(float* __restrict__ h, const PnGroup g0, const PnG
     for (int k = 0; k < NV; ++k) v[k] = live[k] ? pn_load4(hrow + col[k]) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   if (!out) return;
+  TO* orow = out + (size_t)r * d;
+  if (!gain) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+      if (live[k]) pn_store4(orow + col[k], v[k]);
+    return;
+  }
   float mean, rstd;
   pn_stats_reg<NV>(v, live, d, center != 0, eps, red, mean, rstd);
-  TO* orow = out + (size_t)r * d;
 #pragma unroll
   for (int k = 0; k < NV; ++k)
     if (live[k]) {
@@ -290,7 +301,7 @@ LLMX_API int llmx_post_norm_add_norm_gated(float* h, const void* delta0, int dty
   if (gate && (!delta0 || gate_split < 1 || (gate_dtype != LLMX_F32 && gate_dtype != LLMX_BF16))) return LLMX_REFUSED(1);
   const PnGroup gz = {gate, gate_split, gate_dtype == LLMX_BF16, (size_t)gate_stride, 1.0f};
   const float* zb = gate ? gate_bias : nullptr;
-  if (d <= 0 || (delta0 && n_split0 < 1) || (delta1 && (n_split1 < 1 || !delta0)) || (out && !gain))
+  if (d <= 0 || (delta0 && n_split0 < 1) || (delta1 && (n_split1 < 1 || !delta0)))
     return LLMX_REFUSED(1);
   if ((delta0 && dtype0 != LLMX_F32 && dtype0 != LLMX_BF16) || (delta1 && dtype1 != LLMX_F32 && dtype1 != LLMX_BF16))
     return LLMX_REFUSED(2);

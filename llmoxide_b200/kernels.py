@@ -122,7 +122,8 @@ def _library(lib_name: str):
 # waited for a step anyway (no copy, no extra synchronisation).
 
 _STATUS_SLOTS = {"gemm_tc": 0, "attention_prefill_tc": 1, "attention_decode": 2, "sampling": 3, "moe_tc": 4,
-                 "short_conv": 5, "stream_mix": 6, "moe": 7, "attention": 8, "latent_attention": 9}
+                 "short_conv": 5, "stream_mix": 6, "moe": 7, "attention": 8, "latent_attention": 9,
+                 "attention_prefill_tc_capped": 10, "attention_decode_capped": 11, "qk_row_norm": 12, "delta_rule": 13}
 _STATUS_MEANING = {
     "gemm_tc": {1: "the producer's wait for a free stage ran out", 2: "the MMA issuer's wait for a stage's data ran out",
                 3: "the epilogue's wait for an accumulator ran out", 4: "the MMA issuer's wait for a drained accumulator ran out",
@@ -143,7 +144,14 @@ _STATUS_MEANING = {
     "attention": {1: "a block's row has no page in the store of one row per block",
                   2: "a block's positions are no longer held by the cache"},
     "latent_attention": {1: "a token's sequence, position or page lies outside the launch's arrays"},
+    "qk_row_norm": {1: "a token's sequence, position or page lies outside the launch's arrays"},
+    "delta_rule": {1: "a sequence's rows or slot lie outside the launch's arrays (preparation)",
+                   2: "a sequence's slot lies outside the state area",
+                   3: "a sequence's rows or slot lie outside the launch's arrays (convolution rows)",
+                   4: "a sequence's position or slot lies outside the launch's arrays (single tokens)"},
 }
+for _capped in ("attention_prefill_tc", "attention_decode"):
+    _STATUS_MEANING[_capped + "_capped"] = _STATUS_MEANING[_capped]
 _status_host = None
 
 
@@ -151,7 +159,7 @@ def status_words() -> torch.Tensor:
     """The page-locked int32 words, one per library that reports (see ``_STATUS_SLOTS``)."""
     global _status_host
     if _status_host is None:
-        _status_host = torch.zeros(16, dtype=torch.int32).pin_memory()
+        _status_host = torch.zeros(32, dtype=torch.int32).pin_memory()
     return _status_host
 
 
@@ -412,7 +420,8 @@ def post_norm_add_norm(h, groups, bias, post_gain, post_center: bool, post_eps: 
     """A sublayer's result normed before it joins the residual stream ``h`` (float32 [T, d], in place), and the norm
     the next sublayer reads.  ``groups``: up to two (delta, weight), delta [T, d] or split partials [S, T, d] summed
     in order; y = sum_g weight_g * delta_g + ``bias``; with ``post_gain`` y = norm(y) * post_gain; v = h + y (stored
-    when ``write_h``); with ``out`` out[r] = norm(v[rows[r]]) * gain (every row without ``rows``).  A norm with
+    when ``write_h``); with ``out`` out[r] = norm(v[rows[r]]) * gain (every row without ``rows``; ``gain`` None: v as it
+    is, for a sublayer that reads the stream itself).  A norm with
     ``center`` subtracts the mean (layer norm without bias), without it is an RMS norm; both are float32.
     ``gate`` = (z, b): y is multiplied by sigmoid(z + b) element by element before its norm; z [T, d] or split
     partials [S, T, d], b float32 [d] or None."""
@@ -557,18 +566,24 @@ def sum_splits(parts: torch.Tensor, out: torch.Tensor) -> None:
              _stream()), "sum_splits")
 
 
+def _check_sinks(sinks, n_heads: int) -> None:
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads and sinks.is_contiguous())
+
+
 def attention_paged(q, out, k_cache, v_cache, block_table, token_seq, token_pos, n_heads: int,
                     n_kv_heads: int, head_dim: int, window, scale: float, v_head_dim=None, keep_first: int = 0,
                     sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None,
-                    gate=None) -> None:
+                    gate=None, softcap: float = 0.0, sinks=None) -> None:
     """General attention over the paged cache; q [T,H*D] (rows may be the first columns of wider rows), out
     [T,H*Dv].  Under a window the first ``keep_first`` keys of a sequence stay visible.  ``sink`` is added to the
     softmax's denominator (as many keys of score 0 that have no value).  With ``chunk`` n > 0 a query sees only the
     keys of its own chunk of n positions, counted from the sequence's position 0.  With ``pool`` n > 0 (beside a
     window) every block of n positions that lies wholly before the window is seen as row b of ``pool_k`` / ``pool_v``
     (paged like the cache, block table ``pool_table``).  ``gate`` float32 [T, >= H] (a view with any row stride):
-    head h's output is multiplied by sigmoid(gate[t, h])."""
-    _dev(q, out, k_cache, v_cache, block_table, token_seq, token_pos, pool_k, pool_v, pool_table, gate)
+    head h's output is multiplied by sigmoid(gate[t, h]).  ``softcap`` c > 0: every scaled score s becomes
+    c * tanh(s / c).  ``sinks`` float32 [H]: exp(sinks[h]) joins head h's denominator (no key, no value, not capped)."""
+    _dev(q, out, k_cache, v_cache, block_table, token_seq, token_pos, pool_k, pool_v, pool_table, gate, sinks)
+    _check_sinks(sinks, n_heads)
     _contig("out", out), _contig("block_table", block_table)
     if pool:
         _contig("pool_table", pool_table)
@@ -581,15 +596,15 @@ def attention_paged(q, out, k_cache, v_cache, block_table, token_seq, token_pos,
         raise Unsupported(f"head_dim {head_dim}/{v_head_dim}: the general attention kernel takes sizes up to 256")
     if n_heads % n_kv_heads:
         raise Unsupported(f"{n_heads} heads are not a multiple of {n_kv_heads} kv heads")
-    f = _fn("attention", "llmx_attention_paged_pooled",
+    f = _fn("attention", "llmx_attention_paged_capped",
             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
              c_int, c_int, c_int, c_int, c_int, c_longlong, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p,
-             c_void_p, c_void_p, c_void_p, c_longlong, c_void_p])
+             c_void_p, c_void_p, c_void_p, c_longlong, c_float, c_void_p, c_void_p])
     _check(f(_ptr(q), _ptr(out), _tag(q), _ptr(k_cache), _ptr(v_cache), _tag(k_cache), _ptr(block_table),
              block_table.shape[1], _ptr(token_seq), _ptr(token_pos), q.shape[0], n_heads, n_kv_heads, head_dim,
              v_head_dim, q.stride(0), int(window or 0), int(keep_first or 0), scale, float(sink or 0.0), int(chunk or 0),
              int(pool or 0), _ptr(pool_k), _ptr(pool_v), _ptr(pool_table), _ptr(gate),
-             gate.stride(0) if gate is not None else 0, _stream()), "attention_paged")
+             gate.stride(0) if gate is not None else 0, float(softcap or 0.0), _ptr(sinks), _stream()), "attention_paged")
 
 
 def pool_blocks(k_cache, v_cache, block_table, pool_k, pool_v, pool_table, seq_start, seq_past, n_seqs: int,
@@ -611,20 +626,23 @@ def pool_blocks(k_cache, v_cache, block_table, pool_k, pool_v, pool_table, seq_s
 
 
 def latent_norms(down, q_gain, kv_gain, eps: float, cq, c, q_rank: int, kv_rank: int) -> None:
-    """The two latents of a latent attention out of its fused first product: ``down`` [T, >= q_rank + kv_rank]
+    """The two latents of a latent attention (``q_rank`` 0, ``q_gain`` and ``cq`` None: only the key/value latent) out
+    of its fused first product: ``down`` [T, >= q_rank + kv_rank]
     (or float32 split partials [S, T, ..]) -> cq = rms(down[:, :q_rank]) * q_gain, c = rms(down[:, q_rank :
     q_rank + kv_rank]) * kv_gain, float32 statistics, in the dtype of ``cq`` and ``c``."""
     _dev(down, q_gain, kv_gain, cq, c)
-    _contig("down", down), _contig("cq", cq), _contig("c", c)
+    _contig("down", down), _contig("c", c)
     n_split, stride = (down.shape[0], down.stride(0)) if down.dim() == 3 else (1, 0)
     T = down.shape[-2]
-    assert cq.shape == (T, q_rank) and c.shape == (T, kv_rank) and cq.dtype == c.dtype
-    assert q_gain.dtype == kv_gain.dtype == torch.float32 and q_gain.numel() == q_rank and kv_gain.numel() == kv_rank
+    assert c.shape == (T, kv_rank) and kv_gain.dtype == torch.float32 and kv_gain.numel() == kv_rank
+    if q_rank:
+        _contig("cq", cq)
+        assert cq.shape == (T, q_rank) and cq.dtype == c.dtype and q_gain.dtype == torch.float32 and q_gain.numel() == q_rank
     f = _fn("latent_attention", "llmx_latent_norms",
             [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
              c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(down), _tag(down), n_split, stride, down.shape[-1], _ptr(q_gain), _ptr(kv_gain), eps, _ptr(cq),
-             _ptr(c), _tag(cq), T, q_rank, kv_rank, _stream()), "latent_norms")
+             _ptr(c), _tag(c), T, q_rank, kv_rank, _stream()), "latent_norms")
 
 
 def latent_rope_cache(q, kv, down, k_rot_off: int, q_out, k_cache, v_cache, block_table, ctx, cos, sin, n_heads: int,
@@ -702,15 +720,23 @@ def _counters(device, n: int):
     return buf
 
 
+def capped_library(name: str, softcap) -> str:
+    """The library of a tiled attention kernel: its own build where scores are capped."""
+    return name + "_capped" if softcap else name
+
+
 def attention_decode(q, out, k_cache, v_cache, block_table, seq_past, n_heads: int, n_kv_heads: int,
                      head_dim: int, window, scale: float, n_chunks: int = 0, keep_first: int = 0,
-                     sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None) -> None:
+                     sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None,
+                     softcap: float = 0.0, sinks=None) -> None:
     """One new token per sequence, bfloat16: q, out [B,H*D] in batch order;
     seq_past[b] is the token's position.  Each sequence's keys are split over
     n_chunks CTAs (0: chosen from the batch's shape), which merge inside a
     cluster, or beyond 8 chunks through a float32 workspace.  ``chunk`` n > 0 is
-    the chunked mask of ``attention_paged`` (nothing to do with n_chunks); ``pool`` with its second store likewise."""
-    _dev(q, out, k_cache, v_cache, block_table, seq_past, pool_k, pool_v, pool_table)
+    the chunked mask of ``attention_paged`` (nothing to do with n_chunks); ``pool`` with its second store, ``softcap`` and ``sinks``
+    likewise (capped scores run in a library of their own; no pooled blocks there)."""
+    _dev(q, out, k_cache, v_cache, block_table, seq_past, pool_k, pool_v, pool_table, sinks)
+    _check_sinks(sinks, n_heads)
     _contig("q", q), _contig("out", out), _contig("block_table", block_table)
     if pool:
         _contig("pool_table", pool_table)
@@ -734,14 +760,15 @@ def attention_decode(q, out, k_cache, v_cache, block_table, seq_past, n_heads: i
         ws = guard.scratch((B * n_heads * n_chunks * (head_dim + 4),), torch.float32, q.device,
                            "decode attention workspace")
         counters = _counters(q.device, B * n_kv_heads * ((group + 7) // 8))
-    f = _fn("attention_decode", "llmx_attention_decode_pooled",
+    f = _fn(capped_library("attention_decode", softcap), "llmx_attention_decode_capped",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_longlong,
-             c_void_p, c_void_p])
+             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float, c_int, c_int, c_void_p,
+             c_void_p, c_longlong, c_void_p, c_void_p])
     _check(f(_ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(block_table),
              block_table.shape[1],
              _ptr(seq_past), _ptr(ws), _ptr(counters), B, n_heads, n_kv_heads, head_dim, int(window or 0),
-             int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0), n_chunks, int(pool or 0), _ptr(pool_k),
+             int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0), _ptr(sinks), float(softcap or 0.0), n_chunks,
+             int(pool or 0), _ptr(pool_k),
              _ptr(pool_v), pool_k.shape[0] if pool else 0, _ptr(pool_table), _stream()), "attention_decode")
 
 
@@ -758,11 +785,14 @@ def attention_prefill_supports(q, k_cache, head_dim: int) -> bool:
 
 def attention_prefill(q, out, k_cache, v_cache, block_table, seq_start, seq_past, n_seqs: int, max_new: int,
                       n_heads: int, n_kv_heads: int, head_dim: int, window, scale: float, keep_first: int = 0,
-                      sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None) -> None:
+                      sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None,
+                      softcap: float = 0.0, sinks=None) -> None:
     """Prompt attention on the tensor cores, bfloat16, head sizes 64 and 128:
     q, out [T,H*D] packed sequence after sequence.  Under a window the first ``keep_first`` keys stay visible;
-    ``chunk`` n > 0 is the chunked mask of ``attention_paged``, ``pool`` with its second store its pooled blocks."""
-    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, pool_k, pool_v, pool_table)
+    ``chunk`` n > 0 is the chunked mask of ``attention_paged``, ``pool`` with its second store its pooled blocks;
+    ``softcap`` and ``sinks`` as there (capped scores run in a library of their own; no pooled blocks there)."""
+    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, pool_k, pool_v, pool_table, sinks)
+    _check_sinks(sinks, n_heads)
     _contig("q", q), _contig("out", out), _contig("block_table", block_table)
     if pool:
         _contig("pool_table", pool_table)
@@ -770,33 +800,35 @@ def attention_prefill(q, out, k_cache, v_cache, block_table, seq_start, seq_past
         assert pool_k.is_contiguous() and pool_v.is_contiguous() and pool_k.shape[1:] == k_cache.shape[1:]
     if not attention_prefill_supports(q, k_cache, head_dim):
         raise Unsupported(f"the tiled prompt attention takes bfloat16 and head sizes 64 or 128, not {head_dim}")
-    f = _fn("attention_prefill", "llmx_attention_prefill_pooled",
+    f = _fn(capped_library("attention_prefill", softcap), "llmx_attention_prefill_capped",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-             c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
+             c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
+             c_void_p])
     _check(f(_ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
              _ptr(seq_start), _ptr(seq_past), n_seqs, max_new, n_heads, n_kv_heads, head_dim, int(window or 0),
              int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0), int(pool or 0), _ptr(pool_k), _ptr(pool_v),
-             _ptr(pool_table), _stream()), "attention_prefill")
+             _ptr(pool_table), _ptr(sinks), float(softcap or 0.0), _stream()), "attention_prefill")
 
 
 def attention_prefill_tc(q, out, k_cache, v_cache, block_table, seq_start, seq_past, n_seqs: int, max_new: int,
                          n_heads: int, n_kv_heads: int, head_dim: int, window, scale: float, keep_first: int = 0,
-                         sink: float = 0.0, chunk: int = 0) -> None:
+                         sink: float = 0.0, chunk: int = 0, softcap: float = 0.0, sinks=None) -> None:
     """Prompt attention on tcgen05, bfloat16, head size 128: q, out [T,H*128]
     packed sequence after sequence; the cache entry is [n_pages,G,64,128].  ``chunk`` n > 0 is the chunked mask
-    of ``attention_paged``."""
-    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past)
+    of ``attention_paged``, ``softcap`` and ``sinks`` as there (capped scores run in a library of their own)."""
+    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, sinks)
+    _check_sinks(sinks, n_heads)
     _contig("q", q), _contig("out", out), _contig("block_table", block_table)
     assert k_cache.is_contiguous() and v_cache.is_contiguous()
     if head_dim != 128 or q.dtype != torch.bfloat16 or k_cache.dtype != torch.bfloat16:
         raise Unsupported("the tcgen05 prompt attention takes bfloat16 and head size 128")
-    f = _fn("attention_prefill_tc", "llmx_attention_prefill_tc_masked",
+    f = _fn(capped_library("attention_prefill_tc", softcap), "llmx_attention_prefill_tc_capped",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float, c_void_p])
     _check(f(_ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(block_table),
              block_table.shape[1], _ptr(seq_start), _ptr(seq_past), n_seqs, q.shape[0], max_new, n_heads,
              n_kv_heads, head_dim, int(window or 0), int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0),
-             _stream()), "attention_prefill_tc")
+             _ptr(sinks), float(softcap or 0.0), _stream()), "attention_prefill_tc")
 
 
 def attention_prefill_tc_status(reset: bool = True) -> int:
@@ -1061,6 +1093,96 @@ def gate_scan(proj, i_off: int, f_off: int, bias_i, bias_f, cap: float, gates, s
     _check(f(_ptr(proj), _tag(proj), n_split, split_stride, row_stride, i_off, f_off, _ptr(bias_i), _ptr(bias_f),
              float(cap or 0.0), _ptr(gates), _ptr(state), state.stride(1), m_off, _ptr(seq_start), _ptr(seq_slot),
              seq_slot.numel(), n_heads, seg_len or 128, _stream()), "gate_scan")
+
+
+def qk_row_norm(proj, q_out, k_cache, v_cache, block_table, ctx, q_gain, k_gain, eps: float, temp, n_heads: int,
+                n_kv_heads: int, head_dim: int, v_head_dim: int, has_kv: bool) -> None:
+    """RMS norm of a token's whole query row (all heads at once) and whole key row, then ``temp`` = (coef, every) on the
+    query: times 1 + coef ln(floor((p + 1) / every) + 1) at position p (None: no temperature).  ``proj`` [T, N] (or
+    float32 partials [S, T, N]) holds q | k | v, or q alone (``has_kv`` false); q goes to ``q_out`` [T, H*D], keys and
+    values into the paged cache entry."""
+    _dev(proj, q_out, k_cache, v_cache, block_table, q_gain, k_gain)
+    _contig("proj", proj), _contig("q_out", q_out)
+    n_split, split_stride, row_stride = _split_view(proj)
+    T, H, G, D, Dv = q_out.shape[0], n_heads, n_kv_heads, head_dim, v_head_dim
+    assert proj.shape[-1] == H * D + (G * (D + Dv) if has_kv else 0) and q_out.shape[1] == H * D and proj.shape[-2] == T
+    assert q_gain.dtype == torch.float32 and q_gain.numel() == H * D and q_gain.is_contiguous()
+    if has_kv:
+        _contig("k_cache", k_cache), _contig("v_cache", v_cache), _contig("block_table", block_table)
+        assert k_gain.dtype == torch.float32 and k_gain.numel() == G * D and k_gain.is_contiguous()
+        assert k_cache.shape[1:] == (G, PAGE, D) and v_cache.shape[1:] == (G, PAGE, Dv) and k_cache.dtype == v_cache.dtype
+    coef, every = temp or (0.0, 0)
+    f = _fn("qk_row_norm", "llmx_qk_row_norm",
+            [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
+             c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+             c_int, c_longlong, c_void_p])
+    _check(f(_ptr(proj), _tag(proj), n_split, split_stride, row_stride, _ptr(q_out), _tag(q_out),
+             _ptr(k_cache) if has_kv else None, _ptr(v_cache) if has_kv else None,
+             _tag(k_cache) if has_kv else _tag(q_out), _ptr(block_table) if has_kv else None,
+             block_table.shape[1] if has_kv else 0, _ptr(ctx.token_seq), _ptr(ctx.token_pos), _ptr(q_gain),
+             _ptr(k_gain) if has_kv else None, eps, float(coef), int(every), T, H, G, D, Dv, int(has_kv), ctx.n_seqs,
+             k_cache.shape[0] if has_kv else 0, _stream()), "qk_row_norm")
+
+
+DELTA_MAX_TAPS = 16        # the same constants as DR_MAX_TAPS, DR_CHUNK and DR_COEF in delta_rule.cu
+DELTA_CHUNK, DELTA_COEF = 8, 156
+
+
+def _delta_args(proj, offsets, conv_w, taps, a_log, dt_bias, q_scale, unit_eps, state, ring_off, H, G, D, Dv):
+    _dev(proj, conv_w, a_log, dt_bias, state)
+    _contig("proj", proj), _contig("state", state), _contig("conv_w", conv_w)
+    C = 2 * G * D + H * Dv
+    assert conv_w.dtype == torch.float32 and conv_w.shape == (taps, C)
+    assert all(v.dtype == torch.float32 and v.numel() == H and v.is_contiguous() for v in (a_log, dt_bias))
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.shape[1] >= ring_off + taps * C
+    n_split, split_stride, row_stride = _split_view(proj)
+    return (_ptr(proj), _tag(proj), n_split, split_stride, row_stride, *offsets, _ptr(conv_w), taps, _ptr(a_log),
+            _ptr(dt_bias), float(q_scale), float(unit_eps), _ptr(state), state.stride(0), ring_off, state.shape[0])
+
+
+_DELTA_ARGTYPES = [c_void_p, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                   c_void_p, c_void_p, c_float, c_float, c_void_p, c_longlong, c_longlong, c_int]
+
+
+def delta_prompt(proj, offsets, conv_w, taps: int, a_log, dt_bias, q_scale: float, unit_eps: float, state, ring_off: int,
+                 out, ctx, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int) -> None:
+    """The gated delta rule over every sequence's tokens of the step (csrc/delta_rule.cu): convolution, SiLU and unit
+    norms, then S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q.  ``proj`` [T, N] (or float32 partials) with
+    the columns of q, k, v, b, a and the output gate at ``offsets`` (six numbers in that order); ``conv_w`` float32
+    [taps, C]; ``state`` float32 [slots, n]: S [H, D, Dv], then from ``ring_off`` the convolution's ring [taps, C].
+    ``out`` float32 [T, H*Dv] is o, without norm and gate."""
+    H, G, D, Dv = n_heads, n_kv_heads, head_dim, v_head_dim
+    args = _delta_args(proj, offsets, conv_w, taps, a_log, dt_bias, q_scale, unit_eps, state, ring_off, H, G, D, Dv)
+    T = out.shape[0]
+    assert out.dtype == torch.float32 and out.shape == (proj.shape[-2], H * Dv) and out.is_contiguous()
+    pad4 = lambda n: (n + 3) // 4 * 4
+    chunks = T // DELTA_CHUNK + ctx.n_seqs
+    new = lambda n, what: guard.scratch((n,), torch.float32, out.device, what)
+    qk = new(chunks * G * 2 * DELTA_CHUNK * pad4(D), "prepared keys and queries of the delta rule")
+    vv = new(chunks * H * DELTA_CHUNK * pad4(Dv), "prepared values of the delta rule")
+    co = new(chunks * H * DELTA_COEF, "coefficients of the delta rule's chunks")
+    f = _fn("delta_rule", "llmx_delta_prompt",
+            _DELTA_ARGTYPES + [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                               c_int, c_int, c_int, c_void_p])
+    _check(f(*args, _ptr(qk), _ptr(vv), _ptr(co), _ptr(out), _ptr(ctx.seq_start), _ptr(ctx.seq_past), _ptr(ctx.seq_slot),
+             T, ctx.n_seqs, H, G, D, Dv, _stream()), "delta_prompt")
+    global launch_count
+    launch_count += 2 if taps > 1 else 1          # beside the preparation: the recurrence, and the convolution's rows
+
+
+def delta_decode(proj, offsets, conv_w, taps: int, a_log, dt_bias, q_scale: float, unit_eps: float, state, ring_off: int,
+                 gain, eps: float, y, ctx, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int) -> None:
+    """The same for a step in which every sequence brings one token, with the norm and gate behind the recurrence:
+    y [B, H*Dv] = o / sqrt(mean(o^2) + eps) * gain * silu(gate) per head, ``gain`` float32 [Dv]."""
+    H, G, D, Dv = n_heads, n_kv_heads, head_dim, v_head_dim
+    args = _delta_args(proj, offsets, conv_w, taps, a_log, dt_bias, q_scale, unit_eps, state, ring_off, H, G, D, Dv)
+    assert y.shape == (proj.shape[-2], H * Dv) and y.is_contiguous() and y.shape[0] == ctx.n_seqs
+    assert gain.dtype == torch.float32 and gain.numel() == Dv and gain.is_contiguous()
+    f = _fn("delta_rule", "llmx_delta_decode",
+            _DELTA_ARGTYPES + [c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                               c_void_p])
+    _check(f(*args, _ptr(gain), eps, _ptr(y), _tag(y), _ptr(ctx.seq_past), _ptr(ctx.seq_slot), ctx.n_seqs, H, G, D, Dv,
+             _stream()), "delta_decode")
 
 
 def gated_norm(o, proj, g_off: int, gain, eps: float, gate: str, per_head: bool, y, n_heads: int,

@@ -38,6 +38,10 @@ The cache entry then owns a second store of one row per block (``KVNeed.pool``),
 block's last position; positions that have left the window and whose block is not complete are not seen.  A position
 encoding that pairs neighbouring dimensions is met by reordering the rows of the q and k projections once
 (``parts.position.halves_order``).
+``qk_norm`` "rows": the RMS norm of q and k is taken over the whole projected row, before it is split into heads
+(gains ``q_norm`` [H*D] and ``k_norm`` [G*D]; built without a rotation); beside it ``q_temp`` = (coef, every)
+multiplies the query at position p by 1 + coef ln(floor((p + 1) / every) + 1).  ``softcap`` c: a scaled score s becomes
+c tanh(s / c) before the softmax.
 Tensors ``q_bias``, ``k_bias``, ``v_bias``, ``o_bias``: biases of the four
 projections (q, k, v: added where the projected row is read, before norm and
 rotation; o: offered as ``out_bias`` to an arrangement that adds it in its
@@ -115,9 +119,21 @@ class GQAttention:
             bk = halves_order(position, bk.unsqueeze(1), self.G, self.D).squeeze(1)
             self.qkv_bias = torch.cat([bq, bk, bv]).contiguous()
         self.q_gain = self.k_gain = None
+        self.qk_norm = spec.get("qk_norm", "heads")          # what q and k are normed over: each head, or whole rows
         if "q_norm" in t:
             self.q_gain = weights.pop(t["q_norm"].name).to(torch.float32).contiguous()
-            self.k_gain = weights.pop(t["k_norm"].name).to(torch.float32).contiguous()
+            if self.own_kv or self.qk_norm == "heads":
+                self.k_gain = weights.pop(t["k_norm"].name).to(torch.float32).contiguous()
+        self.q_temp = spec.get("q_temp")
+        self.softcap = float(spec.get("softcap") or 0.0)
+        self.row_norm = self.qk_norm == "rows"
+        if self.row_norm and (self.q_gain is None or self.qkv_bias is not None or spec.get("conv_taps") or spec.get("v_mix")
+                              or (position is not None and position.rotary_tables() is not None)):
+            raise Unsupported("a norm over whole q/k rows is built without rotation, biases, convolution and mixed values")
+        if self.q_temp and not self.row_norm:
+            raise Unsupported("a query temperature is built beside a norm over whole q/k rows")
+        if self.softcap and self.pool:
+            raise Unsupported("capped scores beside pooled blocks are not built")
         self.position = position
         if getattr(position, "pairing", "halves") == "neighbours" and ("q_norm" in t or spec.get("conv_taps")):
             raise Unsupported("a rotation of neighbouring pairs beside a q/k norm or a short convolution is not built")
@@ -157,12 +173,15 @@ class GQAttention:
             libs.add("short_conv")
         if self.pool:
             libs.add("attention")           # the blocks' means are made there
+        if self.row_norm:
+            libs.add("qk_row_norm")
         if not self.plain:
             return libs | {"attention"}
         if self.rt.dtype == "bfloat16" and self.rt.tensor_cores:
             tc = self.D == 128 and not self.pool      # (pooled blocks: the mma.sync kernel, at both head sizes)
-            libs |= {"attention_decode",
-                     "attention_prefill_tc" if tc else "attention_prefill" if self.D in (64, 128) else "attention"}
+            cap = lambda name: kernels.capped_library(name, self.softcap)
+            libs |= {cap("attention_decode"),
+                     cap("attention_prefill_tc") if tc else cap("attention_prefill") if self.D in (64, 128) else "attention"}
         else:
             libs.add("attention")
         return libs
@@ -195,6 +214,11 @@ class GQAttention:
                                     n_rot, v_first, self.v_lambda, mode, H, G, D, Dv, inline_state=inline)
             if not inline:
                 kernels.conv_state_update(qkv, view.state, self.taps, ctx)
+        elif self.row_norm:
+            proj = self.qkv(x, splits_ok=True) if writes_cache else self.q_only(x, splits_ok=True)
+            q = torch.empty((T, H * D), dtype=self.rt.act_dtype, device=dev)
+            kernels.qk_row_norm(proj, q, view.k, view.v, block_table, ctx, self.q_gain, self.k_gain, self.eps, self.q_temp,
+                                H, G, D, Dv, writes_cache)
         elif not writes_cache and self.q_gain is None and n_rot == 0 and self.qkv_bias is None:
             # A call that reads another call's cache entry makes only queries; nothing is done to them.
             q = self.q_only(x, out_dtype=self.rt.act_dtype)
@@ -229,20 +253,22 @@ class GQAttention:
         H, G, D = self.H, self.G, self.D
         fast = (self.plain and q.dtype == torch.bfloat16 and view.k.dtype == torch.bfloat16
                 and self.rt.tensor_cores and self.scale > 0)       # (the tiled kernels take the maximum before the scale)
-        pooled = dict(pool=self.pool, pool_k=view.pool_k, pool_v=view.pool_v,
+        extra = dict(pool=self.pool, pool_k=view.pool_k, pool_v=view.pool_v,
                       pool_table=ctx.block_tables[view.pool_group]) if self.pool else {}
+        if self.softcap:
+            extra["softcap"] = self.softcap
         if fast and ctx.is_decode:
             kernels.attention_decode(q, out, view.k, view.v, block_table, ctx.seq_past, H, G, D, self.window,
-                                     self.scale, keep_first=self.keep_first, sink=self.sink, chunk=self.chunk, **pooled)
+                                     self.scale, keep_first=self.keep_first, sink=self.sink, chunk=self.chunk, **extra)
         elif fast and D == 128 and not self.pool:
             kernels.attention_prefill_tc(q, out, view.k, view.v, block_table, ctx.seq_start, ctx.seq_past,
                                          ctx.n_seqs, ctx.max_new, H, G, D, self.window, self.scale,
-                                         keep_first=self.keep_first, sink=self.sink, chunk=self.chunk)
+                                         keep_first=self.keep_first, sink=self.sink, chunk=self.chunk, **extra)
         elif fast and kernels.attention_prefill_supports(q, view.k, D):
             kernels.attention_prefill(q, out, view.k, view.v, block_table, ctx.seq_start, ctx.seq_past,
                                       ctx.n_seqs, ctx.max_new, H, G, D, self.window, self.scale,
-                                      keep_first=self.keep_first, sink=self.sink, chunk=self.chunk, **pooled)
+                                      keep_first=self.keep_first, sink=self.sink, chunk=self.chunk, **extra)
         else:
             kernels.attention_paged(q, out, view.k, view.v, block_table, ctx.token_seq, ctx.token_pos,
                                     H, G, D, self.window, self.scale, v_head_dim=self.Dv, keep_first=self.keep_first,
-                                    sink=self.sink, chunk=self.chunk, **pooled)
+                                    sink=self.sink, chunk=self.chunk, **extra)

@@ -17,6 +17,7 @@ reads u + conv(u) instead of the normed stream u, conv a causal convolution over
 ``result_gate`` "sigmoid", every sublayer's result is multiplied by sigmoid(W u + b) before the norm behind it (tensors
 ``mixer_gate`` / ``mixer_gate_bias``, ``feed_forward_gate`` / ``feed_forward_gate_bias``; u is the normed stream, before
 the convolution); the product W u is one more matrix product, sigmoid and multiplication happen in the norm kernel.
+``post_norm`` norms a sublayer's result only: h += norm(mixer(h)), then h += norm(feed_forward(h)).
 A part whose last product has a bias offers it as ``out_bias``; an arrangement that can add it in its own norm
 kernel sets the part's ``defer_out_bias``, and the part then leaves the bias to it."""
 
@@ -28,6 +29,7 @@ from .. import kernels
 from ..cache import StateNeed
 from ..errors import Unsupported
 from .linear import Linear
+from .norm import stream_rows
 from .registry import (ARRANGEMENTS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, lookup, register_arrangement)
 
 
@@ -313,3 +315,53 @@ class SandwichBlock:
             if out is not None:
                 probe("ffn_out", _summed(out))
         return self.ff_post.owed(out, bias=getattr(self.feed_forward, "out_bias", None), gate=gate)
+
+
+@register_arrangement("post_norm")
+class PostNormBlock:
+    """A norm behind each sublayer and none before it: h += post(mixer(h)), then h += post(feed_forward(h)) (norms
+    ``mixer_post``, ``feed_forward_post``; a layer without a feed-forward has the first).  The sublayers read the
+    stream itself, rounded to the compute dtype; a result is owed to whoever reads the stream next, whose kernel norms
+    it, adds it to the float32 stream and hands out the rows (or norms them, at the model's end)."""
+
+    def __init__(self, spec, weights: dict, rt):
+        position = None
+        if spec.position is not None:
+            position = rt_shared_position(spec.position, weights, rt)
+        self.act_dtype = rt.act_dtype
+        self.mixer_post = build_part(NORMS, "norm", spec.norms["mixer_post"], weights, rt)
+        self.mixer = lookup(MIXERS, "mixer", spec.mixer.kind)(spec.mixer, position, weights, rt)
+        self.feed_forward = build_part(FEED_FORWARDS, "feed-forward", spec.feed_forward, weights, rt)
+        self.ff_post = None
+        if "feed_forward_post" in spec.norms:
+            self.ff_post = build_part(NORMS, "norm", spec.norms["feed_forward_post"], weights, rt)
+        for part in (self.mixer, self.feed_forward):
+            if getattr(part, "out_bias", None) is not None:
+                part.defer_out_bias = True           # added by the norm kernel behind the part
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def libraries(self) -> set:
+        libs = {"post_norm"}
+        for part in (self.mixer_post, self.ff_post, self.mixer, self.feed_forward):
+            if part is not None:
+                libs |= getattr(part, "libraries", set)()
+        return libs
+
+    def forward(self, h, pending, ctx, view, writes_cache=True):
+        probe = getattr(ctx, "probe", None)
+        x = stream_rows(h, pending, self.act_dtype)
+        if probe:
+            probe("resid_in", h)
+        a = self.mixer.forward(x, ctx, view, writes_cache)
+        if probe:
+            probe("attn_output", _summed(a))
+        pending = self.mixer_post.owed(a, bias=getattr(self.mixer, "out_bias", None))
+        if self.ff_post is None:
+            return pending
+        x = stream_rows(h, pending, self.act_dtype)
+        out = self.feed_forward.forward(x, ctx)
+        if probe:
+            probe("attn_residual", h), probe("ffn_out", _summed(out))
+        return self.ff_post.owed(out, bias=getattr(self.feed_forward, "out_bias", None))

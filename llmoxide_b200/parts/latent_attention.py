@@ -12,6 +12,11 @@ R rotated query/key dimensions and values of size Dv:
     s   = (q_plain . k_plain + rot(q_rot) . rot(kr)) * scale, softmax over the window's keys
     out = W_o concat_h( sigmoid(W_g x)_h * sum_j w_j v_j )      (``out_gate`` "sigmoid"; None: no gate)
 
+``q_rank`` 0: queries come straight from the input, q = W_q x (tensor ``q`` in
+place of ``dq``, ``dq_norm``, ``uq``).  Tensor ``sink`` [H]: exp(sink_h) joins
+head h's softmax denominator, a learned score without key and value that is
+not scaled.
+
 rms is x / sqrt(mean(x^2) + eps) in float32.  The rotation is the position
 part's (any table of ``rot_dim`` dimensions: scaled frequencies, an amplitude).
 
@@ -63,16 +68,16 @@ class LatentAttention:
             raise Unsupported(f"head sizes {self.E}/{self.Dv}: the attention kernels take sizes up to 256")
         H, D, R, Dv = self.H, self.D, self.R, self.Dv
         t = spec.tensors
-        wdq, wdkv = weights.pop(t["dq"].name), weights.pop(t["dkv"].name)
+        wdkv = weights.pop(t["dkv"].name)
         # the shared rotated part's rows in the order the kernels pair them
         wdkv = torch.cat([wdkv[: self.Rkv], halves_order(position, wdkv[self.Rkv :], 1, R)], dim=0)
-        rows = [wdq, wdkv] + ([weights.pop(t["g"].name)] if self.gate else [])
+        rows = ([weights.pop(t["dq"].name)] if self.Rq else []) + [wdkv] + ([weights.pop(t["g"].name)] if self.gate else [])
         if len({w.dtype for w in rows}) > 1:
             rows = [w.float() for w in rows]
         self.down = Linear(torch.cat(rows, dim=0).contiguous(), rt)
         self.k_rot_off, self.gate_off = self.Rq + self.Rkv, self.Rq + self.Rkv + R
         # queries: every head's rows become [rotated (paired as the kernels pair) | unrotated]
-        wuq = weights.pop(t["uq"].name)
+        wuq = weights.pop(t["uq" if self.Rq else "q"].name)
         wuq = halves_order(position, wuq, H, D + R, first=D)
         index = torch.tensor([h * (D + R) + i for h in range(H) for i in list(range(D, D + R)) + list(range(D))],
                              device=wuq.device)
@@ -81,7 +86,8 @@ class LatentAttention:
         if wuk.dtype != wuv.dtype:
             wuk, wuv = wuk.float(), wuv.float()
         self.ukv = Linear(torch.cat([wuk, wuv], dim=0).contiguous(), rt)
-        self.q_gain = weights.pop(t["dq_norm"].name).to(torch.float32).contiguous()
+        self.q_gain = weights.pop(t["dq_norm"].name).to(torch.float32).contiguous() if self.Rq else None
+        self.sinks = weights.pop(t["sink"].name).to(torch.float32).contiguous() if "sink" in t else None
         self.kv_gain = weights.pop(t["dkv_norm"].name).to(torch.float32).contiguous()
         self.o = Linear(weights.pop(t["o"].name), rt)
         self.out_bias, self.defer_out_bias = None, False
@@ -106,10 +112,10 @@ class LatentAttention:
         H, D, R, Dv, E = self.H, self.D, self.R, self.Dv, self.E
         T, dev, act = x.shape[0], x.device, self.rt.act_dtype
         down = self.down(x, out_dtype=torch.float32)                         # [T, Rq + Rkv + R (+ H)]
-        cq = torch.empty((T, self.Rq), dtype=act, device=dev)
+        cq = torch.empty((T, self.Rq), dtype=act, device=dev) if self.Rq else None
         c = torch.empty((T, self.Rkv), dtype=act, device=dev)
         kernels.latent_norms(down, self.q_gain, self.kv_gain, self.eps, cq, c, self.Rq, self.Rkv)
-        q_up = self.uq(cq)
+        q_up = self.uq(cq if self.Rq else x)
         kv_up = self.ukv(c)
         cos, sin, _ = self.position.rotary_tables()
         block_table = ctx.block_tables[view.group]
@@ -128,16 +134,17 @@ class LatentAttention:
         fast = (self.plain and q.dtype == torch.bfloat16 and view.k.dtype == torch.bfloat16
                 and self.rt.tensor_cores and self.scale > 0)
         if fast and ctx.is_decode:
-            kernels.attention_decode(q, out, view.k, view.v, block_table, ctx.seq_past, H, H, E, self.window, self.scale)
+            kernels.attention_decode(q, out, view.k, view.v, block_table, ctx.seq_past, H, H, E, self.window, self.scale,
+                                     sinks=self.sinks)
         elif fast and E == 128:
             kernels.attention_prefill_tc(q, out, view.k, view.v, block_table, ctx.seq_start, ctx.seq_past,
-                                         ctx.n_seqs, ctx.max_new, H, H, E, self.window, self.scale)
+                                         ctx.n_seqs, ctx.max_new, H, H, E, self.window, self.scale, sinks=self.sinks)
         elif fast and kernels.attention_prefill_supports(q, view.k, E):
             kernels.attention_prefill(q, out, view.k, view.v, block_table, ctx.seq_start, ctx.seq_past,
-                                      ctx.n_seqs, ctx.max_new, H, H, E, self.window, self.scale)
+                                      ctx.n_seqs, ctx.max_new, H, H, E, self.window, self.scale, sinks=self.sinks)
         else:
             kernels.attention_paged(q, out, view.k, view.v, block_table, ctx.token_seq, ctx.token_pos,
-                                    H, H, E, self.window, self.scale, v_head_dim=self.Dv, gate=gate)
+                                    H, H, E, self.window, self.scale, v_head_dim=self.Dv, gate=gate, sinks=self.sinks)
             return
         if gate is not None:
             kernels.head_gate(out, gate, H, self.Dv)

@@ -16,7 +16,13 @@ the next norm's kernel: ``owed(y)`` wraps a sublayer's result into the
 BEHIND a sublayer ("sandwich" blocks, h += norm_b(f(norm_a(h)))): ``owed(y)``
 then wraps the sublayer's result into a ``PostNormed``, and the next norm's
 kernel norms it, adds it to the stream and norms the stream in one pass.  Two
-mixers side by side hand over a ``WeightedSum`` of their results."""
+mixers side by side hand over a ``WeightedSum`` of their results.  In a block
+whose sublayers read the stream itself (``post_norm``) there is no norm on the
+other side: ``stream_rows`` adds what is owed and returns the stream's rows in
+the compute dtype, by the same kernel.
+
+``gain_offset`` (parameter of ``rms_norm``): the gain is the stored weight plus
+this number, for weights stored as their distance from one."""
 
 from __future__ import annotations
 
@@ -79,6 +85,15 @@ def _general_add_norm(h, delta, gain, center: bool, eps: float, out, rows, write
                                write_h=write_h, gate=gate)
 
 
+def stream_rows(h, delta, act_dtype):
+    """h += ``delta`` (None, or what a sublayer owes the stream); the stream's rows in ``act_dtype``, not normed.  In
+    float32 those are the stream itself: whoever reads them does so before anything is added again."""
+    out = None if act_dtype == torch.float32 else torch.empty(h.shape, dtype=act_dtype, device=h.device)
+    if out is not None or delta is not None:
+        _general_add_norm(h, delta, None, False, 0.0, out, None, True)
+    return h if out is None else out
+
+
 @register_norm("layer_norm")
 class LayerNorm:
     """(x - mean) / sqrt(variance + eps) * gain, the variance the mean of the squared deviations; no bias."""
@@ -113,6 +128,8 @@ class RMSNorm:
     def __init__(self, spec, weights: dict, rt):
         self.size, self.eps, self.rt = spec["size"], float(spec["eps"]), rt
         self.gain = weights[spec.tensors["gain"].name].to(torch.float32).contiguous()
+        if spec.get("gain_offset"):
+            self.gain = self.gain + float(spec["gain_offset"])
         self.mult = float(spec.get("residual_mult", 1.0))
         self.read = self.mix = self.write = None
         if "hc_mix" in spec.tensors:
