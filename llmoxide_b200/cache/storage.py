@@ -27,7 +27,8 @@ class KVNeed:
     """Keys and values for every position (window None) or for the last
     ``window`` positions, beside which the first ``keep_first`` positions of a
     sequence stay visible for good.  Values may be narrower or wider than keys
-    (``v_head_dim``, default ``head_dim``), and an entry may keep its keys and
+    (``v_head_dim``, default ``head_dim``; 0: no store of values, for a mixer that makes them from its cached rows),
+    and an entry may keep its keys and
     values in a dtype of its own (default: the runtime's cache dtype).  With ``pool`` n > 1 the entry owns a second
     store beside the first, one key and one value per block of n positions (block b = positions b*n .. b*n+n-1, its
     row exists once the sequence holds all of them); that store keeps every row, whatever the window.  ``every`` is
@@ -103,7 +104,7 @@ class Cache:
         self.k_store, self.v_store = [], []
         for kv in self.groups:
             k_shape = (len(members[kv]), pages_of(kv), kv.n_kv_heads, PAGE, kv.head_dim)
-            v_shape = k_shape[:-1] + (kv.v_head_dim or kv.head_dim,)
+            v_shape = k_shape[:-1] + (kv.head_dim if kv.v_head_dim is None else kv.v_head_dim,)
             # (every long-lived buffer carries guard words behind it: guard.py)
             g = len(self.k_store)
             self.k_store.append(guarded(k_shape, kv.dtype or dtype, device, f"cache group {g} keys", zero=True))

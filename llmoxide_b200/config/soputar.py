@@ -204,7 +204,7 @@ class SoputarConfig:
                            sink=vector("sink", H, SINK_INIT), o=matrix("o", d, H * Dv))
             mixer = PartSpec("latent_attention", dict(
                 hidden_size=d, n_heads=H, head_dim=D, rot_dim=R, v_head_dim=Dv, q_rank=0, kv_rank=rank, eps=eps,
-                scale=float(m["scale"]), window=None, out_gate=None), tensors)
+                scale=float(m["scale"]), window=None, out_gate=None, cache="latent"), tensors)
             return mixer, PartSpec("rope_neox", dict(n_rot=R, base=float(m["rot"]["base"]), angles="float32",
                                                      pairing="neighbours"))
         G, D, taps = m["kv_heads"], m["dim"], m["conv"]

@@ -48,6 +48,7 @@ LIBRARIES = {
     "gemm_tc": (["gemm_tc.cu"], []),
     "linear_attention": (["linear_attention.cu"], []),
     "latent_attention": (["latent_attention.cu"], []),
+    "latent_cache": (["latent_cache.cu"], []),
     "moe": (["moe.cu"], []),
     "post_norm": (["post_norm.cu"], []),
     "qk_row_norm": (["qk_row_norm.cu"], []),

@@ -239,32 +239,35 @@ Layout make_layout(long long T, long long B, long long W, const std::vector<long
   return l;
 }
 
-void write_meta(const Layout& l, long long max_new, long long max_len, bool is_decode, long long* meta) {
+constexpr int META = 9;        // numbers of a step's facts ahead of the offsets and widths
+
+void write_meta(const Layout& l, long long max_new, long long max_len, bool is_decode, long long ctx_pages, long long* meta) {
   const long long ng = (long long)l.width.size();
   meta[0] = l.n_tokens, meta[1] = l.n_seqs, meta[2] = l.n_want, meta[3] = l.total;
-  meta[4] = max_new, meta[5] = max_len, meta[6] = is_decode ? 1 : 0, meta[7] = ng;
-  for (size_t i = 0; i < l.off.size(); ++i) meta[8 + i] = l.off[i];
-  for (long long g = 0; g < ng; ++g) meta[8 + 7 + ng + g] = l.width[g];
+  meta[4] = max_new, meta[5] = max_len, meta[6] = is_decode ? 1 : 0, meta[7] = ng, meta[8] = ctx_pages;
+  for (size_t i = 0; i < l.off.size(); ++i) meta[META + i] = l.off[i];
+  for (long long g = 0; g < ng; ++g) meta[META + 7 + ng + g] = l.width[g];
 }
 
 // Packs a step.  page_row(g, i, &len) gives sequence i's page list in group g.
 template <typename RowFn>
 int pack(long long B, const int* slots, const int* counts, const int* tokens, const int* want_counts, const int* wants,
          const long long* lengths, int n_groups, RowFn page_row, int* buf, long long cap, long long* meta) {
-  long long T = 0, W = 0, max_new = 0, max_len = 0;
+  long long T = 0, W = 0, max_new = 0, max_len = 0, ctx_pages = 0;
   bool is_decode = true;
   for (long long i = 0; i < B; ++i) {
     T += counts[i];
     W += want_counts[i] < 0 ? 1 : want_counts[i];
     max_new = std::max<long long>(max_new, counts[i]);
     max_len = std::max(max_len, lengths[i] + counts[i]);
+    ctx_pages += pages_for(lengths[i] + counts[i]);
     if (counts[i] != 1) is_decode = false;
   }
   // one width for every group: the longest sequence after this step, rounded up so that a growing sequence
   // changes the layout rarely
   const long long width = align4(std::max(1LL, pages_for(max_len)));
   Layout l = make_layout(T, B, W, std::vector<long long>((size_t)n_groups, width));
-  write_meta(l, max_new, max_len, is_decode, meta);
+  write_meta(l, max_new, max_len, is_decode, ctx_pages, meta);
   if (l.total > cap) return fail(TOO_SMALL, "the step buffer holds %lld elements, the step needs %lld", cap, l.total);
   std::memset(buf, 0, (size_t)l.total * sizeof(int));
   int *tok = buf + l.off[0], *tseq = buf + l.off[1], *tpos = buf + l.off[2], *start = buf + l.off[3];

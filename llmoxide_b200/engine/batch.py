@@ -62,6 +62,7 @@ class StepContext:
     max_new: int             # most new tokens of one sequence
     max_len: int             # longest sequence after this step
     is_decode: bool          # every sequence brings exactly one token
+    ctx_pages: int           # pages of all sequences together after this step, each rounded up to whole pages
     tokens: torch.Tensor
     token_seq: torch.Tensor
     token_pos: torch.Tensor
@@ -76,15 +77,16 @@ class StepContext:
     carry: dict = field(default_factory=dict)
 
 
+N_META = 9         # numbers of a step's facts ahead of the offsets and widths (csrc/host_runtime.cpp, write_meta)
 N_FIXED = 7        # arrays before the block tables: tokens, token_seq, token_pos, seq_start, seq_past, seq_slot, want_rows
 _NAMES = ("tokens", "token_seq", "token_pos", "seq_start", "seq_past", "seq_slot", "want_rows")
 
 
 def layout_from_meta(meta) -> tuple:
     """(layout, facts) from the numbers the C++ packer returns (csrc/host_runtime.cpp, write_meta)."""
-    n_tokens, n_seqs, n_want, total, max_new, max_len, is_decode, n_groups = (int(x) for x in meta[:8])
-    offs = [int(x) for x in meta[8 : 8 + N_FIXED + n_groups]]
-    widths = tuple(int(x) for x in meta[8 + N_FIXED + n_groups : 8 + N_FIXED + 2 * n_groups])
+    n_tokens, n_seqs, n_want, total, max_new, max_len, is_decode, n_groups, ctx_pages = (int(x) for x in meta[:N_META])
+    offs = [int(x) for x in meta[N_META : N_META + N_FIXED + n_groups]]
+    widths = tuple(int(x) for x in meta[N_META + N_FIXED + n_groups : N_META + N_FIXED + 2 * n_groups])
     lay = StepLayout(n_tokens, n_seqs, n_want, widths)
     sizes = (n_tokens, n_tokens, n_tokens, n_seqs + 1, n_seqs, n_seqs, n_want)
     for name, at, n in zip(_NAMES, offs, sizes):
@@ -92,7 +94,7 @@ def layout_from_meta(meta) -> tuple:
     for g, w in enumerate(widths):
         lay.offsets[f"block_table{g}"] = (offs[N_FIXED + g], n_seqs * w)
     lay.total = total
-    return lay, dict(max_new=max_new, max_len=max_len, is_decode=bool(is_decode))
+    return lay, dict(max_new=max_new, max_len=max_len, is_decode=bool(is_decode), ctx_pages=ctx_pages)
 
 
 def flatten_entries(entries, wants):
@@ -138,7 +140,7 @@ def build_host_arrays(entries, wants, lengths, page_rows, n_groups):
     rows = np.asarray(rows if rows else [0], dtype=np.int32)
     row_off = np.asarray(row_off, dtype=np.int64)
     row_len = np.asarray(row_len, dtype=np.int32)
-    meta = np.zeros(8 + N_FIXED + 2 * n_groups, dtype=np.int64)
+    meta = np.zeros(N_META + N_FIXED + 2 * n_groups, dtype=np.int64)
     cap = 4 * int(counts.sum()) + 8 * n + len(want_flat) + n * n_groups * (int(lens.max() + counts.max()) // PAGE + 8) + 64
     buf = np.zeros(cap, dtype=np.int32)
     ptr = lambda a: a.ctypes.data
@@ -206,6 +208,6 @@ class StepBuffers:
         tables = [view(f"block_table{g}").view(lay.n_seqs, w) for g, w in enumerate(lay.widths)]
         return StepContext(
             n_tokens=lay.n_tokens, n_seqs=lay.n_seqs, max_new=facts["max_new"], max_len=facts["max_len"],
-            is_decode=facts["is_decode"], tokens=view("tokens"), token_seq=view("token_seq"),
+            is_decode=facts["is_decode"], ctx_pages=facts["ctx_pages"], tokens=view("tokens"), token_seq=view("token_seq"),
             token_pos=view("token_pos"), seq_start=view("seq_start"), seq_past=view("seq_past"),
             seq_slot=view("seq_slot"), want_rows=view("want_rows"), block_tables=tables, widths=lay.widths)

@@ -26,7 +26,7 @@ from ..errors import CacheExhausted, CacheMisuse, ContextOverflow
 from ..parts import Runtime
 from ..weights import load_checkpoint, random_tensors_on_device
 from ..cache.allocator import _TOO_SMALL, host_library, raise_host_error
-from .batch import N_FIXED, StepBuffers, flatten_entries, layout_from_meta
+from .batch import N_FIXED, N_META, StepBuffers, flatten_entries, layout_from_meta
 from .model import DecoderModel
 
 
@@ -192,7 +192,7 @@ class Engine:
 
     def _prompt_key(self, lay, ctx):
         # what the launches of a prompt step depend on besides the step buffer's contents
-        return (lay.key(), ctx.max_new, ctx.max_len, self.buffers.dev.data_ptr())
+        return (lay.key(), ctx.max_new, ctx.max_len, ctx.ctx_pages, self.buffers.dev.data_ptr())
 
     def _prompt_shape_came_back(self, lay, ctx) -> bool:
         """Whether this prompt step is short enough to be bound by its launches and has a shape that ran
@@ -249,7 +249,7 @@ class Engine:
         alloc = self.cache.alloc
         n_groups = max(1, self.cache.n_groups())
         slots, counts, tokens, want_counts, want_flat = flatten_entries(entries, want)
-        meta = np.zeros(8 + N_FIXED + 2 * n_groups, dtype=np.int64)
+        meta = np.zeros(N_META + N_FIXED + 2 * n_groups, dtype=np.int64)
         ptr = lambda a: a.ctypes.data
         for attempt in range(2):
             host = self.buffers.next_host()

@@ -123,7 +123,8 @@ def _library(lib_name: str):
 
 _STATUS_SLOTS = {"gemm_tc": 0, "attention_prefill_tc": 1, "attention_decode": 2, "sampling": 3, "moe_tc": 4,
                  "short_conv": 5, "stream_mix": 6, "moe": 7, "attention": 8, "latent_attention": 9,
-                 "attention_prefill_tc_capped": 10, "attention_decode_capped": 11, "qk_row_norm": 12, "delta_rule": 13}
+                 "attention_prefill_tc_capped": 10, "attention_decode_capped": 11, "qk_row_norm": 12, "delta_rule": 13,
+                 "latent_cache": 14}
 _STATUS_MEANING = {
     "gemm_tc": {1: "the producer's wait for a free stage ran out", 2: "the MMA issuer's wait for a stage's data ran out",
                 3: "the epilogue's wait for an accumulator ran out", 4: "the MMA issuer's wait for a drained accumulator ran out",
@@ -144,6 +145,9 @@ _STATUS_MEANING = {
     "attention": {1: "a block's row has no page in the store of one row per block",
                   2: "a block's positions are no longer held by the cache"},
     "latent_attention": {1: "a token's sequence, position or page lies outside the launch's arrays"},
+    "latent_cache": {1: "a token's sequence, position or page lies outside the launch's arrays",
+                     2: "a token's sequence, position or page lies outside the launch's arrays (absorbed attention)",
+                     3: "a scratch page stands for no page of the step's sequences"},
     "qk_row_norm": {1: "a token's sequence, position or page lies outside the launch's arrays"},
     "delta_rule": {1: "a sequence's rows or slot lie outside the launch's arrays (preparation)",
                    2: "a sequence's slot lies outside the state area",
@@ -667,6 +671,141 @@ def latent_rope_cache(q, kv, down, k_rot_off: int, q_out, k_cache, v_cache, bloc
              _ptr(q_out), _tag(q_out), _ptr(k_cache), _ptr(v_cache), _tag(k_cache), _ptr(block_table),
              block_table.shape[1], _ptr(ctx.token_seq), _ptr(ctx.token_pos), _ptr(cos), _ptr(sin), T, H, D, R, Dv,
              ctx.n_seqs, k_cache.shape[0], _stream()), "latent_rope_cache")
+
+
+# ---- attention over a cache of latents (csrc/latent_cache.cu) ----------------------------------------------------------
+
+def latent_prep(down, q, gain, eps: float, cache, rot_out, plain_out, block_table, ctx, cos, sin, n_heads: int,
+                head_dim: int, rot_dim: int, rank: int) -> None:
+    """Per token: the latent's RMS norm and the shared key part's rotation into the cache row [c | rotated], and the
+    query, every head [R rotated | D plain] in ``q``, rotated into ``rot_out`` and copied to ``plain_out`` (views
+    [T, H, R] and [T, H, D] with any stride between heads).  ``down`` float32 [T, >= rank + R] or partials [S, T, ..]: the
+    latent, then the shared key part; ``q`` likewise, or bfloat16, rows of at least H * (R + D)."""
+    _dev(down, q, gain, cache, rot_out, plain_out, block_table, cos, sin)
+    _contig("block_table", block_table), _contig("cache", cache)
+    H, D, R = n_heads, head_dim, rot_dim
+    T = rot_out.shape[0]
+    assert rot_out.shape == (T, H, R) and plain_out.shape == (T, H, D) and rot_out.dtype == plain_out.dtype
+    assert rot_out.stride(2) == plain_out.stride(2) == 1
+    assert rot_out.stride(0) == H * rot_out.stride(1) and plain_out.stride(0) == H * plain_out.stride(1)
+    assert cache.shape[1:] == (1, PAGE, rank + R) and gain.dtype == torch.float32 and gain.numel() == rank
+    assert cos.shape[1] == R // 2 and cos.dtype == sin.dtype == torch.float32
+    n_split, split_stride, row_stride = _split_view(down)
+    q_split, q_split_stride, q_row_stride = _split_view(q)
+    f = _fn("latent_cache", "llmx_latent_prep",
+            [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p,
+             c_float, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p,
+             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_void_p])
+    _check(f(_ptr(down), _tag(down), n_split, split_stride, row_stride, _ptr(q), _tag(q), q_split, q_split_stride,
+             q_row_stride, _ptr(gain), eps, _ptr(cache), _tag(cache), _ptr(rot_out), rot_out.stride(1), _ptr(plain_out),
+             plain_out.stride(1), _tag(rot_out), _ptr(block_table), block_table.shape[1], _ptr(ctx.token_seq),
+             _ptr(ctx.token_pos), _ptr(cos), _ptr(sin), T, H, D, R, rank, ctx.n_seqs, cache.shape[0], _stream()),
+           "latent_prep")
+
+
+def head_product(x, w, y) -> None:
+    """y[t, h] = w[h] x[t, h] for every head: x [T, H, K], w [H, N, K], y [T, H, N]; x and y may be views whose heads lie
+    any stride apart (tokens H of those).  bfloat16 throughout runs on the tensor cores where K is a multiple of 8."""
+    _dev(x, w, y)
+    _contig("w", w)
+    (T, H, K), N = x.shape, w.shape[1]
+    assert w.shape == (H, N, K) and y.shape == (T, H, N) and x.stride(2) == y.stride(2) == 1
+    assert x.stride(0) == H * x.stride(1) and y.stride(0) == H * y.stride(1)
+    f = _fn("latent_cache", "llmx_head_product",
+            [c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), _tag(x), x.stride(1), _ptr(w), _tag(w), _ptr(y), _tag(y), y.stride(1), T, H, N, K, _stream()),
+           "head_product")
+
+
+def latent_paged(q, lat, cache, block_table, ctx, sinks, scale: float, rank: int) -> None:
+    """Absorbed attention in float32, any size: q float32 [T, H, rank + R] = [W_uk^T q | rotated], lat float32
+    [T, H, rank] = sum_j w_j c_j over the cached rows 0 .. position of every token."""
+    _dev(q, lat, cache, block_table, sinks)
+    for name, t in (("q", q), ("lat", lat), ("cache", cache), ("block_table", block_table)):
+        _contig(name, t)
+    T, H, E = q.shape
+    assert q.dtype == lat.dtype == torch.float32 and lat.shape == (T, H, rank) and cache.shape[1:] == (1, PAGE, E)
+    _check_sinks(sinks, H)
+    f = _fn("latent_cache", "llmx_latent_paged",
+            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int,
+             c_int, c_void_p])
+    _check(f(_ptr(q), _ptr(lat), _ptr(cache), _tag(cache), _ptr(block_table), block_table.shape[1], _ptr(ctx.token_seq),
+             _ptr(ctx.token_pos), _ptr(sinks), scale, T, H, rank, E - rank, _stream()), "latent_paged")
+
+
+LATENT_MAX_RANK = 512      # the same constant as LC_MAX_RANK in latent_cache.cu
+
+
+def latent_decode_supports(rank: int, rot_dim: int) -> bool:
+    return rank % 16 == 0 and rot_dim % 16 == 0 and rank <= LATENT_MAX_RANK and rot_dim <= 128
+
+
+def latent_decode_chunks(n_tokens: int, n_heads: int, n_pages: int, sms: int = 148) -> int:
+    """Into how many shares ``latent_decode`` cuts a token's cached rows: about two CTAs an SM over the whole grid, no
+    share shorter than a page of a full block table.  From the batch's shape alone."""
+    base = n_tokens * ((n_heads + 15) // 16)
+    return max(1, min(2 * sms // base, n_pages, 64))
+
+
+def latent_decode(q, lat, cache, block_table, ctx, sinks, scale: float, rank: int, n_chunks: int = 0) -> None:
+    """The same on the tensor cores, bfloat16: q, lat, cache as for ``latent_paged``; every token of the step on its
+    own, its rows cut into ``n_chunks`` shares (0: chosen from the batch's shape)."""
+    _dev(q, lat, cache, block_table, sinks)
+    for name, t in (("q", q), ("lat", lat), ("cache", cache), ("block_table", block_table)):
+        _contig(name, t)
+    T, H, E = q.shape
+    assert q.dtype == lat.dtype == cache.dtype == torch.bfloat16
+    assert lat.shape == (T, H, rank) and cache.shape[1:] == (1, PAGE, E)
+    _check_sinks(sinks, H)
+    if not latent_decode_supports(rank, E - rank):
+        raise Unsupported(f"latent_decode takes ranks up to {LATENT_MAX_RANK} and rotated parts in multiples of 16, "
+                          f"not {rank} + {E - rank}")
+    n_chunks = n_chunks or latent_decode_chunks(T, H, block_table.shape[1], n_sm(q.device))
+    part_o = part_ml = None
+    if n_chunks > 1:
+        part_o = guard.scratch((T * H * n_chunks * rank,), torch.float32, q.device, "latent attention partials")
+        part_ml = guard.scratch((T * H * n_chunks * 2,), torch.float32, q.device, "latent attention statistics")
+    f = _fn("latent_cache", "llmx_latent_decode",
+            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_int,
+             c_int, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p])
+    _check(f(_ptr(q), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(ctx.token_seq), _ptr(ctx.token_pos),
+             _ptr(ctx.seq_past), _ptr(sinks), scale, T, H, rank, E - rank, n_chunks, _ptr(part_o), _ptr(part_ml), _ptr(lat),
+             ctx.n_seqs, cache.shape[0], _stream()), "latent_decode")
+    if n_chunks > 1:
+        global launch_count
+        launch_count += 1
+
+
+def latent_gather(cache, block_table, ctx, scratch_table, c_out, rank: int) -> None:
+    """The latents of the step's sequences (bfloat16), out of their pages into rows of ``c_out`` [64 * ctx.ctx_pages,
+    rank], every sequence from a multiple of 64; ``scratch_table`` [n_seqs, width] becomes the block table that finds
+    sequence b's page i at its place in that order."""
+    _dev(cache, block_table, scratch_table, c_out)
+    _contig("cache", cache), _contig("block_table", block_table), _contig("scratch_table", scratch_table), _contig("c_out", c_out)
+    assert cache.dtype == c_out.dtype == torch.bfloat16 and c_out.shape == (PAGE * ctx.ctx_pages, rank)
+    assert scratch_table.shape == block_table.shape and scratch_table.dtype == torch.int32
+    f = _fn("latent_cache", "llmx_latent_gather",
+            [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p])
+    _check(f(_ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(ctx.seq_start), _ptr(ctx.seq_past), ctx.n_seqs,
+             ctx.ctx_pages, _ptr(scratch_table), _ptr(c_out), rank, cache.shape[3] - rank, cache.shape[0], _stream()),
+           "latent_gather")
+
+
+def latent_assemble(kv, cache, block_table, ctx, k_out, v_out, n_heads: int, head_dim: int, rot_dim: int, v_head_dim: int,
+                    rank: int) -> None:
+    """Every head's keys [rotated part | W_uk c] and values in scratch pages: ``kv`` [64 * pages, H*D + H*Dv] in the rows'
+    order of ``latent_gather``, k_out [pages, H, 64, R + D], v_out [pages, H, 64, Dv]."""
+    _dev(kv, cache, block_table, k_out, v_out)
+    for name, t in (("kv", kv), ("cache", cache), ("block_table", block_table), ("k_out", k_out), ("v_out", v_out)):
+        _contig(name, t)
+    H, D, R, Dv, n = n_heads, head_dim, rot_dim, v_head_dim, ctx.ctx_pages
+    assert kv.shape == (PAGE * n, H * (D + Dv)) and k_out.shape == (n, H, PAGE, R + D) and v_out.shape == (n, H, PAGE, Dv)
+    assert kv.dtype == k_out.dtype == v_out.dtype == cache.dtype == torch.bfloat16
+    f = _fn("latent_cache", "llmx_latent_assemble",
+            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+             c_int, c_int, c_longlong, c_void_p])
+    _check(f(_ptr(kv), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(ctx.seq_start), _ptr(ctx.seq_past),
+             ctx.n_seqs, n, _ptr(k_out), _ptr(v_out), H, D, R, Dv, rank, cache.shape[0], _stream()), "latent_assemble")
 
 
 def head_gate(out, gate, n_heads: int, v_head_dim: int) -> None:

@@ -21,15 +21,29 @@ rms is x / sqrt(mean(x^2) + eps) in float32.  The rotation is the position
 part's (any table of ``rot_dim`` dimensions: scaled frequencies, an amplitude).
 
 What is cached.  The latent c and the rotated part kr are all that later
-tokens need, and a cache of those alone is the smallest there is; this part
-caches every head's assembled key [rot(kr) | k_plain] and value instead, H
-heads of R + D and Dv, because the design it was built for attends under a
-window: the cache holds at most the window's tokens per sequence whatever the
-context's length, and assembled keys run on every attention kernel of this
-package (tensor cores for prompts and decode at R + D = Dv in {64, 128})
-without a product per cached token in every step.  Within a head the rotated
-part is stored first, which no scalar product notices as queries are laid out
-alike.
+tokens need.  ``cache`` "heads" (the default) keeps every head's assembled key
+[rot(kr) | k_plain] and value, H heads of R + D and Dv: for a design that
+attends under a window the cache holds at most the window's tokens per sequence
+whatever the context's length, and assembled keys run on every attention kernel
+of this package (tensor cores for prompts and decode at R + D = Dv in {64,
+128}) without a product per cached token in every step.  Within a head the
+rotated part is stored first, which no scalar product notices as queries are
+laid out alike.
+
+``cache`` "latent" keeps the row [c | rot(kr)] alone, kv_rank + R numbers per
+position for all heads together (built without a window, without an output
+gate, with queries straight from the input).  Three ways to attend over it, all
+the same sums:
+  * few new tokens (decode steps, short portions), bfloat16: the query goes
+    through W_uk first, so that the cached rows are keys and values of every
+    head as they are (``kernels.latent_decode``), and the sum of latents goes
+    through W_uv behind it;
+  * prompts at R + D = Dv in {64, 128}, bfloat16: the latents of the step's
+    sequences are gathered, one product [W_uk; W_uv] c makes every head's keys
+    and values for them, these are laid out in scratch pages, and the tiled
+    prompt attention reads those like a cache;
+  * everything else (float32, other sizes): absorbed like the first, in float32
+    arithmetic (``kernels.latent_paged``).
 
 Products: W_dq, W_dkv and W_g read the same rows and are one fused product
 (float32 out, so the norms and the gate see unrounded sums); W_uk and W_uv are
@@ -49,6 +63,11 @@ from .position import halves_order
 from .registry import register_mixer
 
 
+# Steps of single tokens, and others of up to this many, attend over the latents as they are; longer ones expand them
+# first (see above).
+ABSORB_MAX_TOKENS = 64
+
+
 @register_mixer("latent_attention")
 class LatentAttention:
     def __init__(self, spec, position, weights: dict, rt):
@@ -64,24 +83,23 @@ class LatentAttention:
             raise Unsupported("latent attention rotates exactly its rot_dim dimensions: the position part must say so")
         self.position = position
         self.E = self.R + self.D                      # an assembled key, a query head
-        if max(self.E, self.Dv) > 256:
+        self.latent_cache = spec.get("cache", "heads") == "latent"
+        if max(self.E, self.Dv) > 256 and not self.latent_cache:
             raise Unsupported(f"head sizes {self.E}/{self.Dv}: the attention kernels take sizes up to 256")
         H, D, R, Dv = self.H, self.D, self.R, self.Dv
         t = spec.tensors
         wdkv = weights.pop(t["dkv"].name)
         # the shared rotated part's rows in the order the kernels pair them
         wdkv = torch.cat([wdkv[: self.Rkv], halves_order(position, wdkv[self.Rkv :], 1, R)], dim=0)
+        if self.latent_cache:
+            self._init_latent_cache(wdkv, weights, t)
+            return
         rows = ([weights.pop(t["dq"].name)] if self.Rq else []) + [wdkv] + ([weights.pop(t["g"].name)] if self.gate else [])
         if len({w.dtype for w in rows}) > 1:
             rows = [w.float() for w in rows]
         self.down = Linear(torch.cat(rows, dim=0).contiguous(), rt)
         self.k_rot_off, self.gate_off = self.Rq + self.Rkv, self.Rq + self.Rkv + R
-        # queries: every head's rows become [rotated (paired as the kernels pair) | unrotated]
-        wuq = weights.pop(t["uq" if self.Rq else "q"].name)
-        wuq = halves_order(position, wuq, H, D + R, first=D)
-        index = torch.tensor([h * (D + R) + i for h in range(H) for i in list(range(D, D + R)) + list(range(D))],
-                             device=wuq.device)
-        self.uq = Linear(wuq.index_select(0, index).contiguous(), rt)
+        self.uq = Linear(self._query_rows(weights.pop(t["uq" if self.Rq else "q"].name)), rt)
         wuk, wuv = weights.pop(t["uk"].name), weights.pop(t["uv"].name)
         if wuk.dtype != wuv.dtype:
             wuk, wuv = wuk.float(), wuv.float()
@@ -94,10 +112,53 @@ class LatentAttention:
         # the shape the tiled kernels are written for
         self.plain = self.E == Dv and self.E % 16 == 0
 
+    def _query_rows(self, w):
+        """Every head's rows of a query projection become [rotated (paired as the kernels pair) | unrotated]."""
+        H, D, R = self.H, self.D, self.R
+        w = halves_order(self.position, w, H, D + R, first=D)
+        index = torch.tensor([h * (D + R) + i for h in range(H) for i in list(range(D, D + R)) + list(range(D))],
+                             device=w.device)
+        return w.index_select(0, index).contiguous()
+
+    def _init_latent_cache(self, wdkv, weights, t):
+        if self.Rq or self.gate or self.window:
+            raise Unsupported("a cache of latents is built without a query latent, an output gate and a window")
+        H, D, Dv, rank, rt = self.H, self.D, self.Dv, self.Rkv, self.rt
+        wq = self._query_rows(weights.pop(t["q"].name))
+        if wq.dtype != wdkv.dtype:
+            wq, wdkv = wq.float(), wdkv.float()
+        fused = torch.cat([wdkv, wq], dim=0).contiguous()
+        n = rank + self.R
+        # one product for both in steps of few tokens; in prompts the latent's rows leave it in float32, the query's in
+        # the compute dtype
+        self.down_q, self.down, self.q_proj = Linear(fused, rt), Linear(fused[:n], rt), Linear(fused[n:], rt)
+        wuk, wuv = weights.pop(t["uk"].name), weights.pop(t["uv"].name)
+        if wuk.dtype != wuv.dtype:
+            wuk, wuv = wuk.float(), wuv.float()
+        # keys into the query: W_uk,h^T as [H, rank, D]; values out of the sum of latents: W_uv,h as [H, Dv, rank]
+        self.absorb_w = wuk.view(H, D, rank).transpose(1, 2).contiguous()
+        ukv = torch.cat([wuk, wuv], dim=0).contiguous()
+        self.expand_w = ukv[H * D :].view(H, Dv, rank)
+        self.ukv = Linear(ukv, rt)
+        self.kv_gain = weights.pop(t["dkv_norm"].name).to(torch.float32).contiguous()
+        self.sinks = weights.pop(t["sink"].name).to(torch.float32).contiguous() if "sink" in t else None
+        self.o = Linear(weights.pop(t["o"].name), rt)
+        self.out_bias, self.defer_out_bias = None, False
+        bf16 = rt.dtype == "bfloat16" and rt.tensor_cores and ukv.dtype == torch.bfloat16 and self.scale > 0
+        self.fast_absorbed = bf16 and kernels.latent_decode_supports(rank, self.R) and D % 8 == 0
+        self.fast_expanded = bf16 and self.E == Dv and self.E in (64, 128)
+
     def cache_need(self):
+        if self.latent_cache:
+            return KVNeed(1, self.Rkv + self.R, None, v_head_dim=0), None
         return KVNeed(self.H, self.E, self.window, v_head_dim=None if self.Dv == self.E else self.Dv), None
 
     def libraries(self) -> set:
+        if self.latent_cache:
+            libs = {"latent_cache", "elementwise"} | self.down_q.libraries() | self.ukv.libraries() | self.o.libraries()
+            if self.fast_expanded:
+                libs.add("attention_prefill_tc" if self.E == 128 else "attention_prefill")
+            return libs
         libs = {"latent_attention", "elementwise"} | self.down.libraries() | self.uq.libraries() | self.o.libraries()
         if self.plain and self.rt.dtype == "bfloat16" and self.rt.tensor_cores:
             libs |= {"attention_decode",
@@ -109,6 +170,8 @@ class LatentAttention:
     def forward(self, x, ctx, view, writes_cache=True):
         if not writes_cache:
             raise Unsupported("a latent attention layer owns its cache entry")
+        if self.latent_cache:
+            return self.o(self._attend_latents(x, ctx, view), splits_ok=True)
         H, D, R, Dv, E = self.H, self.D, self.R, self.Dv, self.E
         T, dev, act = x.shape[0], x.device, self.rt.act_dtype
         down = self.down(x, out_dtype=torch.float32)                         # [T, Rq + Rkv + R (+ H)]
@@ -126,6 +189,45 @@ class LatentAttention:
         out = torch.empty((T, H * Dv), dtype=act, device=dev)
         self.attend(q, out, view, block_table, ctx, gate)
         return self.o(out, splits_ok=True)
+
+    def _attend_latents(self, x, ctx, view):
+        H, D, R, Dv, E, rank = self.H, self.D, self.R, self.Dv, self.E, self.Rkv
+        T, dev, act = x.shape[0], x.device, self.rt.act_dtype
+        cos, sin, _ = self.position.rotary_tables()
+        block_table = ctx.block_tables[view.group]
+        new = lambda *shape, dtype=act: torch.empty(shape, dtype=dtype, device=dev)
+        if T <= ABSORB_MAX_TOKENS:
+            both = self.down_q(x, out_dtype=torch.float32, splits_ok=True)
+            down, q = both, both[..., rank + R :]
+        else:
+            down, q = self.down(x, out_dtype=torch.float32, splits_ok=True), self.q_proj(x)
+        prep = lambda rot, plain: kernels.latent_prep(down, q, self.kv_gain, self.eps, view.k, rot, plain, block_table, ctx,
+                                                      cos, sin, H, D, R, rank)
+        out = new(T, H, Dv)
+        if self.fast_expanded and T > ABSORB_MAX_TOKENS and not ctx.is_decode:
+            qa = new(T, H, E)
+            prep(qa[:, :, :R], qa[:, :, R:])
+            n = ctx.ctx_pages
+            table, c = torch.empty_like(block_table), new(kernels.PAGE * n, rank)
+            kernels.latent_gather(view.k, block_table, ctx, table, c, rank)
+            kv = self.ukv(c)
+            keys, values = new(n, H, kernels.PAGE, E), new(n, H, kernels.PAGE, Dv)
+            kernels.latent_assemble(kv, view.k, block_table, ctx, keys, values, H, D, R, Dv, rank)
+            prompt = kernels.attention_prefill_tc if E == 128 else kernels.attention_prefill
+            prompt(qa.view(T, H * E), out.view(T, H * Dv), keys, values, table, ctx.seq_start, ctx.seq_past, ctx.n_seqs,
+                   ctx.max_new, H, H, E, None, self.scale, sinks=self.sinks)
+            return out.view(T, H * Dv)
+        # absorbed: [W_uk^T q_plain | rot(q_rot)] against the cached rows, then W_uv
+        dtype = act if self.fast_absorbed else torch.float32
+        qa, plain, lat = new(T, H, rank + R, dtype=dtype), new(T, H, D, dtype=dtype), new(T, H, rank, dtype=dtype)
+        prep(qa[:, :, rank:], plain)
+        kernels.head_product(plain, self.absorb_w, qa[:, :, :rank])
+        if self.fast_absorbed:
+            kernels.latent_decode(qa, lat, view.k, block_table, ctx, self.sinks, self.scale, rank)
+        else:
+            kernels.latent_paged(qa, lat, view.k, block_table, ctx, self.sinks, self.scale, rank)
+        kernels.head_product(lat, self.expand_w, out)
+        return out.view(T, H * Dv)
 
     def attend(self, q, out, view, block_table, ctx, gate):
         """The general kernel applies the heads' gates itself; the tiled bfloat16 kernels (decode, and prompts at
