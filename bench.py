@@ -9,6 +9,8 @@ B200.  A "step" is one decode step of a batch of 8 sequences from depth 2048
     python bench.py --design voserax    # the Voserax decoder beside the Tifapel decoder's attention layers, two sizes
     python bench.py --design ninenex    # the Ninenex decoder beside the Tifapel decoder's retention and attention layers, two sizes
     python bench.py --design fusasun    # the Fusasun decoder beside the Tifapel decoder's attention layers, two sizes
+    python bench.py --design soputar    # the Soputar decoder beside the Tifapel decoder's attention and retention layers and
+                                        # the Fusasun decoder's latent layers, two sizes
 
 ``value`` is device-timed (CUDA events around K steps queued back to back);
 ``e2e`` is the same metric through ``Session.generate`` with host token ids in
@@ -197,7 +199,7 @@ def main() -> int:
                          "one replayed decode step, when each kernel's dependency resolved")
     ap.add_argument("--cpu-baseline", action="store_true",
                     help="instead of the benchmark: time the plain implementation of tests/ on the CPU (tiny configurations)")
-    ap.add_argument("--design", choices=["tifapel", "voserax", "ninenex", "fusasun"], default=None,
+    ap.add_argument("--design", choices=["tifapel", "voserax", "ninenex", "fusasun", "soputar"], default=None,
                     help="instead of the benchmark: prefill and decode rates of that design at layer sizes of a real "
                          "model (random weights), beside the dense Qwen3 decoder at equal sizes, with every kernel's "
                          "time per step (one JSON line of its own; the default workload is untouched)")
@@ -487,6 +489,26 @@ def fusasun_layers(n_layers, heads, kv_heads, dim, window, pool, experts, top, f
     return [json.loads(json.dumps(att if i % 2 else latent)) for i in range(n_layers)]
 
 
+def soputar_layers(n_layers, heads, kv_heads, dim, kv_rank, ff):
+    """Layers in the order attention, gated delta rule, latent attention, attention reading the first one's keys and
+    values; dense feed-forwards; a quarter of a latent head's query/key dimensions are rotated."""
+    mlp = dict(kind="dense", ff=ff, limit=7.0)
+    rot = dim // 4
+    att = dict(type="attention", mlp=mlp, mixer=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5,
+                                                     softcap=30.0, q_temp=dict(coef=0.1, every=1024)))
+    delta = dict(type="delta", mlp=mlp, mixer=dict(heads=heads, kv_heads=heads // 2, dim=dim, vdim=dim, conv=4))
+    latent = dict(type="latent_attention", mlp=mlp, mixer=dict(heads=heads, dim=dim - rot, rot_dim=rot, vdim=dim,
+                                                               kv_rank=kv_rank, scale=dim ** -0.5,
+                                                               rot=dict(base=10000.0, dims=rot)))
+    out = []
+    for i in range(n_layers):
+        layer = json.loads(json.dumps((att, delta, latent, att)[i % 4]))
+        if i % 4 == 3:
+            layer["mixer"]["kv_from"] = i - 3
+        out.append(layer)
+    return out
+
+
 def design_bench(args) -> int:
     """``--design tifapel``: prefill and decode rates of the Tifapel decoder at layer sizes that resemble a real model's (width 2048,
     16 heads of 128 on 4 key/value heads, a window of 1024 that keeps 4 tokens, 16 experts of 1024 of which a
@@ -507,7 +529,12 @@ def design_bench(args) -> int:
 
     ``--design fusasun``: the same measurement of the Fusasun decoder (latent attention and attention over a window
     with pooled blocks in turn, a 4-tap convolution before every mixer, gated results between two norms, experts
-    named by a token table) at the same two sizes, beside the Tifapel decoder's attention layers with routed experts."""
+    named by a token table) at the same two sizes, beside the Tifapel decoder's attention layers with routed experts.
+
+    ``--design soputar``: the same measurement of the Soputar decoder (attention with capped scores, the gated delta
+    rule, latent attention over a cache of latents, attention on borrowed keys and values; dense feed-forwards) at two
+    sizes, beside the Tifapel decoder with attention and retention layers in turn and the Fusasun decoder's latent
+    layers, all without a window that binds, with experts of the same active width."""
     import numpy as np
     import torch
 
@@ -558,6 +585,34 @@ def design_bench(args) -> int:
             runs.append(dict(sizes=dict(width=width, heads=heads, kv_heads=kv, head_dim=dim, window=window, pool=pool,
                                         experts=E, top=top, expert_ff=ff, q_rank=rq, kv_rank=rkv, taps=4, vocab=vocab), **res))
         print(json.dumps(dict(design="fusasun", unit="tokens/s", dtype="bf16", layers=L, peaks=pk_src, hbm_gbs=pk["hbm_gbs"],
+                              bf16_tflops=pk["bf16_tflops"], data="synthetic: seeded uniform token ids, random weights",
+                              runs=runs)))
+        return 0
+    if args.design == "soputar":
+        runs = []
+        for width, heads, kv, dim, rank, E, top, ff in ((2048, 16, 4, 128, 512, 16, 2, 1024), (1024, 16, 8, 64, 256, 8, 2, 512)):
+            moe = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=E, top=top, scale=1.0))
+            far, rot = 1 << 19, dim // 4
+            decay = [1.0 - 2.0 ** -(3 + 7 * h / max(1, heads - 1)) for h in range(heads)]
+            ret = dict(type="retention", mlp=moe, mixer=dict(heads=heads, dim=dim, vdim=dim, decay=decay))
+            att = dict(type="attention", mlp=moe, mixer=dict(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5,
+                                                             mask=dict(size=far, keep_first=0)))
+            lat = dict(type="latent_attention", mlp=dict(kind="moe", expert=dict(ff=ff), router=dict(experts=E, top=top)),
+                       mixer=dict(heads=heads, dim=dim - rot, rot_dim=rot, vdim=dim, q_rank=rank, kv_rank=rank,
+                                  scale=dim ** -0.5, mask=dict(size=far), rot=dict(dims=rot, base=10000.0)))
+            models = {
+                "soputar": dict(architecture="Soputar", vocab=vocab, width=width, norm=dict(eps=1e-6),
+                                embedding=dict(scale=1.0), layers=soputar_layers(L, heads, kv, dim, rank, top * ff)),
+                "tifapel": dict(architecture="Tifapel", vocab=vocab, width=width, norm=dict(eps=1e-6),
+                                layers=[json.loads(json.dumps(ret if i % 2 else att)) for i in range(L)]),
+                "fusasun": dict(architecture="Fusasun", vocab=vocab, width=width, norm=dict(eps=1e-6),
+                                embedding=dict(scale=1.0), canon=dict(taps=4),
+                                layers=[json.loads(json.dumps(lat)) for _ in range(L)]),
+            }
+            res = _design_models(args, models, vocab, T, B, depth, rng)
+            runs.append(dict(sizes=dict(width=width, heads=heads, kv_heads=kv, head_dim=dim, kv_rank=rank, experts=E, top=top,
+                                        expert_ff=ff, dense_ff=top * ff, conv=4, vocab=vocab), **res))
+        print(json.dumps(dict(design="soputar", unit="tokens/s", dtype="bf16", layers=L, peaks=pk_src, hbm_gbs=pk["hbm_gbs"],
                               bf16_tflops=pk["bf16_tflops"], data="synthetic: seeded uniform token ids, random weights",
                               runs=runs)))
         return 0
@@ -624,7 +679,9 @@ def _design_models(args, models, vocab, T, B, depth, rng) -> dict:
             f = raw_fn(lib, name, argtypes)
 
             def call(*a):
-                tag = name.replace("llmx_", "")
+                tag = name.replace("llmx_", "").replace("_capped", "")      # (the entry that also takes a cap's arguments)
+                if lib.endswith("_capped"):
+                    tag += " (capped scores)"
                 if name.startswith("llmx_gemm_tc") and len(a) > 6:
                     tag += f" N{a[5]} K{a[6]}"
                 elif name == "llmx_gemm_fma":

@@ -22,26 +22,30 @@
 // k = q = v = 0, beta = 0, g = 1, which change nothing.
 //   delta_prep   one CTA per (chunk, key head): convolution, activation, unit norms, the two 8 x 8 matrices of dot
 //                products, and per value head the gates and the coefficients above
-//   delta_scan   a group of lanes (32, 16 or 8: D / 4) owns four columns of S, four dims a lane and the columns in
-//                registers; partial products are added up by a transposing reduction.  It also moves the ring on.
+//   delta_scan   a group of lanes (32, 16 or 8: D / 4) owns two or four columns of S, four dims a lane and column in
+//                registers; the partial products of a chunk's eight tokens are added up by a halving reduction that
+//                leaves every lane the sums of its own token and column
+//   delta_ring   moves the ring on
 // Single tokens: delta_decode, one CTA per (sequence, value head), does all of it and the norm and gate behind the
 // recurrence (y = o / sqrt(mean o^2 + eps) * gain * silu(gate)), reading and writing S once.
 //
 // Everything is float32.  A decode step's sums and a prompt's are ordered differently, so a position's result may
 // differ in rounding between cuttings.
-#include "common.cuh"
+#include "tc_ptx.cuh"
 
 #define DR_CHUNK 8
 #define DR_STAGES 3
 #define DR_MAX_D 256
 #define DR_MAX_TAPS 16
-#define DR_A 0                   // coefficients of a (chunk, value head): A [8][8] (column j < i: beta_i R_ij k_i.k_j)
-#define DR_B 64                  // B [8][8] (column j <= i: R_ij q_i.k_j)
-#define DR_BG 128                // beta_i gamma_i [8]
-#define DR_G 136                 // gamma_i [8]
-#define DR_W 144                 // R_7j [8]
-#define DR_GL 152                // gamma_7, then padding
-#define DR_COEF 156              // floats
+// coefficients of a (chunk, value head), floats
+#define DR_A 0                   // A, rows 1..7 of a strictly lower triangle: row i at i (i - 1) / 2, beta_i R_ij k_i.k_j
+#define DR_BG 28                 // beta_i gamma_i [8]
+#define DR_W 36                  // R_7j [8]
+#define DR_G 44                  // gamma_i [8]
+#define DR_GL 52                 // gamma_7, three unused
+#define DR_B 56                  // B [8][8] (column j <= i: R_ij q_i.k_j)
+#define DR_COEF 120
+#define DR_PAD 16                // floats between the rows of q and k in delta_prep: its 16-byte reads meet no bank twice
 
 __device__ __forceinline__ float dr_silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float dr_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -117,19 +121,20 @@ __device__ __forceinline__ void dr_conv8(const DeltaIn& in, const TIN* proj, con
   for (int i = 0; i < DR_CHUNK; ++i) y[i] = i < n ? dr_silu(y[i]) : 0.f;
 }
 
-// prep buffers: qk [slots][G][2][8][Dp] (keys, then queries), vv [slots][H][8][Dvp] (beta_i v_i), co [slots][H][DR_COEF]
+// prep buffers: qk [slots][G][2][8][DL] (keys, then queries; DL: the staged row of delta_scan, zeros beyond D), vv [slots][H][Dvp][8] (beta_i v_i, a column's tokens
+// together), co [slots][H][DR_COEF]
 template <typename TIN, int TAPS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* __restrict__ state,
                   float* __restrict__ qk, float* __restrict__ vv, float* __restrict__ co,
                   const int* __restrict__ seq_start, const int* __restrict__ seq_past,
-                  const int* __restrict__ seq_slot, int n_seqs, int n_tokens, int n_slots) {
-  extern __shared__ __align__(16) float dr_smem[];
+                  const int* __restrict__ seq_slot, int n_seqs, int n_tokens, int n_slots, int DL) {
+  extern __shared__ __align__(128) float dr_smem[];
   pdl_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int slot = blockIdx.x, j = blockIdx.y;        // chunk slot, key/query head
   const int H = in.H, G = in.G, D = in.D, Dv = in.Dv, R = H / G, C = 2 * G * D + H * Dv;
-  const int Dp = (D + 3) & ~3, Dvp = (Dv + 3) & ~3, ld = Dp + 4;
+  const int Dp = (D + 3) & ~3, Dvp = (Dv + 3) & ~3, ld = Dp + DR_PAD;
   const int b = dr_find_seq(seq_start, n_seqs, slot);
   const int row0 = seq_start[b], n_new = seq_start[b + 1] - row0, p0 = seq_past[b], sl = seq_slot[b];
   const int chunk = slot - (row0 / DR_CHUNK + b);
@@ -145,6 +150,23 @@ delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* _
   float* dots = sq + DR_CHUNK * ld;                   // [2][8][8]: k_i . k_j, q_i . k_j
   float* gates = dots + 128;                          // [R][2][8]: beta, g
   pdl_wait();
+  // ---- values of the head's value heads, a channel a thread; the first ones wait in registers for their beta, so that
+  // their loads are in flight together with those of q and k
+  auto value = [&](int e, float* y) {
+    const int hr = e / Dvp, d = e - hr * Dvp;
+#pragma unroll
+    for (int i = 0; i < DR_CHUNK; ++i) y[i] = 0.f;
+    if (d < Dv) dr_conv8<TAPS>(in, proj, ring, C, 2 * G * D + (j * R + hr) * Dv + d, row0, p0, pos0, n, y);
+  };
+  auto put_value = [&](int e, const float* y) {
+    const int hr = e / Dvp, d = e - hr * Dvp;
+    const float* beta = gates + hr * 16;
+    float4* out = reinterpret_cast<float4*>(vv + (((size_t)slot * H + j * R + hr) * Dvp + d) * DR_CHUNK);
+    out[0] = make_float4(y[0] * beta[0], y[1] * beta[1], y[2] * beta[2], y[3] * beta[3]);
+    out[1] = make_float4(y[4] * beta[4], y[5] * beta[5], y[6] * beta[6], y[7] * beta[7]);
+  };
+  float y_first[DR_CHUNK];
+  if (tid < R * Dvp) value(tid, y_first);
   // ---- q and k of this head: convolution and activation, one channel a thread
   for (int e = tid; e < 2 * Dp; e += blockDim.x) {
     const bool is_k = e >= Dp;
@@ -157,7 +179,7 @@ delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* _
 #pragma unroll
     for (int i = 0; i < DR_CHUNK; ++i) dst[i * ld] = y[i];
   }
-  // ---- gates of the head's value heads
+  // ---- gates
   for (int e = tid; e < R * DR_CHUNK; e += blockDim.x) {
     const int hr = e / DR_CHUNK, i = e - hr * DR_CHUNK, h = j * R + hr;
     float beta = 0.f, g = 1.f;
@@ -171,6 +193,7 @@ delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* _
     gates[hr * 16 + 8 + i] = g;
   }
   __syncthreads();
+  if (tid < R * Dvp) put_value(tid, y_first);
   // ---- unit norms: one warp per row
   for (int r = warp; r < 2 * DR_CHUNK; r += blockDim.x >> 5) {
     const bool is_q = r >= DR_CHUNK;
@@ -178,22 +201,28 @@ delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* _
     float ss = 0.f;
     for (int d = lane; d < D; d += 32) ss += row[d] * row[d];
     const float scale = (is_q ? in.q_scale : 1.f) / sqrtf(warp_sum(ss) + in.unit_eps);
-    float* out = qk + (((size_t)slot * G + j) * 2 + (is_q ? 1 : 0)) * DR_CHUNK * Dp + (size_t)(r & 7) * Dp;
-    for (int d = lane; d < Dp; d += 32) {
-      const float x = row[d] * scale;
-      row[d] = x;
+    float* out = qk + (((size_t)slot * G + j) * 2 + (is_q ? 1 : 0)) * DR_CHUNK * DL + (size_t)(r & 7) * DL;
+    for (int d = lane; d < DL; d += 32) {
+      const float x = d < Dp ? row[d] * scale : 0.f;
+      if (d < Dp) row[d] = x;
       out[d] = x;
     }
   }
   __syncthreads();
-  // ---- the dot products, four lanes each
+  // ---- the dot products, four lanes each (rows of 4-float pieces, a lane every fourth piece)
   for (int e = tid; e < 128 * 4; e += blockDim.x) {   // (a warp's 32 threads take part together: 512 is a multiple)
     const int pair = e >> 2, part = e & 3, which = pair >> 6, i = (pair >> 3) & 7, jj = pair & 7;
     const float* x = (which ? sq : sk) + i * ld;
     const float* y = sk + jj * ld;
     float s = 0.f;
     if (which ? jj <= i : jj < i)
-      for (int d = part; d < D; d += 4) s = fmaf(x[d], y[d], s);
+      for (int d = 4 * part; d < Dp; d += 16) {
+        const float4 xa = *reinterpret_cast<const float4*>(x + d), ya = *reinterpret_cast<const float4*>(y + d);
+        s = fmaf(xa.x, ya.x, s);
+        s = fmaf(xa.y, ya.y, s);
+        s = fmaf(xa.z, ya.z, s);
+        s = fmaf(xa.w, ya.w, s);
+      }
     s += __shfl_xor_sync(0xffffffffu, s, 1);
     s += __shfl_xor_sync(0xffffffffu, s, 2);
     if (part == 0) dots[pair] = s;
@@ -207,7 +236,7 @@ delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* _
     float* c = co + ((size_t)slot * H + j * R + hr) * DR_COEF;
     float rij = 1.f;
     for (int m = jj + 1; m <= i; ++m) rij *= g[m];
-    c[DR_A + i * 8 + jj] = jj < i ? beta[i] * rij * dots[i * 8 + jj] : 0.f;
+    if (jj < i) c[DR_A + i * (i - 1) / 2 + jj] = beta[i] * rij * dots[i * 8 + jj];
     c[DR_B + i * 8 + jj] = jj <= i ? rij * dots[64 + i * 8 + jj] : 0.f;
     if (i == 7) c[DR_W + jj] = rij;
     if (jj == 0) {
@@ -217,61 +246,54 @@ delta_prep_kernel(const TIN* __restrict__ proj, const DeltaIn in, const float* _
       if (i == 7) c[DR_GL] = gam, c[DR_GL + 1] = c[DR_GL + 2] = c[DR_GL + 3] = 0.f;
     }
   }
-  // ---- values
-  for (int e = tid; e < R * Dvp; e += blockDim.x) {
-    const int hr = e / Dvp, d = e - hr * Dvp, h = j * R + hr;
+  for (int e = tid + blockDim.x; e < R * Dvp; e += blockDim.x) {        // the value channels beyond a thread's first
     float y[DR_CHUNK];
-#pragma unroll
-    for (int i = 0; i < DR_CHUNK; ++i) y[i] = 0.f;
-    if (d < Dv) dr_conv8<TAPS>(in, proj, ring, C, 2 * G * D + h * Dv + d, row0, p0, pos0, n, y);
-    float* out = vv + ((size_t)slot * H + h) * DR_CHUNK * Dvp + d;
-#pragma unroll
-    for (int i = 0; i < DR_CHUNK; ++i) out[(size_t)i * Dvp] = y[i] * gates[hr * 16 + i];
+    value(e, y);
+    put_value(e, y);
   }
 }
 
-__device__ __forceinline__ void dr_cp_async16(float* dst, const float* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src)
+__host__ __device__ constexpr int dr_log2(int n) { return n <= 1 ? 0 : 1 + dr_log2(n / 2); }
+
+__device__ __forceinline__ void dr_bulk_copy(uint32_t dst, const float* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
+               "l"(src), "r"(bytes), "r"(bar)
                : "memory");
 }
-
-// Adds N values over LANES neighbouring lanes; afterwards lane r (of the group) holds the sums of the values
-// r * (N / LANES) .. + N / LANES - 1 in v[0 ..].  Halving: at every step a lane hands half of its values to its partner.
-template <int N, int LANES>
-__device__ __forceinline__ void dr_reduce(float* v, int r) {
-  int n = N;
-#pragma unroll
-  for (int bit = LANES / 2; bit > 0; bit >>= 1) {
-    n >>= 1;
-    const bool up = (r & bit) != 0;
-#pragma unroll
-    for (int i = 0; i < N / 2; ++i) {
-      if (i < n) {
-        const float mine = up ? v[n + i] : v[i], give = up ? v[i] : v[n + i];
-        v[i] = mine + __shfl_xor_sync(0xffffffffu, give, bit);
-      }
-    }
-  }
+// Eight neighbouring floats of shared memory, 16-byte aligned.
+__device__ __forceinline__ void dr_load8(const float* p, float* x) {
+  const float4 a = *reinterpret_cast<const float4*>(p), c = *reinterpret_cast<const float4*>(p + 4);
+  x[0] = a.x, x[1] = a.y, x[2] = a.z, x[3] = a.w, x[4] = c.x, x[5] = c.y, x[6] = c.z, x[7] = c.w;
 }
 
-#define DR_WARPS 4
-
-// Four columns of S per group of LANES lanes; lane r of a group owns dims 4 (r + LANES i) + 0..3, i < NI.
-template <int LANES, int NI>
-__global__ void __launch_bounds__(DR_WARPS * 32)
+// CPG columns of S per group of LANES lanes; lane r of a group owns dims 4 (r + LANES i) + 0..3, i < NI, of each.
+// Chunks come into a ring of shared-memory stages by bulk copies of one thread, two chunks ahead.
+//
+// How a chunk's partial products are added up.  A lane's bits say, from the top, which tokens, which column and which
+// copy of them it ends up with: TB token bits (a lane ends with NT = 8 >> TB neighbouring tokens), CB column bits, the
+// rest copies.  A lane takes the rows of k or q in the order i ^ (its token bits) and keeps column p ^ (its column) at
+// place p of its registers, so that at every halving what it keeps lies in the lower half of its array and what its
+// partner is owed in the upper half: one shuffle and one addition a value, no selects.  The same order gives every lane
+// the other columns' u with one shuffle each.
+template <int LANES, int NI, int CPG>
+__global__ void __launch_bounds__(128)
 delta_scan_kernel(const float* __restrict__ qk, const float* __restrict__ vv, const float* __restrict__ co,
                   float* __restrict__ out, float* __restrict__ state, size_t slot_stride,
                   const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int H, int G, int D, int Dv,
                   int n_slots) {
-  extern __shared__ __align__(16) float dr_smem[];
-  constexpr int GROUPS = 32 / LANES, COLS = DR_WARPS * GROUPS * 4;     // columns of a CTA
-  const int Dp = (D + 3) & ~3, Dvp = (Dv + 3) & ~3;
-  const int stage_len = 2 * DR_CHUNK * Dp + DR_CHUNK * COLS + DR_COEF;
-  float* work = dr_smem + DR_STAGES * stage_len;       // [DR_WARPS][GROUPS][64 sums | 32 weighted u]
+  extern __shared__ __align__(128) float dr_smem[];
+  __shared__ __align__(8) uint64_t dr_bars[DR_STAGES];
+  constexpr int GROUPS = 32 / LANES, CB = dr_log2(CPG), LB = dr_log2(LANES);
+  constexpr int TB = LB - CB < 3 ? LB - CB : 3, DUP = LB - CB - TB, NT = 8 >> TB;
+  constexpr int DL = 4 * LANES * NI;                   // dims of a staged row (beyond D: zeros)
+  const int cols = (blockDim.x >> 5) * GROUPS * CPG;   // columns of the CTA
+  const int Dvp = (Dv + 3) & ~3;
+  const int stage_len = 2 * DR_CHUNK * DL + DR_COEF + DR_CHUNK * cols;
   pdl_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, grp = lane / LANES, r = lane % LANES;
-  const int b = blockIdx.z, h = blockIdx.y, c_cta = blockIdx.x * COLS;
-  const int c_loc = (warp * GROUPS + grp) * 4, c0 = c_cta + c_loc;     // this group's first column
+  const int b = blockIdx.z, h = blockIdx.y, c_cta = blockIdx.x * cols;
+  const int c_loc = (warp * GROUPS + grp) * CPG, c0 = c_cta + c_loc;   // this group's first column
+  const int tl = r >> (CB + DUP), cl = (r >> DUP) & (CPG - 1), flip = tl << (3 - TB);
   const int row0 = seq_start[b], n_new = seq_start[b + 1] - row0, sl = seq_slot[b];
   if (n_new <= 0) return;
   if (sl < 0 || sl >= n_slots) {
@@ -281,157 +303,170 @@ delta_scan_kernel(const float* __restrict__ qk, const float* __restrict__ vv, co
   float* S = state + (size_t)sl * slot_stride + (size_t)h * D * Dv;
   const int slot0 = row0 / DR_CHUNK + b, n_chunks = (n_new + DR_CHUNK - 1) / DR_CHUNK;
   const int j = h / (H / G);
-  float* wsum = work + (warp * GROUPS + grp) * 96;
-  float* wu = wsum + 64;
+  const uint32_t bars = smem_u32(dr_bars), ring = smem_u32(dr_smem);
+  if (tid == 0) {
+    for (int i = 0; i < DR_STAGES; ++i) mbar_init(bars + 8 * i, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  const uint32_t v_bytes = (uint32_t)(DR_CHUNK * min(cols, Dvp - c_cta)) * 4u;
+  auto load_chunk = [&](int ch) {                      // one thread
+    const int st = ch % DR_STAGES;
+    const uint32_t dst = ring + (uint32_t)(st * stage_len) * 4u, bar = bars + 8 * st;
+    mbar_expect_tx(bar, 2u * DR_CHUNK * DL * 4u + DR_COEF * 4u + v_bytes);
+    dr_bulk_copy(dst, qk + ((size_t)(slot0 + ch) * G + j) * 2 * DR_CHUNK * DL, 2u * DR_CHUNK * DL * 4u, bar);
+    dr_bulk_copy(dst + 2u * DR_CHUNK * DL * 4u, co + ((size_t)(slot0 + ch) * H + h) * DR_COEF, DR_COEF * 4u, bar);
+    dr_bulk_copy(dst + (2u * DR_CHUNK * DL + DR_COEF) * 4u, vv + (((size_t)(slot0 + ch) * H + h) * Dvp + c_cta) * DR_CHUNK,
+                 v_bytes, bar);
+  };
+  __syncthreads();
   pdl_wait();
+  if (tid == 0)
+    for (int c = 0; c < DR_STAGES - 1 && c < n_chunks; ++c) load_chunk(c);
 
-  float s[NI][4][4];                                   // [dims block][dim][column]
+  float s[NI][4][CPG];                                 // [dims block][dim][column c0 + (place ^ cl)]
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
     for (int d = 0; d < 4; ++d)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int dim = 4 * (r + LANES * i) + d;
-        s[i][d][c] = (dim < D && c0 + c < Dv) ? S[(size_t)dim * Dv + c0 + c] : 0.f;
+      for (int c = 0; c < CPG; ++c) {
+        const int dim = 4 * (r + LANES * i) + d, col = c0 + (c ^ cl);
+        s[i][d][c] = (dim < D && col < Dv) ? S[(size_t)dim * Dv + col] : 0.f;
       }
-
-  const int qk_pieces = 2 * DR_CHUNK * Dp / 4, v_pieces = DR_CHUNK * COLS / 4, co_pieces = DR_COEF / 4;
-  auto load_chunk = [&](int ch) {
-    float* buf = dr_smem + (ch % DR_STAGES) * stage_len;
-    const float* qsrc = qk + ((size_t)(slot0 + ch) * G + j) * 2 * DR_CHUNK * Dp;
-    for (int e = tid; e < qk_pieces; e += DR_WARPS * 32) dr_cp_async16(buf + 4 * e, qsrc + 4 * e);
-    const float* vsrc = vv + ((size_t)(slot0 + ch) * H + h) * DR_CHUNK * Dvp;
-    float* vbuf = buf + 2 * DR_CHUNK * Dp;
-    for (int e = tid; e < v_pieces; e += DR_WARPS * 32) {
-      const int i = e / (COLS / 4), c = (e - i * (COLS / 4)) * 4;
-      if (c_cta + c < Dvp) dr_cp_async16(vbuf + i * COLS + c, vsrc + (size_t)i * Dvp + c_cta + c);
-    }
-    const float* csrc = co + ((size_t)(slot0 + ch) * H + h) * DR_COEF;
-    float* cbuf = vbuf + DR_CHUNK * COLS;
-    for (int e = tid; e < co_pieces; e += DR_WARPS * 32) dr_cp_async16(cbuf + 4 * e, csrc + 4 * e);
-  };
-  for (int c = 0; c < DR_STAGES - 1; ++c) {
-    if (c < n_chunks) load_chunk(c);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  }
-  const int col = lane & 3, c_of_lane = c_loc + col;   // (LANES is a multiple of 4)
-  const bool live = c0 + col < Dv;
-  float* out_col = out + (size_t)row0 * H * Dv + (size_t)h * Dv + c0 + col;
+  const bool writes = c0 + cl < Dv && (r & ((1 << DUP) - 1)) == 0;
+  const size_t out_stride = (size_t)H * Dv;
+  float* out_col = out + ((size_t)row0 + tl * NT) * out_stride + (size_t)h * Dv + c0 + cl;    // its first token of a chunk
   for (int ch = 0; ch < n_chunks; ++ch) {
-    if (ch + DR_STAGES - 1 < n_chunks) load_chunk(ch + DR_STAGES - 1);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group %0;" ::"n"(DR_STAGES - 1) : "memory");
-    __syncthreads();
-    const float* buf = dr_smem + (ch % DR_STAGES) * stage_len;
-    const float* kbuf = buf;
-    const float* qbuf = buf + DR_CHUNK * Dp;
-    const float* vbuf = buf + 2 * DR_CHUNK * Dp;
-    const float* cbuf = vbuf + DR_CHUNK * COLS;
-    // ---- S^T k_i and S^T q_i: this lane's dims, then the sum over the group
-    // value index of a sum: column * 8 + token
-    float acc[32];
-    auto products = [&](const float* rows) {
+    // this chunk has landed; everyone has left the one before, whose stage the next copy fills
+    const bool ok = mbar_wait(bars + 8 * (ch % DR_STAGES), (ch / DR_STAGES) & 1);
+    if (!__syncthreads_and(ok)) {
+      if (tid == 0) llmx_report(5);
+      break;
+    }
+    if (tid == 0 && ch + DR_STAGES - 1 < n_chunks) load_chunk(ch + DR_STAGES - 1);
+    const float* kbuf = dr_smem + (ch % DR_STAGES) * stage_len;
+    const float* qbuf = kbuf + DR_CHUNK * DL;
+    const float* cbuf = qbuf + DR_CHUNK * DL;
+    const float* vbuf = cbuf + DR_COEF;
+    // ---- rows . S over this lane's dims, then over the group: afterwards res[e] belongs to token tl NT + e, column cl
+    auto products = [&](const float* rows, float* res) {
+      float acc[DR_CHUNK][CPG];
 #pragma unroll
       for (int i = 0; i < DR_CHUNK; ++i) {
-        float p[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int c = 0; c < CPG; ++c) acc[i][c] = 0.f;
+        const float* row = rows + (i ^ flip) * DL + 4 * r;
 #pragma unroll
         for (int ni = 0; ni < NI; ++ni) {
-          const int d = 4 * (r + LANES * ni);
-          if (d < Dp) {
-            const float4 x = *reinterpret_cast<const float4*>(rows + i * Dp + d);
+          const float4 x = *reinterpret_cast<const float4*>(row + 4 * LANES * ni);
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
-              p[c] = fmaf(x.x, s[ni][0][c], p[c]);
-              p[c] = fmaf(x.y, s[ni][1][c], p[c]);
-              p[c] = fmaf(x.z, s[ni][2][c], p[c]);
-              p[c] = fmaf(x.w, s[ni][3][c], p[c]);
-            }
+          for (int c = 0; c < CPG; ++c) {
+            acc[i][c] = fmaf(x.x, s[ni][0][c], acc[i][c]);
+            acc[i][c] = fmaf(x.y, s[ni][1][c], acc[i][c]);
+            acc[i][c] = fmaf(x.z, s[ni][2][c], acc[i][c]);
+            acc[i][c] = fmaf(x.w, s[ni][3][c], acc[i][c]);
           }
         }
-#pragma unroll
-        for (int c = 0; c < 4; ++c) acc[c * 8 + i] = p[c];
       }
-      dr_reduce<32, LANES>(acc, r);
+#pragma unroll
+      for (int t = 0; t < TB; ++t) {
+        const int half = 4 >> t;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (i < half)
+#pragma unroll
+            for (int c = 0; c < CPG; ++c) acc[i][c] += __shfl_xor_sync(0xffffffffu, acc[i + half][c], LANES >> (t + 1));
+      }
+#pragma unroll
+      for (int t = 0; t < CB; ++t) {
+        const int half = CPG >> (t + 1);
+#pragma unroll
+        for (int i = 0; i < NT; ++i)
+#pragma unroll
+          for (int c = 0; c < CPG / 2; ++c)
+            if (c < half) acc[i][c] += __shfl_xor_sync(0xffffffffu, acc[i][c + half], half << DUP);
+      }
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        res[i] = acc[i][0];
+#pragma unroll
+        for (int t = 0; t < DUP; ++t) res[i] += __shfl_xor_sync(0xffffffffu, res[i], 1 << t);
+      }
     };
-    products(kbuf);
-#pragma unroll
-    for (int i = 0; i < 32 / LANES; ++i) wsum[r * (32 / LANES) + i] = acc[i];
-    products(qbuf);
-#pragma unroll
-    for (int i = 0; i < 32 / LANES; ++i) wsum[32 + r * (32 / LANES) + i] = acc[i];
-    __syncwarp();
+    float ks_own[NT], qs[NT], u[DR_CHUNK], w[DR_CHUNK];
+    products(kbuf, ks_own);
+    products(qbuf, qs);
     // ---- the chain from token to token, for this lane's column (every lane of a column alike)
-    float u[DR_CHUNK];
     {
-      const float4 k0 = *reinterpret_cast<const float4*>(wsum + col * 8), k1 = *reinterpret_cast<const float4*>(wsum + col * 8 + 4);
-      const float ks[DR_CHUNK] = {k0.x, k0.y, k0.z, k0.w, k1.x, k1.y, k1.z, k1.w};
+      float bg[DR_CHUNK], a[28];
+      dr_load8(vbuf + (c_loc + cl) * 8, u);
+      dr_load8(cbuf + DR_BG, bg);
 #pragma unroll
-      for (int i = 0; i < DR_CHUNK; ++i) u[i] = fmaf(-cbuf[DR_BG + i], ks[i], vbuf[i * COLS + c_of_lane]);
+      for (int i = 0; i < 28; i += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(cbuf + DR_A + i);
+        a[i] = x.x, a[i + 1] = x.y, a[i + 2] = x.z, a[i + 3] = x.w;
+      }
+      const int base = lane & ~((LANES - 1) & ~((1 << (CB + DUP)) - 1));      // token bits cleared
 #pragma unroll
-      for (int i = 0; i < DR_CHUNK; ++i)
+      for (int i = 0; i < DR_CHUNK; ++i) {
+        const float ks = __shfl_sync(0xffffffffu, ks_own[i % NT], base | ((i / NT) << (CB + DUP)));
+        u[i] = fmaf(-bg[i], ks, u[i]);
+      }
 #pragma unroll
-        for (int m = i + 1; m < DR_CHUNK; ++m) u[m] = fmaf(-cbuf[DR_A + m * 8 + i], u[i], u[m]);
+      for (int i = 1; i < DR_CHUNK; ++i)
+#pragma unroll
+        for (int m = 0; m < i; ++m) u[i] = fmaf(-a[i * (i - 1) / 2 + m], u[m], u[i]);
     }
-    // ---- outputs: the lanes of a column share its eight tokens
-    const int n_tok = min(DR_CHUNK, n_new - ch * DR_CHUNK);
-#pragma unroll
-    for (int e = 0; e < DR_CHUNK * 4 / LANES; ++e) {
-      const int i = (r >> 2) + e * (LANES / 4);
-      float o = cbuf[DR_G + i] * wsum[32 + col * 8 + i];
-      const float4 b0 = *reinterpret_cast<const float4*>(cbuf + DR_B + i * 8), b1 = *reinterpret_cast<const float4*>(cbuf + DR_B + i * 8 + 4);
-      o = fmaf(b0.x, u[0], o);
-      o = fmaf(b0.y, u[1], o);
-      o = fmaf(b0.z, u[2], o);
-      o = fmaf(b0.w, u[3], o);
-      o = fmaf(b1.x, u[4], o);
-      o = fmaf(b1.y, u[5], o);
-      o = fmaf(b1.z, u[6], o);
-      o = fmaf(b1.w, u[7], o);
-      if (live && i < n_tok) out_col[(size_t)(ch * DR_CHUNK + i) * H * Dv] = o;
-    }
-    // ---- the state: every lane needs all four columns' u, weighted
-    if (r < 4) {
-#pragma unroll
-      for (int i = 0; i < DR_CHUNK; ++i) wu[i * 4 + col] = cbuf[DR_W + i] * u[i];
-    }
-    __syncwarp();
+    dr_load8(cbuf + DR_W, w);
     const float gl = cbuf[DR_GL];
 #pragma unroll
-    for (int i = 0; i < NI; ++i)
+    for (int i = 0; i < DR_CHUNK; ++i) w[i] *= u[i];
+#pragma unroll
+    for (int ni = 0; ni < NI; ++ni)
 #pragma unroll
       for (int d = 0; d < 4; ++d)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) s[i][d][c] *= gl;
+        for (int c = 0; c < CPG; ++c) s[ni][d][c] *= gl;
 #pragma unroll
     for (int i = 0; i < DR_CHUNK; ++i) {
-      const float4 w = *reinterpret_cast<const float4*>(wu + i * 4);
+      float wc[CPG];
+      wc[0] = w[i];
+#pragma unroll
+      for (int c = 1; c < CPG; ++c) wc[c] = __shfl_xor_sync(0xffffffffu, w[i], c << DUP);
 #pragma unroll
       for (int ni = 0; ni < NI; ++ni) {
-        const int d = 4 * (r + LANES * ni);
-        if (d < Dp) {
-          const float4 x = *reinterpret_cast<const float4*>(kbuf + i * Dp + d);
-          const float xs[4] = {x.x, x.y, x.z, x.w};
+        const float4 x = *reinterpret_cast<const float4*>(kbuf + i * DL + 4 * (r + LANES * ni));
 #pragma unroll
-          for (int dd = 0; dd < 4; ++dd) {
-            s[ni][dd][0] = fmaf(xs[dd], w.x, s[ni][dd][0]);
-            s[ni][dd][1] = fmaf(xs[dd], w.y, s[ni][dd][1]);
-            s[ni][dd][2] = fmaf(xs[dd], w.z, s[ni][dd][2]);
-            s[ni][dd][3] = fmaf(xs[dd], w.w, s[ni][dd][3]);
-          }
+        for (int c = 0; c < CPG; ++c) {
+          s[ni][0][c] = fmaf(x.x, wc[c], s[ni][0][c]);
+          s[ni][1][c] = fmaf(x.y, wc[c], s[ni][1][c]);
+          s[ni][2][c] = fmaf(x.z, wc[c], s[ni][2][c]);
+          s[ni][3][c] = fmaf(x.w, wc[c], s[ni][3][c]);
         }
       }
     }
-    __syncthreads();                                   // the buffer is refilled by the next round's copies
+    // ---- outputs
+    const int n_tok = n_new - ch * DR_CHUNK;
+#pragma unroll
+    for (int e = 0; e < NT; ++e) {
+      const int i = tl * NT + e;
+      float bi[DR_CHUNK];
+      dr_load8(cbuf + DR_B + i * 8, bi);
+      float o = cbuf[DR_G + i] * qs[e];
+#pragma unroll
+      for (int m = 0; m < DR_CHUNK; ++m) o = fmaf(bi[m], u[m], o);
+      if (writes && i < n_tok) out_col[e * out_stride] = o;
+    }
+    out_col += DR_CHUNK * out_stride;
   }
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
     for (int d = 0; d < 4; ++d)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int dim = 4 * (r + LANES * i) + d;
-        if (dim < D && c0 + c < Dv) S[(size_t)dim * Dv + c0 + c] = s[i][d][c];
+      for (int c = 0; c < CPG; ++c) {
+        const int dim = 4 * (r + LANES * i) + d, col = c0 + (c ^ cl);
+        if (dim < D && col < Dv) S[(size_t)dim * Dv + col] = s[i][d][c];
       }
 }
 
@@ -464,7 +499,7 @@ __global__ void __launch_bounds__(256)
 delta_decode_kernel(const TIN* __restrict__ proj, const DeltaIn in, float* __restrict__ state,
                     const float* __restrict__ gain, float eps, TO* __restrict__ y, const int* __restrict__ seq_past,
                     const int* __restrict__ seq_slot, int n_slots) {
-  extern __shared__ __align__(16) float dr_smem[];
+  extern __shared__ __align__(128) float dr_smem[];
   pdl_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int h = blockIdx.x, b = blockIdx.y;
@@ -632,13 +667,13 @@ static int dr_check(const DeltaIn& in, long long row_stride) {
 
 // proj: [T, row_stride] float32 or bfloat16, or n_split float32 partials; state: float32 [n_slots, slot_stride].
 // Prompts: qk, vv, co are float32 scratch, 16-byte aligned, for T / 8 + n_seqs chunks:
-// [chunks, G, 16, Dp], [chunks, H, 8, Dvp], [chunks, H, 156]; out float32 [T, H*Dv].
+// [chunks, G, 16, DL] (DL: D rounded up to 32, 64, 128 or 256), [chunks, H, Dvp, 8], [chunks, H, 120]; out float32 [T, H*Dv].
 LLMX_API int llmx_delta_prompt(const void* proj, int in_dtype, int n_split, long long split_stride, long long row_stride,
                                int q_off, int k_off, int v_off, int b_off, int a_off, int g_off, const float* conv_w,
                                int taps, const float* a_log, const float* dt_bias, float q_scale, float unit_eps,
                                float* state, long long slot_stride, long long ring_off, int n_slots, float* qk, float* vv,
                                float* co, float* out, const int* seq_start, const int* seq_past, const int* seq_slot,
-                               int n_tokens, int n_seqs, int H, int G, int D, int Dv, cudaStream_t stream) {
+                               int n_tokens, int n_seqs, int H, int G, int D, int Dv, int n_sm, cudaStream_t stream) {
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
   const DeltaIn in = {n_split, (size_t)split_stride, (size_t)row_stride, q_off, k_off, v_off, b_off, a_off, g_off,
                       conv_w, a_log, dt_bias, taps, H, G, D, Dv, q_scale, unit_eps, (size_t)slot_stride, (size_t)ring_off};
@@ -646,13 +681,13 @@ LLMX_API int llmx_delta_prompt(const void* proj, int in_dtype, int n_split, long
   if (bad) return bad;
   if (n_seqs > 65535 || H > 65535 || (((uintptr_t)qk | (uintptr_t)vv | (uintptr_t)co | (uintptr_t)state) & 15)) return LLMX_REFUSED(3);
   if (in_dtype != LLMX_F32 && in_dtype != LLMX_BF16) return LLMX_REFUSED(2);
-  const int Dp = (D + 3) & ~3, R = H / G;
-  const size_t psmem = (size_t)(2 * DR_CHUNK * (Dp + 4) + 128 + R * 16) * sizeof(float);
+  const int Dp = (D + 3) & ~3, R = H / G, DL = Dp <= 32 ? 32 : Dp <= 64 ? 64 : Dp <= 128 ? 128 : 256;
+  const size_t psmem = (size_t)(2 * DR_CHUNK * (Dp + DR_PAD) + 128 + R * 16) * sizeof(float);
   if (psmem > 48 * 1024) return LLMX_REFUSED(3);
   const dim3 pgrid(n_tokens / DR_CHUNK + n_seqs, G);
 #define PREP(TIN, TAPS)                                                                                                 \
   launch_pdl(delta_prep_kernel<TIN, TAPS>, pgrid, dim3(256), psmem, stream, (const TIN*)proj, in, (const float*)state,  \
-             qk, vv, co, seq_start, seq_past, seq_slot, n_seqs, n_tokens, n_slots)
+             qk, vv, co, seq_start, seq_past, seq_slot, n_seqs, n_tokens, n_slots, DL)
 #define PREP_T(TIN)                       \
   do {                                    \
     if (taps == 4) PREP(TIN, 4);          \
@@ -666,25 +701,39 @@ LLMX_API int llmx_delta_prompt(const void* proj, int in_dtype, int n_split, long
 #undef PREP
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-#define SCAN(LANES, NI)                                                                                                 \
+  // Launched in order, never beside the preparation: its CTAs all run at once for the whole prompt, and those placed
+  // while another kernel still fills part of the GPU would stay crowded on the SMs that had room (measured: twice the
+  // time).
+  // Two columns a group while that leaves the GPU less than two warps a scheduler, else four; fewer warps a CTA while
+  // there are fewer CTAs than SMs.
+  const int groups = Dp <= 32 ? 4 : Dp <= 64 ? 2 : 1;                   // lane groups per warp
+  const long long heads = (long long)n_seqs * H;
+  const int cpg = heads * ((Dv + 4 * groups - 1) / (4 * groups)) < 8LL * n_sm ? 2 : 4;
+  int warps = 4;
+  while (warps > 1 && heads * ((Dv + warps * groups * cpg - 1) / (warps * groups * cpg)) < n_sm) warps >>= 1;
+  const int cols = warps * groups * cpg;
+  const size_t smem = (size_t)DR_STAGES * (2 * DR_CHUNK * DL + DR_COEF + DR_CHUNK * cols) * sizeof(float);
+#define SCAN2(LANES, NI, CPG)                                                                                           \
   do {                                                                                                                  \
-    const int cols = DR_WARPS * (32 / LANES) * 4;                                                                       \
-    const size_t smem = (size_t)(DR_STAGES * (2 * DR_CHUNK * Dp + DR_CHUNK * cols + DR_COEF) +                          \
-                                 DR_WARPS * (32 / LANES) * 96) * sizeof(float);                                         \
     static bool attr_set = false;                                                                                       \
     if (!attr_set && smem > 48 * 1024) {                                                                                \
-      e = cudaFuncSetAttribute(delta_scan_kernel<LANES, NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);  \
+      e = cudaFuncSetAttribute(delta_scan_kernel<LANES, NI, CPG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); \
       if (e != cudaSuccess) return (int)e;                                                                              \
       attr_set = true;                                                                                                  \
     }                                                                                                                   \
-    launch_pdl(delta_scan_kernel<LANES, NI>, dim3((Dv + cols - 1) / cols, H, n_seqs), dim3(DR_WARPS * 32), smem, stream, \
-               (const float*)qk, (const float*)vv, (const float*)co, out, state, (size_t)slot_stride, seq_start,        \
-               seq_slot, H, G, D, Dv, n_slots);                                                                         \
+    delta_scan_kernel<LANES, NI, CPG><<<dim3((Dv + cols - 1) / cols, H, n_seqs), warps * 32, smem, stream>>>(           \
+        qk, vv, co, out, state, (size_t)slot_stride, seq_start, seq_slot, H, G, D, Dv, n_slots);                        \
+  } while (0)
+#define SCAN(LANES, NI)               \
+  do {                                \
+    if (cpg == 2) SCAN2(LANES, NI, 2); \
+    else SCAN2(LANES, NI, 4);         \
   } while (0)
   if (Dp <= 32) SCAN(8, 1);
   else if (Dp <= 64) SCAN(16, 1);
   else if (Dp <= 128) SCAN(32, 1);
   else SCAN(32, 2);
+#undef SCAN2
 #undef SCAN
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;

@@ -152,7 +152,8 @@ _STATUS_MEANING = {
     "delta_rule": {1: "a sequence's rows or slot lie outside the launch's arrays (preparation)",
                    2: "a sequence's slot lies outside the state area",
                    3: "a sequence's rows or slot lie outside the launch's arrays (convolution rows)",
-                   4: "a sequence's position or slot lies outside the launch's arrays (single tokens)"},
+                   4: "a sequence's position or slot lies outside the launch's arrays (single tokens)",
+                   5: "a chunk's copy into shared memory never completed"},
 }
 for _capped in ("attention_prefill_tc", "attention_decode"):
     _STATUS_MEANING[_capped + "_capped"] = _STATUS_MEANING[_capped]
@@ -1264,7 +1265,7 @@ def qk_row_norm(proj, q_out, k_cache, v_cache, block_table, ctx, q_gain, k_gain,
 
 
 DELTA_MAX_TAPS = 16        # the same constants as DR_MAX_TAPS, DR_CHUNK and DR_COEF in delta_rule.cu
-DELTA_CHUNK, DELTA_COEF = 8, 156
+DELTA_CHUNK, DELTA_COEF = 8, 120
 
 
 def _delta_args(proj, offsets, conv_w, taps, a_log, dt_bias, q_scale, unit_eps, state, ring_off, H, G, D, Dv):
@@ -1297,14 +1298,15 @@ def delta_prompt(proj, offsets, conv_w, taps: int, a_log, dt_bias, q_scale: floa
     pad4 = lambda n: (n + 3) // 4 * 4
     chunks = T // DELTA_CHUNK + ctx.n_seqs
     new = lambda n, what: guard.scratch((n,), torch.float32, out.device, what)
-    qk = new(chunks * G * 2 * DELTA_CHUNK * pad4(D), "prepared keys and queries of the delta rule")
+    row = next(n for n in (32, 64, 128, 256) if D <= n)         # floats of a prepared key or query
+    qk = new(chunks * G * 2 * DELTA_CHUNK * row, "prepared keys and queries of the delta rule")
     vv = new(chunks * H * DELTA_CHUNK * pad4(Dv), "prepared values of the delta rule")
     co = new(chunks * H * DELTA_COEF, "coefficients of the delta rule's chunks")
     f = _fn("delta_rule", "llmx_delta_prompt",
             _DELTA_ARGTYPES + [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                               c_int, c_int, c_int, c_void_p])
+                               c_int, c_int, c_int, c_int, c_void_p])
     _check(f(*args, _ptr(qk), _ptr(vv), _ptr(co), _ptr(out), _ptr(ctx.seq_start), _ptr(ctx.seq_past), _ptr(ctx.seq_slot),
-             T, ctx.n_seqs, H, G, D, Dv, _stream()), "delta_prompt")
+             T, ctx.n_seqs, H, G, D, Dv, n_sm(out.device), _stream()), "delta_prompt")
     global launch_count
     launch_count += 2 if taps > 1 else 1          # beside the preparation: the recurrence, and the convolution's rows
 
