@@ -226,10 +226,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       tmem_ld_wait();
 #if LLMX_SCORE_CAP
 #pragma unroll
-      for (int e = 0; e < AT_KEYS; ++e) {       // (as capped_score_log2, with the one-instruction exponential)
-        const float ex = ex2_approx(cap.mul * __uint_as_float(sr[e]));
-        sr[e] = __float_as_uint(cap.top - __fdividef(2.0f * cap.top, 1.0f + ex));
-      }
+      for (int e = 0; e < AT_KEYS; ++e) sr[e] = __float_as_uint(capped_score_log2(cap, __uint_as_float(sr[e])));
 #endif
       // Tiles that some row of this CTA sees only in part (the diagonal, a window's edge, rows past the
       // sequence's end) are masked; the others, which is most of them, skip the compares.

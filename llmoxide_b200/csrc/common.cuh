@@ -198,7 +198,7 @@ template <> __device__ __forceinline__ bf16 from_f32<bf16>(float x) { return __f
 // Capped attention scores.  The tiled attention kernels are compiled twice, with LLMX_SCORE_CAP 0 and 1; the second
 // library caps every scaled score s at c: c * tanh(s / c).  They keep scores in base-2 logarithms, where that is
 // top * tanh(z) = top - 2 top / (1 + 2^(mul * raw)) for the unscaled product `raw`, top = c log2(e) and
-// mul = 2 log2(e) scale / c: one exponential and one division, off by a few 1e-7 of top.  A product that overflows
+// mul = 2 log2(e) scale / c: one exponential and one reciprocal, off by a few 1e-7 of top.  A product that overflows
 // the exponential gives the limits +-top.
 #ifndef LLMX_SCORE_CAP
 #define LLMX_SCORE_CAP 0
@@ -207,7 +207,10 @@ struct ScoreCap {
   float mul, top;
 };
 __device__ __forceinline__ float capped_score_log2(const ScoreCap c, float raw) {
-  return c.top - __fdividef(2.0f * c.top, 1.0f + exp2f(c.mul * raw));
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(c.mul * raw));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return fmaf(-2.0f * c.top, r, c.top);
 }
 static inline ScoreCap make_score_cap(float scale, float softcap) {
   ScoreCap c = {0.f, 0.f};
@@ -275,6 +278,23 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   __syncthreads();
   float t = (lane < n_warps) ? scratch[lane] : 0.f;
   return warp_sum(t);
+}
+
+// Element `at` of a product's output: one tensor, or n_split partials `stride` elements apart, added in order.  The
+// first eight are asked for together.
+template <typename T>
+__device__ __forceinline__ float split_value(const T* p, size_t at, int n_split, size_t stride) {
+  float v = to_f32(p[at]);
+  if (n_split > 1) {
+    float t[7];
+#pragma unroll
+    for (int s = 0; s < 7; ++s) t[s] = s + 1 < n_split ? to_f32(p[at + (size_t)(s + 1) * stride]) : 0.f;
+#pragma unroll
+    for (int s = 0; s < 7; ++s)
+      if (s + 1 < n_split) v += t[s];
+    for (int s = 8; s < n_split; ++s) v += to_f32(p[at + (size_t)s * stride]);
+  }
+  return v;
 }
 
 // Element offset of (physical page, kv head, row in page, dim 0) in one cache

@@ -54,9 +54,7 @@ __device__ __forceinline__ float dr_softplus(float x) { return fmaxf(x, 0.f) + l
 // value of column c of a row: one tensor, or split partials added in order
 template <typename TIN>
 __device__ __forceinline__ float dr_value(const TIN* row, int c, int n_split, size_t split_stride) {
-  float v = to_f32(row[c]);
-  for (int s = 1; s < n_split; ++s) v += to_f32(row[s * split_stride + c]);
-  return v;
+  return split_value(row, c, n_split, split_stride);
 }
 
 struct DeltaIn {
@@ -541,17 +539,28 @@ delta_decode_kernel(const TIN* __restrict__ proj, const DeltaIn in, float* __res
     }
   };
   load_tile(lane * V);
+  // ... then what the end needs of the projection, and the head's gates
+  float z_own = 0.f;
+  if (tid < Dv) z_own = dr_value(row, in.g_off + h * Dv + tid, in.n_split, in.split_stride);
+  if (tid == 255) {
+    sums[3] = dr_sigmoid(dr_value(row, in.b_off + h, in.n_split, in.split_stride));
+    const float a = dr_value(row, in.a_off + h, in.n_split, in.split_stride);
+    sums[4] = expf(-expf(in.a_log[h]) * dr_softplus(a + in.dt_bias[h]));
+  }
   // ---- convolution, activation; the token's projected row joins the ring
+  const int p_place = p % taps;
   for (int e = tid; e < 2 * D + Dv; e += 256) {
     const int c = e < D ? j * D + e : e < 2 * D ? G * D + j * D + (e - D) : 2 * G * D + h * Dv + (e - 2 * D);
     const float own = dr_value(row, dr_column(in, c), in.n_split, in.split_stride);
     float acc = 0.f;
+    int place = p_place;                                  // the row of position p - taps + 1: the one behind p's
+#pragma unroll 4
     for (int m = 0; m < taps; ++m) {
-      const int pp = p - taps + 1 + m;
-      const float u = m == taps - 1 ? own : pp >= 0 ? ring[(size_t)(pp % taps) * C + c] : 0.f;
+      place = place + 1 == taps ? 0 : place + 1;
+      const float u = m == taps - 1 ? own : p - taps + 1 + m >= 0 ? ring[(size_t)place * C + c] : 0.f;
       acc = fmaf(in.conv_w[(size_t)m * C + c], u, acc);
     }
-    if (taps > 1) ring[(size_t)(p % taps) * C + c] = own;      // (heads that share a key head write the same number)
+    if (taps > 1) ring[(size_t)p_place * C + c] = own;      // (heads that share a key head write the same number)
     acc = dr_silu(acc);
     if (e < D) sq[e] = acc;
     else if (e < 2 * D) sk[e - D] = acc;
@@ -565,10 +574,6 @@ delta_decode_kernel(const TIN* __restrict__ proj, const DeltaIn in, float* __res
     for (int d = lane; d < D; d += 32) ss += x[d] * z[d];
     ss = warp_sum(ss);
     if (lane == 0) sums[warp] = ss;
-  } else if (warp == 3 && lane == 0) {
-    sums[3] = dr_sigmoid(dr_value(row, in.b_off + h, in.n_split, in.split_stride));
-    const float a = dr_value(row, in.a_off + h, in.n_split, in.split_stride);
-    sums[4] = expf(-expf(in.a_log[h]) * dr_softplus(a + in.dt_bias[h]));
   }
   __syncthreads();
   const float fq = in.q_scale / sqrtf(sums[0] + in.unit_eps), fk = 1.f / sqrtf(sums[1] + in.unit_eps);
@@ -644,7 +649,7 @@ delta_decode_kernel(const TIN* __restrict__ proj, const DeltaIn in, float* __res
   // ---- the head's norm and gate
   const float rstd = 1.0f / sqrtf(block_sum(ss_o, red) / (float)Dv + eps);
   for (int c = tid; c < Dv; c += 256) {
-    const float z = dr_value(row, in.g_off + h * Dv + c, in.n_split, in.split_stride);
+    const float z = c == tid ? z_own : dr_value(row, in.g_off + h * Dv + c, in.n_split, in.split_stride);
     y[((size_t)b * H + h) * Dv + c] = from_f32<TO>(((so[c] * rstd) * gain[c]) * dr_silu(z));
   }
 }

@@ -17,19 +17,18 @@
 //
 // Scores, statistics, rotations and norms are float32; bfloat16 is rounded to only where something is stored or is an
 // operand of a tensor-core product.
-#include "common.cuh"
+#include "tc_ptx.cuh"
 
 #define LC_TILE 32           // cached rows per tile of latent_decode
 #define LC_HEADS 16          // heads per CTA
 #define LC_WARPS 4
+#define LC_PREP_HEADS 4      // query heads per CTA of latent_prep
 #define LC_MAX_RANK 512      // latent_decode; latent_paged takes up to LC_MAX_RANK_GENERAL
 #define LC_MAX_RANK_GENERAL 1024
 
 template <typename T>
 __device__ __forceinline__ float lc_value(const T* p, int n_split, size_t split_stride) {
-  float v = to_f32(p[0]);
-  for (int s = 1; s < n_split; ++s) v += to_f32(p[(size_t)s * split_stride]);
-  return v;
+  return split_value(p, 0, n_split, split_stride);
 }
 
 // Where token t lives: false (and a report) when the step's arrays do not fit the launch.
@@ -41,7 +40,7 @@ __device__ __forceinline__ bool lc_page(const int* block_table, int table_width,
 }
 
 // ---------------------------------------------------------------------------
-// One CTA per token.  down: [T, down_stride] with the latent at column 0 and the shared key part at column rank (float32
+// CTA (t, 0) does the token's latent and its cache row, CTA (t, y > 0) LC_PREP_HEADS query heads.  down: [T, down_stride] with the latent at column 0 and the shared key part at column rank (float32
 // or float32 partials); q: [T, q_stride], every head [ R rotated | D plain ].  Pairs (i, i + R/2) turn by the
 // position's angles.  q goes to rot_out[(t H + h) rot_ld + 0..R-1] and plain_out[(t H + h) plain_ld + 0..D-1].
 // ---------------------------------------------------------------------------
@@ -67,11 +66,11 @@ latent_prep_kernel(const TIN* __restrict__ down, int n_split, size_t split_strid
   const float* sn = sin_t + (size_t)pos * half;
   pdl_wait();
   const TIN* row = down + (size_t)t * down_stride;
+  if (blockIdx.y > 0) {
   const TQ* qrow = q + (size_t)t * q_stride;
-  // the query first: its loads do not wait for the latent's sum
-  const int heads_rot = H * half, E = R + D;
-  for (int e = threadIdx.x; e < heads_rot; e += blockDim.x) {
-    const int h = e / half, i = e - h * half;
+  const int h_lo = (blockIdx.y - 1) * LC_PREP_HEADS, n_h = min(LC_PREP_HEADS, H - h_lo), E = R + D;
+  for (int e = threadIdx.x; e < n_h * half; e += blockDim.x) {
+    const int h = h_lo + e / half, i = e % half;
     const float c = cs[i], s = sn[i];
     const float x = lc_value(qrow + (size_t)h * E + i, q_split, q_split_stride);
     const float y = lc_value(qrow + (size_t)h * E + i + half, q_split, q_split_stride);
@@ -79,9 +78,11 @@ latent_prep_kernel(const TIN* __restrict__ down, int n_split, size_t split_strid
     dst[0] = from_f32<TR>(x * c - y * s);
     dst[half] = from_f32<TR>(y * c + x * s);
   }
-  for (int e = threadIdx.x; e < H * D; e += blockDim.x) {
-    const int h = e / D, i = e - h * D;
+  for (int e = threadIdx.x; e < n_h * D; e += blockDim.x) {
+    const int h = h_lo + e / D, i = e % D;
     plain_out[((size_t)t * H + h) * plain_ld + i] = from_f32<TP>(lc_value(qrow + (size_t)h * E + R + i, q_split, q_split_stride));
+  }
+  return;
   }
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
@@ -114,8 +115,9 @@ LLMX_API int llmx_latent_prep(const void* down, int in_dtype, int n_split, long 
   if (!cos_t || !sin_t || !gain) return LLMX_REFUSED(4);
   const size_t smem = (size_t)rank * sizeof(float);
   if (smem > 48 * 1024) return LLMX_REFUSED(3);
+  const dim3 prep_grid(n_tokens, 1 + (H + LC_PREP_HEADS - 1) / LC_PREP_HEADS);
 #define CASE(TQ, TO, TC)                                                                                                 \
-  launch_pdl(latent_prep_kernel<float, TQ, TO, TO, TC>, dim3(n_tokens), dim3(256), smem, stream, (const float*)down,     \
+  launch_pdl(latent_prep_kernel<float, TQ, TO, TO, TC>, prep_grid, dim3(256), smem, stream, (const float*)down,            \
              n_split, (size_t)split_stride, (size_t)down_stride, (const TQ*)q, q_split, (size_t)q_split_stride,          \
              (size_t)q_stride, gain, eps, (TC*)cache, (TO*)rot_out, (size_t)rot_ld, (TO*)plain_out, (size_t)plain_ld,    \
              block_table, table_width, token_seq, token_pos, cos_t, sin_t, H, D, R, rank, n_seqs, (int)n_pages)
@@ -341,13 +343,16 @@ LLMX_API int llmx_latent_paged(const float* q, float* lat, const void* cache, in
 // ---------------------------------------------------------------------------
 // Absorbed attention on the tensor cores.  grid (shares, ceil(H / 16), tokens), 4 warps.  A CTA owns one token, 16 heads
 // (the 16-wide M axis of mma.sync m16n8k16) and one share of the token's cached rows, which it walks in tiles of 32
-// through a ring of shared-memory stages filled by cp.async (rows padded by 16 bytes: ldmatrix without conflicts).
+// through a ring of shared-memory stages; a tile comes as one bulk copy per row, asked for by the lanes of warp 0 (rows
+// padded by 16 bytes in shared memory: ldmatrix without conflicts).
 //   S = Q C^T     warp w: rows 8 w .. 8 w + 7 of the tile, all rank + R dims
 //   O += P C      the warps share the latent's 16-dim blocks (block i belongs to warp i % 4), all 32 rows
 // Maximum and probabilities pass between the warps through shared memory.
 // ---------------------------------------------------------------------------
-__device__ __forceinline__ void lc_cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+__device__ __forceinline__ void lc_bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
+               "l"(src), "r"(bytes), "r"(bar)
+               : "memory");
 }
 __device__ __forceinline__ void lc_ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -376,6 +381,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
                      int n_seqs, int n_pages) {
   extern __shared__ __align__(128) uint8_t lc_smem[];
   __shared__ float s_max[LC_WARPS][LC_HEADS], s_sum[LC_WARPS][LC_HEADS];
+  __shared__ __align__(8) uint64_t lc_bars[STAGES + 1];              // one a stage, then the query's
   pdl_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, tq = lane & 3;
   const int chunk = blockIdx.x, h0 = blockIdx.y * LC_HEADS, t = blockIdx.z;
@@ -393,43 +399,45 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
   uint8_t* pT = lc_smem + LC_HEADS * (row_bytes + LC_P_ROW);
   const int n_all = p / LC_TILE + 1, per = (n_all + n_chunks - 1) / n_chunks;
   const int lo = chunk * per, n_tiles = min(per, n_all - lo);           // <= 0: nothing to do
-  auto load_tile = [&](int i) {
-    const int key0 = (lo + i) * LC_TILE, st = i % STAGES;
-    int page = pages[key0 / LLMX_PAGE];                                  // (a tile lies within one page)
-    if (page < 0 || page >= n_pages) {
-      if (tid == 0) llmx_report(2);
-      page = 0;
+  const uint32_t bars = smem_u32(lc_bars), copy_bytes = (uint32_t)E * 2u;
+  if (tid == 0) {
+    for (int i = 0; i <= STAGES; ++i) mbar_init(bars + 8 * i, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
+  int next_page = 0;                                   // of the tile that load_tile is called for next (warp 0)
+  if (warp == 0 && n_tiles > 0) next_page = pages[lo * LC_TILE / LLMX_PAGE];
+  auto load_tile = [&](int i) {                        // every thread
+    const int key0 = (lo + i) * LC_TILE, st = i % STAGES, valid = min(LC_TILE, p - key0 + 1);
+    if (warp == 0) {
+      int page = next_page;                                              // (a tile lies within one page)
+      if (i + 1 < n_tiles) next_page = pages[(key0 + LC_TILE) / LLMX_PAGE];
+      if (page < 0 || page >= n_pages) {
+        if (lane == 0) llmx_report(2);
+        page = 0;
+      }
+      const bf16* src = cache + cache_row_offset(page, 0, key0 % LLMX_PAGE, 1, E);
+      if (lane == 0) mbar_expect_tx(bars + 8 * st, (uint32_t)valid * copy_bytes);
+      __syncwarp();
+      if (lane < valid)
+        lc_bulk_copy(sT + (uint32_t)(st * tile_bytes + lane * row_bytes), src + (size_t)lane * E, copy_bytes, bars + 8 * st);
     }
-    const bf16* src = cache + cache_row_offset(page, 0, key0 % LLMX_PAGE, 1, E);
-    for (int e = tid; e < LC_TILE * pieces; e += LC_WARPS * 32) {
-      const int r = e / pieces, c = e - r * pieces;
-      const uint32_t off = (uint32_t)(st * tile_bytes + r * row_bytes + c * 16);
-      // rows past the token's own were never written by it (or belong to nobody): weight 0, but 0 * NaN is NaN
-      if (key0 + r <= p) lc_cp_async16(sT + off, src + (size_t)r * E + c * 8);
-      else *reinterpret_cast<uint4*>(pT + off) = make_uint4(0u, 0u, 0u, 0u);
-    }
+    // rows past the token's own were never written by it (or belong to nobody): weight 0, but 0 * NaN is NaN
+    for (int r = valid + warp; r < LC_TILE; r += LC_WARPS)
+      for (int c = lane; c < pieces; c += 32)
+        *reinterpret_cast<uint4*>(pT + st * tile_bytes + r * row_bytes + c * 16) = make_uint4(0u, 0u, 0u, 0u);
   };
   // Tiles wholly of earlier steps are complete: they start before the kernel ahead has ended.
   int issued = 0;
-  for (; issued < STAGES - 1 && issued < n_tiles && (lo + issued + 1) * LC_TILE <= past; ++issued) {
-    load_tile(issued);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  }
+  for (; issued < STAGES - 1 && issued < n_tiles && (lo + issued + 1) * LC_TILE <= past; ++issued) load_tile(issued);
   pdl_wait();
-  // the query tile, rows of missing heads zero; it joins the group committed next
-  for (int e = tid; e < LC_HEADS * pieces; e += LC_WARPS * 32) {
-    const int r = e / pieces, c = e - r * pieces;
-    if (r < n_heads) lc_cp_async16(sQ + r * row_bytes + c * 16, q + ((size_t)t * H + h0 + r) * E + c * 8);
-    else *reinterpret_cast<uint4*>(lc_smem + r * row_bytes + c * 16) = make_uint4(0u, 0u, 0u, 0u);
+  if (warp == 1 && n_tiles > 0) {      // the query tile; rows of missing heads hold anything and are not stored
+    if (lane == 0) mbar_expect_tx(bars + 8 * STAGES, (uint32_t)n_heads * copy_bytes);
+    __syncwarp();
+    if (lane < n_heads)
+      lc_bulk_copy(sQ + (uint32_t)(lane * row_bytes), q + ((size_t)t * H + h0 + lane) * E, copy_bytes, bars + 8 * STAGES);
   }
-  if (issued > 0) {                    // the query's copies behind a tile's would upset the count below: wait for all
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-  }
-  for (; issued < STAGES - 1; ++issued) {
-    if (issued < n_tiles) load_tile(issued);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  }
+  for (; issued < STAGES - 1 && issued < n_tiles; ++issued) load_tile(issued);
 
   const int n_blocks = rank / 16;
   float o[NB][2][4];
@@ -441,37 +449,66 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
   const int ksteps = E / 16;
   const uint32_t q_addr = sQ + (uint32_t)((lane & 15) * row_bytes + (lane >> 4) * 16);
   for (int i = 0; i < n_tiles; ++i) {
+    // the tile has landed (and, first, the query); everyone has left the tile before, whose stage the next copy fills
+    bool ok = i > 0 || mbar_wait(bars + 8 * STAGES, 0);
+    ok = ok && mbar_wait(bars + 8 * (i % STAGES), (i / STAGES) & 1);
+    if (!__syncthreads_and(ok)) {
+      if (tid == 0) llmx_report(4);
+      break;
+    }
     if (i + STAGES - 1 < n_tiles) load_tile(i + STAGES - 1);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 1) : "memory");
-    __syncthreads();
     const uint32_t tile = sT + (uint32_t)((i % STAGES) * tile_bytes);
     const int key0 = (lo + i) * LC_TILE;
-    // ---- scores of this warp's 8 rows: two chains, even and odd 16-dim steps
-    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    // ---- scores of this warp's 8 rows: four chains of 16-dim steps
+    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f}, s3[4] = {0.f, 0.f, 0.f, 0.f};
     const uint32_t k_addr = tile + (uint32_t)((warp * 8 + (lane & 7)) * row_bytes + (lane >> 3) * 16);
-    int ks = 0;
-#pragma unroll 4
-    for (; ks + 2 <= ksteps; ks += 2) {
-      uint32_t b0, b1, b2, b3, a0, a1, a2, a3;
-      lc_ldmatrix_x4(k_addr + ks * 32, b0, b1, b2, b3);
-      lc_ldmatrix_x4(q_addr + ks * 32, a0, a1, a2, a3);
-      lc_mma(s0, a0, a1, a2, a3, b0, b1);
-      lc_ldmatrix_x4(q_addr + ks * 32 + 32, a0, a1, a2, a3);
-      lc_mma(s1, a0, a1, a2, a3, b2, b3);
+    // four steps' operands at a time, the next four asked for before these are multiplied
+    uint32_t kb[2][8], qa[2][16];
+    auto fetch = [&](int at, uint32_t* kf, uint32_t* qf) {
+      lc_ldmatrix_x4(k_addr + at * 32, kf[0], kf[1], kf[2], kf[3]);
+      lc_ldmatrix_x4(k_addr + at * 32 + 64, kf[4], kf[5], kf[6], kf[7]);
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        lc_ldmatrix_x4(q_addr + (at + x) * 32, qf[4 * x], qf[4 * x + 1], qf[4 * x + 2], qf[4 * x + 3]);
+    };
+    auto multiply = [&](const uint32_t* kf, const uint32_t* qf) {
+      lc_mma(s0, qf[0], qf[1], qf[2], qf[3], kf[0], kf[1]);
+      lc_mma(s1, qf[4], qf[5], qf[6], qf[7], kf[2], kf[3]);
+      lc_mma(s2, qf[8], qf[9], qf[10], qf[11], kf[4], kf[5]);
+      lc_mma(s3, qf[12], qf[13], qf[14], qf[15], kf[6], kf[7]);
+    };
+    const int quads = ksteps >> 2;
+    if (quads > 0) fetch(0, kb[0], qa[0]);
+    int g4 = 0;
+    for (; g4 + 2 <= quads; g4 += 2) {
+      fetch(4 * g4 + 4, kb[1], qa[1]);
+      multiply(kb[0], qa[0]);
+      if (g4 + 2 < quads) fetch(4 * g4 + 8, kb[0], qa[0]);
+      multiply(kb[1], qa[1]);
     }
-    if (ks < ksteps) {
+    if (g4 < quads) multiply(kb[0], qa[0]);
+    for (int ks = quads * 4; ks < ksteps; ++ks) {
       uint32_t b0, b1, a0, a1, a2, a3;
       lc_ldmatrix_x2(tile + (uint32_t)((warp * 8 + (lane & 7)) * row_bytes + ((lane >> 3) & 1) * 16) + ks * 32, b0, b1);
       lc_ldmatrix_x4(q_addr + ks * 32, a0, a1, a2, a3);
       lc_mma(s0, a0, a1, a2, a3, b0, b1);
     }
+    // the first block's latents for the second product, ahead of the probabilities
+    uint32_t vb[2][8];
+    auto fetch_v = [&](int blk, uint32_t* vf) {
+      // transposed: (rows 0-7, dims lo), (rows 8-15, dims lo), (rows 0-7, dims hi), (rows 8-15, dims hi)
+#pragma unroll
+      for (int kk = 0; kk < 2; ++kk)
+        lc_ldmatrix_x4_trans(tile + (uint32_t)((kk * 16 + (lane & 15)) * row_bytes + blk * 32 + (lane >> 4) * 16), vf[4 * kk],
+                             vf[4 * kk + 1], vf[4 * kk + 2], vf[4 * kk + 3]);
+    };
+    if (warp < n_blocks) fetch_v(warp, vb[0]);
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const bool vis = key0 + warp * 8 + 2 * tq + e <= p;
-      s0[e] = vis ? (s0[e] + s1[e]) * scale_log2 : -INFINITY;
-      s0[2 + e] = vis ? (s0[2 + e] + s1[2 + e]) * scale_log2 : -INFINITY;
+      s0[e] = vis ? ((s0[e] + s1[e]) + (s2[e] + s3[e])) * scale_log2 : -INFINITY;
+      s0[2 + e] = vis ? ((s0[2 + e] + s1[2 + e]) + (s2[2 + e] + s3[2 + e])) * scale_log2 : -INFINITY;
       mx0 = fmaxf(mx0, s0[e]);
       mx1 = fmaxf(mx1, s0[2 + e]);
     }
@@ -486,11 +523,13 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     for (int w = 0; w < LC_WARPS; ++w) mx0 = fmaxf(mx0, s_max[w][gq]), mx1 = fmaxf(mx1, s_max[w][gq + 8]);
     mx0 = fmaxf(mx0, m0);                              // a tile's first row is always seen
     mx1 = fmaxf(mx1, m1);
-    const float c0 = exp2f(m0 - mx0), c1 = exp2f(m1 - mx1);
+    const float c0 = ex2_approx(m0 - mx0), c1 = ex2_approx(m1 - mx1);
+    const bool rescale = __any_sync(0xffffffffu, mx0 != m0 || mx1 != m1);      // some maximum has grown
     m0 = mx0;
     m1 = mx1;
     {
-      const float e0 = exp2f(s0[0] - mx0), e1 = exp2f(s0[1] - mx0), e2 = exp2f(s0[2] - mx1), e3 = exp2f(s0[3] - mx1);
+      const float e0 = ex2_approx(s0[0] - mx0), e1 = ex2_approx(s0[1] - mx0);
+      const float e2 = ex2_approx(s0[2] - mx1), e3 = ex2_approx(s0[3] - mx1);
       l0 = l0 * c0 + (e0 + e1);
       l1 = l1 * c1 + (e2 + e3);
       __nv_bfloat162 pa = __floats2bfloat162_rn(e0, e1), pb = __floats2bfloat162_rn(e2, e3);
@@ -509,22 +548,21 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     for (int nb = 0; nb < NB; ++nb) {
       const int blk = warp + LC_WARPS * nb;
       if (blk < n_blocks) {
+        if (nb + 1 < NB && blk + LC_WARPS < n_blocks) fetch_v(blk + LC_WARPS, vb[(nb + 1) & 1]);
+        const uint32_t* vf = vb[nb & 1];
+        if (rescale) {
 #pragma unroll
-        for (int j = 0; j < 2; ++j) o[nb][j][0] *= c0, o[nb][j][1] *= c0, o[nb][j][2] *= c1, o[nb][j][3] *= c1;
+          for (int j = 0; j < 2; ++j) o[nb][j][0] *= c0, o[nb][j][1] *= c0, o[nb][j][2] *= c1, o[nb][j][3] *= c1;
+        }
 #pragma unroll
         for (int kk = 0; kk < 2; ++kk) {
-          uint32_t b0, b1, b2, b3;
-          // transposed: (rows 0-7, dims lo), (rows 8-15, dims lo), (rows 0-7, dims hi), (rows 8-15, dims hi)
-          lc_ldmatrix_x4_trans(tile + (uint32_t)((kk * 16 + (lane & 15)) * row_bytes + blk * 32 + (lane >> 4) * 16), b0, b1,
-                               b2, b3);
-          lc_mma(o[nb][0], pf[kk][0], pf[kk][1], pf[kk][2], pf[kk][3], b0, b1);
-          lc_mma(o[nb][1], pf[kk][0], pf[kk][1], pf[kk][2], pf[kk][3], b2, b3);
+          lc_mma(o[nb][0], pf[kk][0], pf[kk][1], pf[kk][2], pf[kk][3], vf[4 * kk], vf[4 * kk + 1]);
+          lc_mma(o[nb][1], pf[kk][0], pf[kk][1], pf[kk][2], pf[kk][3], vf[4 * kk + 2], vf[4 * kk + 3]);
         }
       }
     }
-    __syncthreads();                                   // the stage, the maxima and P are written again
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
   // ---- the sums of the four warps' rows
 #pragma unroll
   for (int sh = 1; sh < 4; sh <<= 1) {
@@ -560,11 +598,10 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     return;
   }
   const size_t u0 = ((size_t)t * H + h0 + gq) * n_chunks + chunk, u1 = ((size_t)t * H + h0 + gq + 8) * n_chunks + chunk;
-  if (warp == 0 && tq == 0) {                          // (a share without rows: maximum -inf, sum 0)
+  if (warp == 0 && tq == 0) {                          // (a share without rows: maximum -inf, sum 0, sums of latents 0)
     if (live0) part_ml[2 * u0] = m0, part_ml[2 * u0 + 1] = l0;
     if (live1) part_ml[2 * u1] = m1, part_ml[2 * u1 + 1] = l1;
   }
-  if (n_tiles <= 0) return;
 #pragma unroll
   for (int nb = 0; nb < NB; ++nb) {
     const int blk = warp + LC_WARPS * nb;
@@ -602,18 +639,21 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
     if (threadIdx.x == 0) inv = 1.0f / l;
   }
   __syncthreads();
-  for (int d = threadIdx.x * 2; d < rank; d += 256) {
-    float a = 0.f, b = 0.f;
+  for (int d = threadIdx.x * 4; d < rank; d += 512) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float* src = part_o + u * rank + d;
 #pragma unroll 8
     for (int c = 0; c < n_chunks; ++c) {
       const float f = fac[c];
-      if (f != 0.f) {                                  // an unused share's row may hold anything
-        const float2 v = *reinterpret_cast<const float2*>(part_o + (u + c) * rank + d);
-        a = fmaf(f, v.x, a);
-        b = fmaf(f, v.y, b);
-      }
+      const float4 v = *reinterpret_cast<const float4*>(src + (size_t)c * rank);
+      a.x = fmaf(f, v.x, a.x);
+      a.y = fmaf(f, v.y, a.y);
+      a.z = fmaf(f, v.z, a.z);
+      a.w = fmaf(f, v.w, a.w);
     }
-    *reinterpret_cast<__nv_bfloat162*>(lat + ((size_t)t * H + h) * rank + d) = __floats2bfloat162_rn(a * inv, b * inv);
+    __nv_bfloat162 lo = __floats2bfloat162_rn(a.x * inv, a.y * inv), hi = __floats2bfloat162_rn(a.z * inv, a.w * inv);
+    *reinterpret_cast<uint2*>(lat + ((size_t)t * H + h) * rank + d) =
+        make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
   }
 }
 

@@ -147,7 +147,8 @@ _STATUS_MEANING = {
     "latent_attention": {1: "a token's sequence, position or page lies outside the launch's arrays"},
     "latent_cache": {1: "a token's sequence, position or page lies outside the launch's arrays",
                      2: "a token's sequence, position or page lies outside the launch's arrays (absorbed attention)",
-                     3: "a scratch page stands for no page of the step's sequences"},
+                     3: "a scratch page stands for no page of the step's sequences",
+                     4: "a copy into shared memory never completed (absorbed attention)"},
     "qk_row_norm": {1: "a token's sequence, position or page lies outside the launch's arrays"},
     "delta_rule": {1: "a sequence's rows or slot lie outside the launch's arrays (preparation)",
                    2: "a sequence's slot lies outside the state area",
