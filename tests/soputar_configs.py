@@ -42,13 +42,13 @@ SP_A = dict(
         _attention(6, 2, 32, 16, 0.5, 6.0, (0.2, 20), None, kv_from=1),
     ])
 # A width that is no multiple of eight (every product on the FMA units), one tap (no convolution beyond the current
-# token), values wider than keys, no cap, no temperature, a single delta head, an odd head size.
+# token), values wider than keys, no cap, no temperature, six delta heads on three key heads, an odd head size.
 SP_B = dict(
     architecture="Soputar", vocab=300, width=100, norm=dict(eps=1e-6), embedding=dict(scale=0.5),
     layers=[
         _latent(5, 20, 12, 12, 28, 0.3, 50000.0, 36),
         _attention(6, 3, 16, 48, 0.25, None, None, 44, limit=10.0),
-        _delta(1, 1, 30, 41, 1, None),
+        _delta(6, 3, 30, 41, 1, None),
         _attention(3, 3, 48, 40, 0.15, 1.0, (0.9, 1), 30),
     ])
 # The sizes the tiled kernels like (64 and 128): capped and plain scores, one kv head, borrowed keys, assembled latent
