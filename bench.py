@@ -742,15 +742,24 @@ def _design_models(args, models, vocab, T, B, depth, rng) -> dict:
         for i in range(W):
             eng.step([(sl, [t]) for sl, t in zip(slots, toks[i])])
         launches = kernels.launch_count
-        dec_ms = event_ms(lambda: [eng.step([(sl, [t]) for sl, t in zip(slots, toks[i])]) for i in range(W, W + K)]) / K
+        marks = [torch.cuda.Event(enable_timing=True) for _ in range(K + 1)]
+
+        def decode_steps():
+            marks[0].record()
+            for i in range(K):
+                eng.step([(sl, [t]) for sl, t in zip(slots, toks[W + i])])
+                marks[i + 1].record()
+
+        dec_ms = event_ms(decode_steps) / K
+        dec_median = statistics.median(marks[i].elapsed_time(marks[i + 1]) for i in range(K))
         launches = (kernels.launch_count - launches) // K
         dec_kernels = per_kernel(eng, [(sl, [t]) for sl, t in zip(slots, toks[W + K])])
         eng.check_status()
         result[name] = dict(prefill_tokens=T, prefill_ms=round(pre_ms, 3), prefill_tokens_per_s=round(T / pre_ms * 1e3),
-                            decode_batch=B, decode_depth=depth, decode_ms_per_step=round(dec_ms, 4),
+                            decode_batch=B, decode_depth=depth, decode_ms_per_step=round(dec_ms, 4), decode_ms_median_step=round(dec_median, 4),
                             decode_tokens_per_s=round(B / dec_ms * 1e3), launches_per_decode_step=launches,
                             prefill_kernels=pre_kernels, decode_kernels=dec_kernels)
-        print(f"[bench] {name}: prefill {T} tokens {pre_ms:.2f} ms, decode b{B} {dec_ms:.3f} ms/step", file=sys.stderr)
+        print(f"[bench] {name}: prefill {T} tokens {pre_ms:.2f} ms, decode b{B} {dec_ms:.3f} ms/step (median step {dec_median:.3f})", file=sys.stderr)
         del eng
         torch.cuda.empty_cache()
     return result

@@ -23,6 +23,7 @@
 #define LC_HEADS 16          // heads per CTA
 #define LC_WARPS 4
 #define LC_PREP_HEADS 4      // query heads per CTA of latent_prep
+#define LC_MAX_CHUNKS 128    // shares of one token's rows
 #define LC_MAX_RANK 512      // latent_decode; latent_paged takes up to LC_MAX_RANK_GENERAL
 #define LC_MAX_RANK_GENERAL 1024
 
@@ -154,7 +155,7 @@ head_product_mma_kernel(const bf16* __restrict__ x, size_t x_ld, const bf16* __r
                         size_t y_ld, int T, int H, int N, int K) {
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gq = lane >> 2, tq = lane & 3;
-  const int h = blockIdx.y, n0 = (blockIdx.x * 4 + warp) * 16, t0 = blockIdx.z * 8 * TN;
+  const int h = blockIdx.y, n0 = (blockIdx.x * (blockDim.x >> 5) + warp) * 16, t0 = blockIdx.z * 8 * TN;
   if (n0 >= N) return;
   const bf16* wlo = w + ((size_t)h * N + n0 + gq) * K;
   const bf16* whi = wlo + (size_t)8 * K;
@@ -172,7 +173,7 @@ head_product_mma_kernel(const bf16* __restrict__ x, size_t x_ld, const bf16* __r
   }
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   pdl_wait();
-#pragma unroll 4
+#pragma unroll(TN == 1 ? 8 : 4)
   for (int k0 = 0; k0 < K; k0 += 32) {
     const int k = k0 + 8 * tq;
     const bool in = k < K;                               // K is a multiple of 8
@@ -223,10 +224,12 @@ LLMX_API int llmx_head_product(const void* x, int x_dtype, long long x_ld, const
   if (x_dtype == LLMX_BF16 && w_dtype == LLMX_BF16 && y_dtype == LLMX_BF16 && K % 8 == 0 && x_ld % 8 == 0 &&
       !(((uintptr_t)x | (uintptr_t)w) & 15)) {
     const int tn = n_tokens <= 8 ? 1 : n_tokens <= 16 ? 2 : 4;
-    const dim3 grid((N + 63) / 64, H, (n_tokens + 8 * tn - 1) / (8 * tn));
+    // warps per CTA: one while four would leave SMs without a CTA
+    const int warps = (long long)((N + 63) / 64) * H * ((n_tokens + 8 * tn - 1) / (8 * tn)) < 148 ? 1 : 4;
+    const dim3 grid((N + 16 * warps - 1) / (16 * warps), H, (n_tokens + 8 * tn - 1) / (8 * tn));
     if (grid.z > 65535) return LLMX_REFUSED(3);
 #define GO(TN)                                                                                                          \
-  launch_pdl(head_product_mma_kernel<TN>, grid, dim3(128), 0, stream, (const bf16*)x, (size_t)x_ld, (const bf16*)w,     \
+  launch_pdl(head_product_mma_kernel<TN>, grid, dim3(32 * warps), 0, stream, (const bf16*)x, (size_t)x_ld, (const bf16*)w,     \
              (bf16*)y, (size_t)y_ld, n_tokens, H, N, K)
     if (tn == 1) GO(1); else if (tn == 2) GO(2); else GO(4);
 #undef GO
@@ -341,10 +344,11 @@ LLMX_API int llmx_latent_paged(const float* q, float* lat, const void* cache, in
 }
 
 // ---------------------------------------------------------------------------
-// Absorbed attention on the tensor cores.  grid (shares, ceil(H / 16), tokens), 4 warps.  A CTA owns one token, 16 heads
+// Absorbed attention on the tensor cores.  grid (shares, ceil(H / 16), tokens), 4 warps and one that copies.  A CTA owns one token, 16 heads
 // (the 16-wide M axis of mma.sync m16n8k16) and one share of the token's cached rows, which it walks in tiles of 32
-// through a ring of shared-memory stages; a tile comes as one bulk copy per row, asked for by the lanes of warp 0 (rows
-// padded by 16 bytes in shared memory: ldmatrix without conflicts).
+// through a ring of shared-memory stages; a tile comes as one bulk copy per row, asked for by the fifth warp's lanes
+// (rows padded by 16 bytes in shared memory: ldmatrix without conflicts; asking takes half as long as multiplying, so it
+// is nobody else's work).
 //   S = Q C^T     warp w: rows 8 w .. 8 w + 7 of the tile, all rank + R dims
 //   O += P C      the warps share the latent's 16-dim blocks (block i belongs to warp i % 4), all 32 rows
 // Maximum and probabilities pass between the warps through shared memory.
@@ -369,11 +373,14 @@ __device__ __forceinline__ void lc_ldmatrix_x4_trans(uint32_t addr, uint32_t& r0
                : "r"(addr));
 }
 
+// A barrier of the four warps that multiply.
+__device__ __forceinline__ void lc_sync_warps() { asm volatile("bar.sync 1, %0;" ::"n"(LC_WARPS * 32) : "memory"); }
+
 #define LC_P_ROW (LC_TILE * 2 + 16)      // bytes of a row of probabilities
 
 // NB: 16-dim blocks of the latent per warp, at most; STAGES: tiles in shared memory
 template <int NB, int STAGES>
-__global__ void __launch_bounds__(LC_WARPS * 32)
+__global__ void __launch_bounds__(LC_WARPS * 32 + 32, 2)
 latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache, const int* __restrict__ block_table,
                      int table_width, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                      const int* __restrict__ seq_past, const float* __restrict__ sinks, float scale_log2, int H, int rank,
@@ -405,39 +412,45 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   __syncthreads();
-  int next_page = 0;                                   // of the tile that load_tile is called for next (warp 0)
-  if (warp == 0 && n_tiles > 0) next_page = pages[lo * LC_TILE / LLMX_PAGE];
-  auto load_tile = [&](int i) {                        // every thread
+  int next_page = 0;                                   // of the tile that load_tile is called for next
+  if (warp == LC_WARPS && n_tiles > 0) next_page = pages[lo * LC_TILE / LLMX_PAGE];
+  auto load_tile = [&](int i) {                        // the copying warp
     const int key0 = (lo + i) * LC_TILE, st = i % STAGES, valid = min(LC_TILE, p - key0 + 1);
-    if (warp == 0) {
-      int page = next_page;                                              // (a tile lies within one page)
-      if (i + 1 < n_tiles) next_page = pages[(key0 + LC_TILE) / LLMX_PAGE];
-      if (page < 0 || page >= n_pages) {
-        if (lane == 0) llmx_report(2);
-        page = 0;
-      }
-      const bf16* src = cache + cache_row_offset(page, 0, key0 % LLMX_PAGE, 1, E);
-      if (lane == 0) mbar_expect_tx(bars + 8 * st, (uint32_t)valid * copy_bytes);
-      __syncwarp();
-      if (lane < valid)
-        lc_bulk_copy(sT + (uint32_t)(st * tile_bytes + lane * row_bytes), src + (size_t)lane * E, copy_bytes, bars + 8 * st);
+    int page = next_page;                              // (a tile lies within one page)
+    if (i + 1 < n_tiles) next_page = pages[(key0 + LC_TILE) / LLMX_PAGE];
+    if (page < 0 || page >= n_pages) {
+      if (lane == 0) llmx_report(2);
+      page = 0;
     }
+    const bf16* src = cache + cache_row_offset(page, 0, key0 % LLMX_PAGE, 1, E);
+    if (lane == 0) mbar_expect_tx(bars + 8 * st, (uint32_t)valid * copy_bytes);
+    __syncwarp();
+    if (lane < valid)
+      lc_bulk_copy(sT + (uint32_t)(st * tile_bytes + lane * row_bytes), src + (size_t)lane * E, copy_bytes, bars + 8 * st);
     // rows past the token's own were never written by it (or belong to nobody): weight 0, but 0 * NaN is NaN
-    for (int r = valid + warp; r < LC_TILE; r += LC_WARPS)
+    for (int r = valid; r < LC_TILE; ++r)
       for (int c = lane; c < pieces; c += 32)
         *reinterpret_cast<uint4*>(pT + st * tile_bytes + r * row_bytes + c * 16) = make_uint4(0u, 0u, 0u, 0u);
   };
   // Tiles wholly of earlier steps are complete: they start before the kernel ahead has ended.
-  int issued = 0;
-  for (; issued < STAGES - 1 && issued < n_tiles && (lo + issued + 1) * LC_TILE <= past; ++issued) load_tile(issued);
-  pdl_wait();
-  if (warp == 1 && n_tiles > 0) {      // the query tile; rows of missing heads hold anything and are not stored
-    if (lane == 0) mbar_expect_tx(bars + 8 * STAGES, (uint32_t)n_heads * copy_bytes);
-    __syncwarp();
-    if (lane < n_heads)
-      lc_bulk_copy(sQ + (uint32_t)(lane * row_bytes), q + ((size_t)t * H + h0 + lane) * E, copy_bytes, bars + 8 * STAGES);
+  if (warp == LC_WARPS) {
+    int issued = 0;
+    for (; issued < STAGES - 1 && issued < n_tiles && (lo + issued + 1) * LC_TILE <= past; ++issued) load_tile(issued);
+    pdl_wait();
+    if (n_tiles > 0) {                 // the query tile; rows of missing heads hold anything and are not stored
+      if (lane == 0) mbar_expect_tx(bars + 8 * STAGES, (uint32_t)n_heads * copy_bytes);
+      __syncwarp();
+      if (lane < n_heads)
+        lc_bulk_copy(sQ + (uint32_t)(lane * row_bytes), q + ((size_t)t * H + h0 + lane) * E, copy_bytes, bars + 8 * STAGES);
+    }
+    for (; issued < STAGES - 1 && issued < n_tiles; ++issued) load_tile(issued);
+    for (int i = 0; i < n_tiles; ++i) {
+      if (!__syncthreads_and(1)) return;               // the tile before is done with: its stage takes the next one
+      if (i + STAGES - 1 < n_tiles) load_tile(i + STAGES - 1);
+    }
+    return;
   }
-  for (; issued < STAGES - 1 && issued < n_tiles; ++issued) load_tile(issued);
+  pdl_wait();
 
   const int n_blocks = rank / 16;
   float o[NB][2][4];
@@ -454,9 +467,8 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     ok = ok && mbar_wait(bars + 8 * (i % STAGES), (i / STAGES) & 1);
     if (!__syncthreads_and(ok)) {
       if (tid == 0) llmx_report(4);
-      break;
+      return;
     }
-    if (i + STAGES - 1 < n_tiles) load_tile(i + STAGES - 1);
     const uint32_t tile = sT + (uint32_t)((i % STAGES) * tile_bytes);
     const int key0 = (lo + i) * LC_TILE;
     // ---- scores of this warp's 8 rows: four chains of 16-dim steps
@@ -518,7 +530,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, sh));
     }
     if (tq == 0) s_max[warp][gq] = mx0, s_max[warp][gq + 8] = mx1;
-    __syncthreads();
+    lc_sync_warps();
 #pragma unroll
     for (int w = 0; w < LC_WARPS; ++w) mx0 = fmaxf(mx0, s_max[w][gq]), mx1 = fmaxf(mx1, s_max[w][gq + 8]);
     mx0 = fmaxf(mx0, m0);                              // a tile's first row is always seen
@@ -537,7 +549,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
       *reinterpret_cast<__nv_bfloat162*>(prow + gq * LC_P_ROW) = pa;
       *reinterpret_cast<__nv_bfloat162*>(prow + (gq + 8) * LC_P_ROW) = pb;
     }
-    __syncthreads();
+    lc_sync_warps();
     // ---- O = c O + P C
     uint32_t pf[2][4];
 #pragma unroll
@@ -562,7 +574,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
       }
     }
   }
-  __syncthreads();
+  lc_sync_warps();
   // ---- the sums of the four warps' rows
 #pragma unroll
   for (int sh = 1; sh < 4; sh <<= 1) {
@@ -570,7 +582,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     l1 += __shfl_xor_sync(0xffffffffu, l1, sh);
   }
   if (tq == 0) s_sum[warp][gq] = l0, s_sum[warp][gq + 8] = l1;
-  __syncthreads();
+  lc_sync_warps();
   l0 = (s_sum[0][gq] + s_sum[1][gq]) + (s_sum[2][gq] + s_sum[3][gq]);
   l1 = (s_sum[0][gq + 8] + s_sum[1][gq + 8]) + (s_sum[2][gq + 8] + s_sum[3][gq + 8]);
   const bool live0 = gq < n_heads, live1 = gq + 8 < n_heads;
@@ -619,7 +631,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                       const float* __restrict__ sinks, bf16* __restrict__ lat, int H, int rank, int n_chunks) {
-  __shared__ float fac[64];
+  __shared__ float fac[LC_MAX_CHUNKS];
   __shared__ float inv;
   pdl_launch_dependents();
   const int h = blockIdx.x, t = blockIdx.y;
@@ -658,14 +670,14 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
 }
 
 // q bf16 [T, H, rank + R] = [ absorbed | rotated ], cache bf16 [pages, 64, rank + R], lat bf16 [T, H, rank]; every token
-// t reads its sequence's rows 0 .. token_pos[t].  rank and R multiples of 16, rank <= 512.  n_chunks <= 64 shares;
+// t reads its sequence's rows 0 .. token_pos[t].  rank and R multiples of 16, rank <= 512.  n_chunks <= LC_MAX_CHUNKS shares;
 // more than one: part_o float32 [T, H, n_chunks, rank], part_ml float32 [T, H, n_chunks, 2].
 LLMX_API int llmx_latent_decode(const void* q, const void* cache, const int* block_table, int table_width,
                                 const int* token_seq, const int* token_pos, const int* seq_past, const float* sinks,
                                 float scale, int n_tokens, int H, int rank, int R, int n_chunks, float* part_o,
                                 float* part_ml, void* lat, int n_seqs, long long n_pages, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (H <= 0 || rank <= 0 || rank % 16 || rank > LC_MAX_RANK || R < 0 || R % 16 || n_chunks < 1 || n_chunks > 64 ||
+  if (H <= 0 || rank <= 0 || rank % 16 || rank > LC_MAX_RANK || R < 0 || R % 16 || n_chunks < 1 || n_chunks > LC_MAX_CHUNKS ||
       n_pages <= 0)
     return LLMX_REFUSED(1);
   if (n_chunks > 1 && (!part_o || !part_ml)) return LLMX_REFUSED(4);
@@ -686,7 +698,7 @@ LLMX_API int llmx_latent_decode(const void* q, const void* cache, const int* blo
       if (e != cudaSuccess) return (int)e;                                                                               \
       attr_set = true;                                                                                                   \
     }                                                                                                                    \
-    launch_pdl(latent_decode_kernel<NB, ST>, grid, dim3(LC_WARPS * 32), smem, stream, (const bf16*)q, (const bf16*)cache, \
+    launch_pdl(latent_decode_kernel<NB, ST>, grid, dim3(LC_WARPS * 32 + 32), smem, stream, (const bf16*)q, (const bf16*)cache, \
                block_table, table_width, token_seq, token_pos, seq_past, sinks, scale * 1.4426950408889634f, H, rank, R, \
                n_chunks, part_o, part_ml, (bf16*)lat, n_seqs, (int)n_pages);                                             \
   } while (0)

@@ -744,9 +744,10 @@ def latent_decode_supports(rank: int, rot_dim: int) -> bool:
 
 def latent_decode_chunks(n_tokens: int, n_heads: int, n_pages: int, sms: int = 148) -> int:
     """Into how many shares ``latent_decode`` cuts a token's cached rows: about two CTAs an SM over the whole grid, no
-    share shorter than a page of a full block table.  From the batch's shape alone."""
+    share shorter than two pages of a full block table (a share's float32 partials are as large as a page and a half of
+    rows).  From the batch's shape alone."""
     base = n_tokens * ((n_heads + 15) // 16)
-    return max(1, min(2 * sms // base, n_pages, 64))
+    return max(1, min(2 * sms // base, (n_pages + 1) // 2, 128))
 
 
 def latent_decode(q, lat, cache, block_table, ctx, sinks, scale: float, rank: int, n_chunks: int = 0) -> None:
