@@ -112,7 +112,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   // complete, so its V stage is free, O may be rescaled and (for the last tile) read.  One commit each per tile:
   // the thread that issues the MMAs is what a CTA waits for most, and a commit costs it as much as an MMA.
   const uint32_t q_full = bar0, k_full0 = bar0 + 8, v_full0 = bar0 + 24;
-  const uint32_t s_full0 = bar0 + 40, pv_done0 = bar0 + 56, p_ready = bar0 + 72;
+  const uint32_t s_full0 = bar0 + 40, pv_done0 = bar0 + 56;
+  // p_ready[st]: the probabilities of a tile are stored, one arrival per softmax warp.  Two of them, taken in turn: the
+  // scores of the next tile are under way before P V of this one, so a fast warp may be done with the next tile while
+  // a slow one still works on this; on a single barrier its second arrival would stand for the slow warp's first.  (It
+  // cannot be two tiles ahead: it waits for P V of every tile before the one after the next.)
+  const uint32_t p_ready0 = bar0 + 72;
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 15);
 
   if (threadIdx.x == 0) {
@@ -123,7 +128,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       mbar_init(s_full0 + 8u * i, 1);
       mbar_init(pv_done0 + 8u * i, 1);
     }
-    mbar_init(p_ready, 4);                   // one arrival per softmax warp
+    for (int i = 0; i < 2; ++i) mbar_init(p_ready0 + 8u * i, 4);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     asm volatile("prefetch.tensormap [%0];" ::"l"(&map_q) : "memory");
     asm volatile("prefetch.tensormap [%0];" ::"l"(&map_k) : "memory");
@@ -170,7 +175,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const uint64_t q0 = umma_desc(sQ);
       auto issue_pv = [&](int j) {       // O += P_j V_j
         const int st = j & 1;
-        if (!mbar_wait(p_ready, j & 1)) { at_report(5); return false; }
+        if (!mbar_wait(p_ready0 + 8u * st, (j >> 1) & 1)) { at_report(5); return false; }
         if (!mbar_wait(v_full0 + 8u * st, (j >> 1) & 1)) { at_report(6); return false; }
         tc_fence_after();
         const uint64_t v0 = umma_desc_mn(sV0 + (uint32_t)st * AT_KTILE, AT_KPANEL, 1024u);
@@ -306,7 +311,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       fence_proxy_async();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_ready);
+      if (lane == 0) mbar_arrive(p_ready0 + 8u * st);
       if (j >= 1 && !rescale) {
         ok = mbar_wait(pv_done0 + 8u * ((j - 1) & 1), ((j - 1) >> 1) & 1);
         if (!ok && lane == 0) at_report(8);

@@ -719,3 +719,26 @@ def test_norm_in_two_halves(T, d, N2):
             kernels.gemm_tc(x, w2d, act, gated=2, scale=(sumsq, parts, eps, d))
             assert rel(act, (plain.silu(blocks[:, :, 0]) * blocks[:, :, 1]).reshape(T, F)) < 1e-2
     assert kernels.gemm_tc_status() == 0
+
+
+def test_tcgen05_prompt_attention_gives_the_same_bits_every_time():
+    """Three hundred launches of one prompt attention.  Its softmax warps run apart by up to a tile, and how far depends
+    on what else the SM does; no order of theirs may reach the result."""
+    from llmoxide_b200 import kernels
+
+    g = torch.Generator().manual_seed(77)
+    H, G, D, n = 16, 4, 128, 2048
+    pages = n // 64
+    q = torch.randn(n, H * D, generator=g).to(torch.bfloat16).cuda()
+    k, v = (torch.randn(pages, G, 64, D, generator=g).to(torch.bfloat16).cuda() for _ in range(2))
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    table, start, past = i32([list(range(pages))]), i32([0, n]), i32([0])
+    first, bad = None, torch.zeros((), dtype=torch.int64, device="cuda")
+    for _ in range(300):
+        out = torch.full_like(q, float("nan"))
+        kernels.attention_prefill_tc(q, out, k, v, table, start, past, 1, n, H, G, D, None, D ** -0.5)
+        if first is None:
+            first = out
+        bad += (out.view(torch.int16) != first.view(torch.int16)).any()
+    assert int(bad) == 0
+    kernels.check_status()
