@@ -44,8 +44,9 @@
 // the chunks are summed in chunk order, so the result does not depend on
 // timing.
 //
-// Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own) every scaled score is capped (common.cuh).
-// `sinks` (float32 [H]): exp(sinks[h]) joins head h's merged denominator once.
+// Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own, so that the first carries none of it) every scaled
+// score is capped when a cap is given (common.cuh), and with `sinks` (float32 [H]) exp(sinks[h]) joins head h's merged
+// denominator once.
 #include "tc_ptx.cuh"
 #include <type_traits>
 
@@ -103,6 +104,24 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 __device__ __forceinline__ float dec_sink(const float* sinks, int head, float mx) {
   return exp2f(sinks[head] * 1.4426950408889634f - mx);
 }
+#if LLMX_SCORE_CAP
+#define DEC_ADD_SINK(l, head, mx) \
+  if (ps.sinks) l += dec_sink(ps.sinks, head, mx);
+#else
+#define DEC_ADD_SINK(l, head, mx)
+#endif
+
+// What the second library's kernel knows beyond the first's; the first takes the empty form.
+struct DecScore {
+  ScoreCap cap;
+  const float* sinks;
+};
+struct DecPlainScore {};
+#if LLMX_SCORE_CAP
+typedef DecScore DecScoreArg;
+#else
+typedef DecPlainScore DecScoreArg;
+#endif
 
 // Two layouts of a tile in shared memory, both free of ldmatrix bank conflicts.  Head sizes that are multiples
 // of 64 come by tensor copies (one request per 64 head dims of a tile, issued by one lane) in panels of
@@ -141,9 +160,12 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ seq_past,
                         float* __restrict__ ws, unsigned int* __restrict__ counters, bf16* __restrict__ out, int H,
                         int G, int window, int keep_first, int mask_chunk, float scale_log2, float sink,
-                        const float* __restrict__ sinks, const ScoreCap cap, int n_chunks, int cluster_merge,
+                        const DecScoreArg ps, int n_chunks, int cluster_merge,
                         const __grid_constant__ std::conditional_t<POOLED, DecPool, DecNoPool> pp) {
   using S = DecSmem<D>;
+#if LLMX_SCORE_CAP
+  const ScoreCap cap = ps.cap;
+#endif
   int pool = 0;
   const CUtensorMap* map_pk = &map_k;
   const CUtensorMap* map_pv = &map_v;
@@ -311,8 +333,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
           const int key = key0 + 16 * i + gq + 8 * e;
           const bool vis = pooled ? key < n_rows : ((key >= first || key < keep_first) && key <= p);
 #if LLMX_SCORE_CAP
-          s[i][2 * e] = vis ? capped_score_log2(cap, s[i][2 * e]) : -INFINITY;
-          s[i][2 * e + 1] = vis ? capped_score_log2(cap, s[i][2 * e + 1]) : -INFINITY;
+          const bool capped = cap.top > 0.f;
+          s[i][2 * e] = !vis ? -INFINITY : capped ? capped_score_log2(cap, s[i][2 * e]) : s[i][2 * e] * scale_log2;
+          s[i][2 * e + 1] = !vis ? -INFINITY : capped ? capped_score_log2(cap, s[i][2 * e + 1]) : s[i][2 * e + 1] * scale_log2;
 #else
           s[i][2 * e] = vis ? s[i][2 * e] * scale_log2 : -INFINITY;
           s[i][2 * e + 1] = vis ? s[i][2 * e + 1] * scale_log2 : -INFINITY;
@@ -421,7 +444,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     }
     if (n_chunks == 1) {                                                              // nothing to merge with
       if (sink > 0.f) ls += sink * exp2f(-mx);       // the sink: keys of score 0 without a value (mx in log2 units)
-      if (sinks) ls += dec_sink(sinks, h0 + h, mx);
+      DEC_ADD_SINK(ls, h0 + h, mx)
       __nv_bfloat162 lo = __floats2bfloat162_rn(a.x / ls, a.y / ls), hi = __floats2bfloat162_rn(a.z / ls, a.w / ls);
       *reinterpret_cast<uint2*>(out + ((size_t)b * H + h0 + h) * D + d) =
           make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
@@ -487,7 +510,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
       }
       if (sink > 0.f) l += sink * exp2f(-mx);        // the sink joins the merged denominator once
-      if (sinks) l += dec_sink(sinks, h0 + h, mx);
+      DEC_ADD_SINK(l, h0 + h, mx)
       const float r = 1.f / l;
       __nv_bfloat162 lo = __floats2bfloat162_rn(a.x * r, a.y * r), hi2 = __floats2bfloat162_rn(a.z * r, a.w * r);
       uint2 packed = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi2));
@@ -535,7 +558,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       if (w != 0.f) l += w * ls[c];
     }
     if (sink > 0.f) l += sink * exp2f(-mx);          // the sink joins the merged denominator once
-    if (sinks) l += dec_sink(sinks, h0 + threadIdx.x, mx);
+    DEC_ADD_SINK(l, h0 + threadIdx.x, mx)
     inv[threadIdx.x] = 1.f / l;
   }
   __syncthreads();
@@ -600,18 +623,22 @@ static int launch_decode_as(const void* q, void* out, const void* k_cache, const
       if (make_map(&pp.map_pv, pool_v, pool_rows, D, D, DEC_TILE, false)) return LLMX_REFUSED(4);
     }
   }
-  const ScoreCap cap = make_score_cap(scale, softcap);
+  DecScoreArg ps{};
+#if LLMX_SCORE_CAP
+  ps.cap = make_score_cap(scale, softcap);
+  ps.sinks = sinks;
+#endif
   // up to 8 chunks (the portable cluster size): merged inside a cluster, nothing goes through the workspace
   const int cluster_merge = (n_chunks > 1 && n_chunks <= 8) ? 1 : 0;
   if (cluster_merge)
     launch_pdl_cluster(kernel, grid, dim3(DEC_WARPS * 32), smem, stream, (unsigned)n_chunks, mk, mv, (const bf16*)q,
                        (const bf16*)k_cache, (const bf16*)v_cache, block_table, table_width, seq_past, ws, counters,
-                       (bf16*)out, H, G, window, keep_first, mask_chunk, scale * 1.4426950408889634f, sink, sinks, cap,
+                       (bf16*)out, H, G, window, keep_first, mask_chunk, scale * 1.4426950408889634f, sink, ps,
                        n_chunks, cluster_merge, pp);
   else
     launch_pdl(kernel, grid, dim3(DEC_WARPS * 32), smem, stream, mk, mv, (const bf16*)q, (const bf16*)k_cache,
                (const bf16*)v_cache, block_table, table_width, seq_past, ws, counters, (bf16*)out, H, G, window,
-               keep_first, mask_chunk, scale * 1.4426950408889634f, sink, sinks, cap, n_chunks, cluster_merge, pp);
+               keep_first, mask_chunk, scale * 1.4426950408889634f, sink, ps, n_chunks, cluster_merge, pp);
   return LLMX_LAUNCH_STATUS();
 }
 
@@ -644,7 +671,7 @@ static int launch_decode(const void* q, void* out, const void* k_cache, const vo
 // pool n > 0 (beside a window, without kept first keys or a chunked mask): every block of n positions that lies
 // wholly before the token's window is seen as row b of pool_k / pool_v, a second store [n_pool_pages, G, 64, D]
 // paged like the cache with the block table pool_table (as wide as block_table).
-// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it.
+// sinks: null, or float32 [H]; softcap: 0, or the cap; both only in the library with LLMX_SCORE_CAP.
 LLMX_API int llmx_attention_decode_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
                                           long long n_pages, const int* block_table, int table_width,
                                           const int* seq_past, float* ws, unsigned int* counters, int B, int H, int G,
@@ -653,7 +680,7 @@ LLMX_API int llmx_attention_decode_capped(const void* q, void* out, const void* 
                                           const void* pool_k, const void* pool_v, long long n_pool_pages,
                                           const int* pool_table, cudaStream_t stream) {
   if (B <= 0) return 0;
-  if ((softcap > 0.f) != (LLMX_SCORE_CAP != 0) || (LLMX_SCORE_CAP && pool > 0)) return LLMX_REFUSED(1);
+  if ((!LLMX_SCORE_CAP && (softcap > 0.f || sinks)) || (LLMX_SCORE_CAP && pool > 0)) return LLMX_REFUSED(1);
   if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || mask_chunk > 0 || !pool_k || !pool_v || !pool_table ||
                                 n_pool_pages <= 0 || ((uintptr_t)pool_k & 15) || ((uintptr_t)pool_v & 15))))
     return LLMX_REFUSED(1);

@@ -863,7 +863,7 @@ def _counters(device, n: int):
 
 
 def capped_library(name: str, softcap) -> str:
-    """The library of a tiled attention kernel: its own build where scores are capped."""
+    """The library of a tiled attention kernel: its own build where scores are capped (decode: or sinks learned)."""
     return name + "_capped" if softcap else name
 
 
@@ -902,7 +902,7 @@ def attention_decode(q, out, k_cache, v_cache, block_table, seq_past, n_heads: i
         ws = guard.scratch((B * n_heads * n_chunks * (head_dim + 4),), torch.float32, q.device,
                            "decode attention workspace")
         counters = _counters(q.device, B * n_kv_heads * ((group + 7) // 8))
-    f = _fn(capped_library("attention_decode", softcap), "llmx_attention_decode_capped",
+    f = _fn(capped_library("attention_decode", softcap or sinks is not None), "llmx_attention_decode_capped",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
              c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float, c_int, c_int, c_void_p,
              c_void_p, c_longlong, c_void_p, c_void_p])

@@ -161,7 +161,7 @@ class LatentAttention:
             return libs
         libs = {"latent_attention", "elementwise"} | self.down.libraries() | self.uq.libraries() | self.o.libraries()
         if self.plain and self.rt.dtype == "bfloat16" and self.rt.tensor_cores:
-            libs |= {"attention_decode",
+            libs |= {kernels.capped_library("attention_decode", self.sinks is not None),
                      "attention_prefill_tc" if self.E == 128 else "attention_prefill" if self.E == 64 else "attention"}
         else:
             libs.add("attention")
