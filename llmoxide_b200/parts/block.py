@@ -183,7 +183,7 @@ class HyperConnectionBlock:
         return self.mixer.cache_need()
 
     def libraries(self) -> set:
-        libs = set()
+        libs = {"stream_mix"}
         for part in (self.mixer_norm, self.ff_norm, self.mixer, self.feed_forward):
             if part is not None:
                 libs |= getattr(part, "libraries", set)()

@@ -140,7 +140,8 @@ class RMSNorm:
         self._plain: dict = {}
 
     def libraries(self) -> set:
-        return {"elementwise", "stream_mix", "post_norm"}
+        # (several copies of the stream: their arrangement names the library for that)
+        return {"elementwise", "post_norm"}
 
     def owed(self, delta, n_streams: int = 0, bias=None, gate=None):
         """The update by which a sublayer's result ``delta`` (None: nothing) joins ``n_streams`` copies; without
