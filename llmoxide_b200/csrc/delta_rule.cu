@@ -308,6 +308,7 @@ delta_scan_kernel(const float* __restrict__ qk, const float* __restrict__ vv, co
   }
   const uint32_t v_bytes = (uint32_t)(DR_CHUNK * min(cols, Dvp - c_cta)) * 4u;
   auto load_chunk = [&](int ch) {                      // one thread
+    if (llmx_withhold && ch == 0 && (blockIdx.x | blockIdx.y | blockIdx.z) == 0) return;     // (tests: never asked for)
     const int st = ch % DR_STAGES;
     const uint32_t dst = ring + (uint32_t)(st * stage_len) * 4u, bar = bars + 8 * st;
     mbar_expect_tx(bar, 2u * DR_CHUNK * DL * 4u + DR_COEF * 4u + v_bytes);

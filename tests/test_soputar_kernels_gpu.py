@@ -333,6 +333,7 @@ class _Delta:
                 outs[b].append(y[at : at + n].cpu())
                 at += n
                 fed[b] += n
+        torch.cuda.synchronize()
         kernels.check_status()
         assert float(state[1::2].min()) == float(state[1::2].max()) == 7.0        # nobody's slots stay as they were
         return [torch.cat(o) for o in outs], state
@@ -601,4 +602,45 @@ def test_gathered_latents_and_assembled_pages(H, D, R, Dv, rank):
                 assert torch.equal(vals[at, h, r], src[H * D + h * Dv : H * D + (h + 1) * Dv])
         if L % 64:
             assert float(vals[first[b] + L // 64, :, L % 64 :].float().abs().max()) == 0.0
+    kernels.check_status()
+
+
+# ---------------------------------------------------------------------------------------------------------
+# waits that run out are reported, and the libraries go on
+# ---------------------------------------------------------------------------------------------------------
+
+def test_a_wait_that_runs_out_is_reported_and_the_library_goes_on():
+    """One CTA of each kernel leaves out its first copy; its bounded wait runs out (a short limit), the kernel winds down
+    and reports, and the next launch is right again."""
+    from llmoxide_b200 import kernels
+    from llmoxide_b200.errors import KernelError
+
+    case = _Delta(2, 1, 32, 16, 2, [20], seed=21)
+    want = case.want(0)[1].numpy()
+    assert _rel(case.run([[20]])[0][0].numpy(), want) < 3e-5
+    H, rank, R, n = 4, 64, 16, 150
+    rows = _latent_rows([n], rank, R, torch.bfloat16, 1)
+    q = _exact(torch.randn(1, H, rank + R, generator=torch.Generator().manual_seed(1)), torch.bfloat16)
+    table, (cache,) = _store([n], 1, rank + R, dtype=torch.bfloat16)
+    _fill(table, cache, 0, rows[0][:, None, :])
+    ctx = _ctx([n - 1], [1])
+    expect = _plain_latents(q[0], rows[0], rank, 0.1, None).numpy()
+
+    def attend():
+        lat = torch.empty((1, H, rank), dtype=torch.bfloat16, device=DEV)
+        kernels.latent_decode(q.to(torch.bfloat16).to(DEV).contiguous(), lat, cache, table, ctx, None, 0.1, rank, n_chunks=2)
+        torch.cuda.synchronize()
+        return lat[0].float().cpu().numpy()
+
+    assert _rel(attend(), expect) < 8e-3
+    for lib, launch in (("delta_rule", lambda: case.run([[20]])), ("latent_cache", attend)):
+        try:
+            kernels.test_waits(lib, 1_000_000, True)
+            with pytest.raises(KernelError, match=lib):
+                launch()
+                kernels.check_status()
+        finally:
+            kernels.test_waits(lib, 0, False)
+        kernels.check_status()                      # the report was cleared
+    assert _rel(case.run([[20]])[0][0].numpy(), want) < 3e-5 and _rel(attend(), expect) < 8e-3
     kernels.check_status()
