@@ -21,6 +21,8 @@
 // With `gate` a head's output is multiplied by sigmoid(gate[t * gate_stride + hq]).
 // With `softcap` c > 0 a scaled score s becomes c * tanh(s / c) before the softmax.  With `sinks` (float32 [H]) the
 // denominator of head hq has exp(sinks[hq]) added: a learned score without key and value, neither scaled nor capped.
+// With `score_bias` (float32 [H, bias_len]) the scaled score of the key at j has score_bias[hq, min(p - j, bias_len - 1)]
+// added: a learned number per distance and head (not beside pooled blocks or a cap).
 //
 // One warp per (token, head).  Keys are taken 32 at a time starting at the
 // range's first key: lane j scores key lo + c*32 + j with a sequential dot over
@@ -42,7 +44,8 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
                                        float scale, float sink, int chunk, int pool,
                                        const TC* __restrict__ pool_k, const TC* __restrict__ pool_v,
                                        const int* __restrict__ pool_table, const float* __restrict__ gate,
-                                       size_t gate_stride, float softcap, const float* __restrict__ sinks) {
+                                       size_t gate_stride, float softcap, const float* __restrict__ sinks,
+                                       const float* __restrict__ score_bias, int bias_len) {
   extern __shared__ float q_buf[];  // [ATT_WARPS][D]
   pdl_launch_dependents();
   pdl_wait();
@@ -90,6 +93,7 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
       for (int i = 0; i < D; ++i) dot += qs[i] * to_f32(krow[i]);
       s = dot * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      if (score_bias) s += score_bias[(size_t)hq * bias_len + min(p - j, bias_len - 1)];
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);  // exp(-inf) = 0 on the first chunk; lane 0 of a chunk is always live
@@ -127,15 +131,16 @@ __global__ void attention_paged_kernel(const TA* __restrict__ q, TA* __restrict_
 // pool > 0: pool_k / pool_v hold one row per block of `pool` positions, paged like the cache, with the block table
 // pool_table (as wide as block_table); needs a window and no kept first keys.  gate: null, or float32 with
 // gate[t * gate_stride + head] the logit of head's output gate.
-// softcap <= 0: scores are not capped; sinks: null, or float32 [H].
-LLMX_API int llmx_attention_paged_capped(const void* q, void* out, int act_dtype, const void* k_cache,
+// softcap <= 0: scores are not capped; sinks: null, or float32 [H]; score_bias: null, or float32 [H, bias_len].
+LLMX_API int llmx_attention_paged_biased(const void* q, void* out, int act_dtype, const void* k_cache,
                                   const void* v_cache, int cache_dtype, const int* block_table, int table_width,
                                   const int* token_seq, const int* token_pos, int n_tokens, int H, int G, int D,
                                   int Dv, long long q_stride, int window, int keep_first, float scale, float sink,
                                   int chunk, int pool, const void* pool_k, const void* pool_v, const int* pool_table,
                                   const float* gate, long long gate_stride, float softcap, const float* sinks,
-                                  cudaStream_t stream) {
+                                  const float* score_bias, int bias_len, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
+  if (score_bias && (bias_len <= 0 || pool > 0 || softcap > 0.f)) return LLMX_REFUSED(1);
   if (chunk < 0 || (chunk > 0 && keep_first > 0)) return LLMX_REFUSED(1);
   if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || chunk > 0 || !pool_k || !pool_v || !pool_table)))
     return LLMX_REFUSED(1);
@@ -148,7 +153,7 @@ LLMX_API int llmx_attention_paged_capped(const void* q, void* out, int act_dtype
   launch_pdl(attention_paged_kernel<TA, TC>, grid, dim3(ATT_WARPS * 32), smem, stream,                    \
       (const TA*)q, (TA*)out, (const TC*)k_cache, (const TC*)v_cache, block_table, table_width, token_seq, \
       token_pos, H, G, D, Dv, (size_t)q_stride, window, keep_first, scale, sink, chunk, pool, (const TC*)pool_k,  \
-      (const TC*)pool_v, pool_table, gate, (size_t)gate_stride, softcap, sinks)
+      (const TC*)pool_v, pool_table, gate, (size_t)gate_stride, softcap, sinks, score_bias, bias_len)
   if (act_dtype == LLMX_F32 && cache_dtype == LLMX_F32) CASE(float, float);
   else if (act_dtype == LLMX_BF16 && cache_dtype == LLMX_BF16) CASE(bf16, bf16);
   else if (act_dtype == LLMX_F32 && cache_dtype == LLMX_BF16) CASE(float, bf16);
@@ -156,6 +161,19 @@ LLMX_API int llmx_attention_paged_capped(const void* q, void* out, int act_dtype
   else return LLMX_REFUSED(2);
 #undef CASE
   return LLMX_LAUNCH_STATUS();
+}
+
+LLMX_API int llmx_attention_paged_capped(const void* q, void* out, int act_dtype, const void* k_cache,
+                                  const void* v_cache, int cache_dtype, const int* block_table, int table_width,
+                                  const int* token_seq, const int* token_pos, int n_tokens, int H, int G, int D,
+                                  int Dv, long long q_stride, int window, int keep_first, float scale, float sink,
+                                  int chunk, int pool, const void* pool_k, const void* pool_v, const int* pool_table,
+                                  const float* gate, long long gate_stride, float softcap, const float* sinks,
+                                  cudaStream_t stream) {
+  return llmx_attention_paged_biased(q, out, act_dtype, k_cache, v_cache, cache_dtype, block_table, table_width,
+                                     token_seq, token_pos, n_tokens, H, G, D, Dv, q_stride, window, keep_first, scale,
+                                     sink, chunk, pool, pool_k, pool_v, pool_table, gate, gate_stride, softcap, sinks,
+                                     nullptr, 0, stream);
 }
 
 LLMX_API int llmx_attention_paged_pooled(const void* q, void* out, int act_dtype, const void* k_cache,

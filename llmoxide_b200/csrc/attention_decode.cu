@@ -46,7 +46,8 @@
 //
 // Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own, so that the first carries none of it) every scaled
 // score is capped when a cap is given (common.cuh), and with `sinks` (float32 [H]) exp(sinks[h]) joins head h's merged
-// denominator once.
+// denominator once.  Compiled a third time with LLMX_SCORE_BIAS=1 a learned bias per distance and head joins every scaled
+// score (common.cuh), asked for before the tile's keys are waited for; that build takes sinks as well.
 #include "tc_ptx.cuh"
 #include <type_traits>
 
@@ -104,7 +105,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 __device__ __forceinline__ float dec_sink(const float* sinks, int head, float mx) {
   return exp2f(sinks[head] * 1.4426950408889634f - mx);
 }
-#if LLMX_SCORE_CAP
+#if LLMX_SCORE_CAP || LLMX_SCORE_BIAS
 #define DEC_ADD_SINK(l, head, mx) \
   if (ps.sinks) l += dec_sink(ps.sinks, head, mx);
 #else
@@ -117,7 +118,7 @@ struct DecScore {
   const float* sinks;
 };
 struct DecPlainScore {};
-#if LLMX_SCORE_CAP
+#if LLMX_SCORE_CAP || LLMX_SCORE_BIAS
 typedef DecScore DecScoreArg;
 #else
 typedef DecPlainScore DecScoreArg;
@@ -160,7 +161,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ seq_past,
                         float* __restrict__ ws, unsigned int* __restrict__ counters, bf16* __restrict__ out, int H,
                         int G, int window, int keep_first, int mask_chunk, float scale_log2, float sink,
-                        const DecScoreArg ps, int n_chunks, int cluster_merge,
+                        const DecScoreArg ps, const ScoreBiasArg bias, int n_chunks, int cluster_merge,
                         const __grid_constant__ std::conditional_t<POOLED, DecPool, DecNoPool> pp) {
   using S = DecSmem<D>;
 #if LLMX_SCORE_CAP
@@ -293,10 +294,24 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         load_tile(tile_lo + issued, issued % DEC_STAGES);
         ++issued;
       }
+      const int key0 = tile_at(tile_lo + t) * DEC_TILE;
+#if LLMX_SCORE_BIAS
+      float sb[DEC_TILE / 16][4];                                // the biases of this lane's scores
+      {
+        const float* b0 = bias.table + (size_t)(h0 + min(2 * tq, n_heads - 1)) * bias.len;
+        const float* b1 = bias.table + (size_t)(h0 + min(2 * tq + 1, n_heads - 1)) * bias.len;
+#pragma unroll
+        for (int i = 0; i < DEC_TILE / 16; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int d = min(max(p - (key0 + 16 * i + gq + 8 * e), 0), bias.len - 1);
+            sb[i][2 * e] = __ldg(b0 + d), sb[i][2 * e + 1] = __ldg(b1 + d);
+          }
+      }
+#endif
       ok = __all_sync(0xffffffffu, mbar_wait(bars + 8 * stage, (t / DEC_STAGES) & 1));   // the warp leaves together
       if (!ok) break;
       const uint32_t sK = sKV + stage * 2 * S::TILE, sV = sK + S::TILE;
-      const int key0 = tile_at(tile_lo + t) * DEC_TILE;
       const bool pooled = POOLED && tile_lo + t < n_kept;
       const int last_row = pooled ? n_rows - 1 : p;               // the last row of the tile's store that is seen
       if (key0 + DEC_TILE - 1 > last_row) {
@@ -336,6 +351,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
           const bool capped = cap.top > 0.f;
           s[i][2 * e] = !vis ? -INFINITY : capped ? capped_score_log2(cap, s[i][2 * e]) : s[i][2 * e] * scale_log2;
           s[i][2 * e + 1] = !vis ? -INFINITY : capped ? capped_score_log2(cap, s[i][2 * e + 1]) : s[i][2 * e + 1] * scale_log2;
+#elif LLMX_SCORE_BIAS
+          s[i][2 * e] = vis ? fmaf(s[i][2 * e], scale_log2, sb[i][2 * e] * LLMX_LOG2E) : -INFINITY;
+          s[i][2 * e + 1] = vis ? fmaf(s[i][2 * e + 1], scale_log2, sb[i][2 * e + 1] * LLMX_LOG2E) : -INFINITY;
 #else
           s[i][2 * e] = vis ? s[i][2 * e] * scale_log2 : -INFINITY;
           s[i][2 * e + 1] = vis ? s[i][2 * e + 1] * scale_log2 : -INFINITY;
@@ -589,7 +607,7 @@ template <int D, bool POOLED>
 static int launch_decode_as(const void* q, void* out, const void* k_cache, const void* v_cache, long long n_pages,
                          const int* block_table, int table_width, const int* seq_past, float* ws, unsigned int* counters, int B, int H, int G,
                          int window, int keep_first, int mask_chunk, float scale, float sink, const float* sinks,
-                         float softcap, int n_chunks, cudaStream_t stream, int pool = 0, const void* pool_k = nullptr, const void* pool_v = nullptr,
+                         float softcap, const ScoreBiasArg bias, int n_chunks, cudaStream_t stream, int pool = 0, const void* pool_k = nullptr, const void* pool_v = nullptr,
                          long long n_pool_pages = 0, const int* pool_table = nullptr) {
   const int R = H / G;
   const int head_groups = (R + DEC_ROWS - 1) / DEC_ROWS;
@@ -624,7 +642,7 @@ static int launch_decode_as(const void* q, void* out, const void* k_cache, const
     }
   }
   DecScoreArg ps{};
-#if LLMX_SCORE_CAP
+#if LLMX_SCORE_CAP || LLMX_SCORE_BIAS
   ps.cap = make_score_cap(scale, softcap);
   ps.sinks = sinks;
 #endif
@@ -634,11 +652,11 @@ static int launch_decode_as(const void* q, void* out, const void* k_cache, const
     launch_pdl_cluster(kernel, grid, dim3(DEC_WARPS * 32), smem, stream, (unsigned)n_chunks, mk, mv, (const bf16*)q,
                        (const bf16*)k_cache, (const bf16*)v_cache, block_table, table_width, seq_past, ws, counters,
                        (bf16*)out, H, G, window, keep_first, mask_chunk, scale * 1.4426950408889634f, sink, ps,
-                       n_chunks, cluster_merge, pp);
+                       bias, n_chunks, cluster_merge, pp);
   else
     launch_pdl(kernel, grid, dim3(DEC_WARPS * 32), smem, stream, mk, mv, (const bf16*)q, (const bf16*)k_cache,
                (const bf16*)v_cache, block_table, table_width, seq_past, ws, counters, (bf16*)out, H, G, window,
-               keep_first, mask_chunk, scale * 1.4426950408889634f, sink, ps, n_chunks, cluster_merge, pp);
+               keep_first, mask_chunk, scale * 1.4426950408889634f, sink, ps, bias, n_chunks, cluster_merge, pp);
   return LLMX_LAUNCH_STATUS();
 }
 
@@ -646,16 +664,16 @@ template <int D>
 static int launch_decode(const void* q, void* out, const void* k_cache, const void* v_cache, long long n_pages,
                          const int* block_table, int table_width, const int* seq_past, float* ws, unsigned int* counters, int B, int H, int G,
                          int window, int keep_first, int mask_chunk, float scale, float sink, const float* sinks,
-                         float softcap, int n_chunks, cudaStream_t stream, int pool = 0, const void* pool_k = nullptr, const void* pool_v = nullptr,
+                         float softcap, const ScoreBiasArg bias, int n_chunks, cudaStream_t stream, int pool = 0, const void* pool_k = nullptr, const void* pool_v = nullptr,
                          long long n_pool_pages = 0, const int* pool_table = nullptr) {
-#if !LLMX_SCORE_CAP            // (pooled blocks beside capped scores are not built)
+#if !LLMX_SCORE_CAP && !LLMX_SCORE_BIAS     // (pooled blocks beside capped or biased scores are not built)
   if (pool > 0)
     return launch_decode_as<D, true>(q, out, k_cache, v_cache, n_pages, block_table, table_width, seq_past, ws, counters, B,
-                                     H, G, window, keep_first, mask_chunk, scale, sink, sinks, softcap, n_chunks, stream, pool, pool_k,
+                                     H, G, window, keep_first, mask_chunk, scale, sink, sinks, softcap, bias, n_chunks, stream, pool, pool_k,
                                      pool_v, n_pool_pages, pool_table);
 #endif
   return launch_decode_as<D, false>(q, out, k_cache, v_cache, n_pages, block_table, table_width, seq_past, ws, counters, B,
-                                    H, G, window, keep_first, mask_chunk, scale, sink, sinks, softcap, n_chunks, stream, 0, nullptr,
+                                    H, G, window, keep_first, mask_chunk, scale, sink, sinks, softcap, bias, n_chunks, stream, 0, nullptr,
                                     nullptr, 0, nullptr);
 }
 
@@ -671,16 +689,21 @@ static int launch_decode(const void* q, void* out, const void* k_cache, const vo
 // pool n > 0 (beside a window, without kept first keys or a chunked mask): every block of n positions that lies
 // wholly before the token's window is seen as row b of pool_k / pool_v, a second store [n_pool_pages, G, 64, D]
 // paged like the cache with the block table pool_table (as wide as block_table).
-// sinks: null, or float32 [H]; softcap: 0, or the cap; both only in the library with LLMX_SCORE_CAP.
-LLMX_API int llmx_attention_decode_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
+// sinks: null, or float32 [H]; softcap: 0, or the cap; both only in the library with LLMX_SCORE_CAP (sinks also in the one
+// with LLMX_SCORE_BIAS).  score_bias: float32 [H, bias_len] in the library with LLMX_SCORE_BIAS, null in the others.
+LLMX_API int llmx_attention_decode_biased(const void* q, void* out, const void* k_cache, const void* v_cache,
                                           long long n_pages, const int* block_table, int table_width,
                                           const int* seq_past, float* ws, unsigned int* counters, int B, int H, int G,
                                           int D, int window, int keep_first, int mask_chunk, float scale, float sink,
                                           const float* sinks, float softcap, int n_chunks, int pool,
                                           const void* pool_k, const void* pool_v, long long n_pool_pages,
-                                          const int* pool_table, cudaStream_t stream) {
+                                          const int* pool_table, const float* score_bias, int bias_len,
+                                          cudaStream_t stream) {
   if (B <= 0) return 0;
-  if ((!LLMX_SCORE_CAP && (softcap > 0.f || sinks)) || (LLMX_SCORE_CAP && pool > 0)) return LLMX_REFUSED(1);
+  if ((!LLMX_SCORE_CAP && softcap > 0.f) || (!LLMX_SCORE_CAP && !LLMX_SCORE_BIAS && sinks) ||
+      ((LLMX_SCORE_CAP || LLMX_SCORE_BIAS) && pool > 0))
+    return LLMX_REFUSED(1);
+  if ((score_bias != nullptr) != (LLMX_SCORE_BIAS != 0) || (score_bias && bias_len <= 0)) return LLMX_REFUSED(1);
   if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || mask_chunk > 0 || !pool_k || !pool_v || !pool_table ||
                                 n_pool_pages <= 0 || ((uintptr_t)pool_k & 15) || ((uintptr_t)pool_v & 15))))
     return LLMX_REFUSED(1);
@@ -695,7 +718,7 @@ LLMX_API int llmx_attention_decode_capped(const void* q, void* out, const void* 
 #define CASE(DD)                                                                                               \
   case DD:                                                                                                     \
     return launch_decode<DD>(q, out, k_cache, v_cache, n_pages, block_table, table_width, seq_past, ws, counters, \
-                             B, H, G, window, keep_first, mask_chunk, scale, sink, sinks, softcap, n_chunks, stream, pool, pool_k,   \
+                             B, H, G, window, keep_first, mask_chunk, scale, sink, sinks, softcap, make_score_bias(score_bias, bias_len), n_chunks, stream, pool, pool_k, \
                              pool_v, n_pool_pages, pool_table)
   switch (D) {
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
@@ -703,6 +726,18 @@ LLMX_API int llmx_attention_decode_capped(const void* q, void* out, const void* 
     default: return LLMX_REFUSED(1);
   }
 #undef CASE
+}
+
+LLMX_API int llmx_attention_decode_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
+                                          long long n_pages, const int* block_table, int table_width,
+                                          const int* seq_past, float* ws, unsigned int* counters, int B, int H, int G,
+                                          int D, int window, int keep_first, int mask_chunk, float scale, float sink,
+                                          const float* sinks, float softcap, int n_chunks, int pool,
+                                          const void* pool_k, const void* pool_v, long long n_pool_pages,
+                                          const int* pool_table, cudaStream_t stream) {
+  return llmx_attention_decode_biased(q, out, k_cache, v_cache, n_pages, block_table, table_width, seq_past, ws,
+                                      counters, B, H, G, D, window, keep_first, mask_chunk, scale, sink, sinks, softcap,
+                                      n_chunks, pool, pool_k, pool_v, n_pool_pages, pool_table, nullptr, 0, stream);
 }
 
 LLMX_API int llmx_attention_decode_pooled(const void* q, void* out, const void* k_cache, const void* v_cache,

@@ -17,11 +17,14 @@
 //
 // Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own) every scaled score is capped (common.cuh).
 // `sinks` (float32 [H]): exp(sinks[h]) joins head h's denominator once.
+// Compiled a third time with LLMX_SCORE_BIAS=1 a learned bias per distance and head joins every scaled score (common.cuh): a
+// warp's 16 rows and 64 keys span 79 distances, which it copies to shared memory once per tile.
 #include "common.cuh"
 
 #define PF_BQ 64          // query tokens per CTA (4 warps x 16 rows)
 #define PF_BK LLMX_PAGE   // keys per tile = one cache page
 #define PF_THREADS 128
+#define PF_BIAS 80         // distances between a warp's rows and a tile's keys (79), padded
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
@@ -68,7 +71,8 @@ attention_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, con
                          const int* __restrict__ seq_start, const int* __restrict__ seq_past, int H, int G,
                          int window, int keep_first, int mask_chunk, float scale_log2, float sink, int pool_arg,
                          const bf16* __restrict__ pool_k, const bf16* __restrict__ pool_v,
-                         const int* __restrict__ pool_table, const float* __restrict__ sinks, const ScoreCap cap) {
+                         const int* __restrict__ pool_table, const float* __restrict__ sinks, const ScoreCap cap,
+                         const ScoreBiasArg bias) {
   const int pool = POOLED ? pool_arg : 0;
   constexpr int CHUNKS = D / 8;              // 16-byte chunks per row
   constexpr int KSTEPS = D / 16;             // k-steps of the score product
@@ -163,6 +167,16 @@ attention_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, con
     }
     const uint32_t sK = sKV + stage * 2 * TILE_BYTES, sV = sK + TILE_BYTES;
     const int key0 = page_of(t) * PF_BK;
+#if LLMX_SCORE_BIAS
+    // the biases of this warp's distances, from the farthest key of the tile's first row to the nearest of its last
+    float* wbias = reinterpret_cast<float*>(smem + PF_BQ * D * 2 + 4 * TILE_BYTES) + warp * PF_BIAS;
+    {
+      const float* brow = bias.table + (size_t)hq * bias.len;
+      const int d0 = past + i0 + warp * 16 - (key0 + PF_BK - 1);
+      for (int i = lane; i < PF_BIAS; i += 32) wbias[i] = brow[min(max(d0 + i, 0), bias.len - 1)] * LLMX_LOG2E;
+    }
+    __syncwarp();
+#endif
     const bool pooled = POOLED && t < n_kept_tiles;
     const int last_row = pooled ? rows_hi - 1 : pos_hi;            // the last row of the tile's store that is seen
     if (key0 + PF_BK - 1 > last_row) {
@@ -208,6 +222,10 @@ attention_prefill_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, con
 #if LLMX_SCORE_CAP
         s[j][e] = v0 ? capped_score_log2(cap, s[j][e]) : -INFINITY;
         s[j][2 + e] = v1 ? capped_score_log2(cap, s[j][2 + e]) : -INFINITY;
+#elif LLMX_SCORE_BIAS
+        const float* wb = wbias + (lane >> 2) + PF_BK - 1 - (key - key0);
+        s[j][e] = v0 ? fmaf(s[j][e], scale_log2, wb[0]) : -INFINITY;
+        s[j][2 + e] = v1 ? fmaf(s[j][2 + e], scale_log2, wb[8]) : -INFINITY;
 #else
         s[j][e] = v0 ? s[j][e] * scale_log2 : -INFINITY;
         s[j][2 + e] = v1 ? s[j][2 + e] * scale_log2 : -INFINITY;
@@ -296,8 +314,9 @@ static int launch_prefill_as(const void* q, void* out, const void* k_cache, cons
                           int table_width, const int* seq_start, const int* seq_past, int B, int max_new, int H,
                           int G, int window, int keep_first, int mask_chunk, float scale, float sink, int pool,
                           const void* pool_k, const void* pool_v, const int* pool_table, const float* sinks,
-                          float softcap, cudaStream_t stream) {
-  const size_t smem = (size_t)PF_BQ * D * 2 + 4 * (size_t)PF_BK * D * 2;
+                          float softcap, const float* score_bias, int bias_len, cudaStream_t stream) {
+  const size_t smem = (size_t)PF_BQ * D * 2 + 4 * (size_t)PF_BK * D * 2 +
+                      (LLMX_SCORE_BIAS ? (PF_THREADS / 32) * PF_BIAS * sizeof(float) : 0);
   auto kernel = attention_prefill_kernel<D, POOLED>;
   static bool attr_set = false;
   if (!attr_set && smem > 48 * 1024) {
@@ -310,13 +329,13 @@ static int launch_prefill_as(const void* q, void* out, const void* k_cache, cons
                                              block_table, table_width, seq_start, seq_past, H, G, window,
                                              keep_first, mask_chunk, scale * 1.4426950408889634f, sink, pool,
                                              (const bf16*)pool_k, (const bf16*)pool_v, pool_table, sinks,
-                                             make_score_cap(scale, softcap));
+                                             make_score_cap(scale, softcap), make_score_bias(score_bias, bias_len));
   return LLMX_LAUNCH_STATUS();
 }
 
 template <int D, typename... Args>
 static int launch_prefill(int pool, Args... args) {
-#if !LLMX_SCORE_CAP            // (pooled blocks beside capped scores are not built)
+#if !LLMX_SCORE_CAP && !LLMX_SCORE_BIAS     // (pooled blocks beside capped or biased scores are not built)
   if (pool > 0) return launch_prefill_as<D, true>(args...);
 #endif
   return launch_prefill_as<D, false>(args...);
@@ -330,15 +349,18 @@ static int launch_prefill(int pool, Args... args) {
 // pool n > 0 (beside a window, without kept first keys or a chunked mask): every block of n positions that lies
 // wholly before a query's window is seen as row b of pool_k / pool_v, a second store paged like the cache with the
 // block table pool_table (as wide as block_table).
-// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it.
-LLMX_API int llmx_attention_prefill_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
+// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it;
+// score_bias: float32 [H, bias_len] in the library with LLMX_SCORE_BIAS, null in the others.
+LLMX_API int llmx_attention_prefill_biased(const void* q, void* out, const void* k_cache, const void* v_cache,
                                            const int* block_table, int table_width, const int* seq_start,
                                            const int* seq_past, int B, int max_new, int H, int G, int D, int window,
                                            int keep_first, int mask_chunk, float scale, float sink, int pool,
                                            const void* pool_k, const void* pool_v, const int* pool_table,
-                                           const float* sinks, float softcap, cudaStream_t stream) {
+                                           const float* sinks, float softcap, const float* score_bias, int bias_len,
+                                           cudaStream_t stream) {
   if (B <= 0 || max_new <= 0) return 0;
-  if ((softcap > 0.f) != (LLMX_SCORE_CAP != 0) || (LLMX_SCORE_CAP && pool > 0)) return LLMX_REFUSED(1);
+  if ((softcap > 0.f) != (LLMX_SCORE_CAP != 0) || ((LLMX_SCORE_CAP || LLMX_SCORE_BIAS) && pool > 0)) return LLMX_REFUSED(1);
+  if ((score_bias != nullptr) != (LLMX_SCORE_BIAS != 0) || (score_bias && bias_len <= 0)) return LLMX_REFUSED(1);
   if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || mask_chunk > 0 || !pool_k || !pool_v || !pool_table ||
                                 ((uintptr_t)pool_k & 15) || ((uintptr_t)pool_v & 15))))
     return LLMX_REFUSED(1);
@@ -349,12 +371,23 @@ LLMX_API int llmx_attention_prefill_capped(const void* q, void* out, const void*
   if (D == 128)
     return launch_prefill<128>(pool, q, out, k_cache, v_cache, block_table, table_width, seq_start, seq_past, B, max_new,
                                H, G, window, window > 0 ? keep_first : 0, mask_chunk, scale, sink, pool, pool_k, pool_v,
-                               pool_table, sinks, softcap, stream);
+                               pool_table, sinks, softcap, score_bias, bias_len, stream);
   if (D == 64)
     return launch_prefill<64>(pool, q, out, k_cache, v_cache, block_table, table_width, seq_start, seq_past, B, max_new, H,
                               G, window, window > 0 ? keep_first : 0, mask_chunk, scale, sink, pool, pool_k, pool_v,
-                              pool_table, sinks, softcap, stream);
+                              pool_table, sinks, softcap, score_bias, bias_len, stream);
   return LLMX_REFUSED(1);
+}
+
+LLMX_API int llmx_attention_prefill_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
+                                           const int* block_table, int table_width, const int* seq_start,
+                                           const int* seq_past, int B, int max_new, int H, int G, int D, int window,
+                                           int keep_first, int mask_chunk, float scale, float sink, int pool,
+                                           const void* pool_k, const void* pool_v, const int* pool_table,
+                                           const float* sinks, float softcap, cudaStream_t stream) {
+  return llmx_attention_prefill_biased(q, out, k_cache, v_cache, block_table, table_width, seq_start, seq_past, B,
+                                       max_new, H, G, D, window, keep_first, mask_chunk, scale, sink, pool, pool_k, pool_v,
+                                       pool_table, sinks, softcap, nullptr, 0, stream);
 }
 
 LLMX_API int llmx_attention_prefill_pooled(const void* q, void* out, const void* k_cache, const void* v_cache,

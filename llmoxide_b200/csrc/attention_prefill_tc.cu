@@ -33,6 +33,9 @@
 //
 // Compiled a second time with LLMX_SCORE_CAP=1 (a library of its own) every scaled score is capped (common.cuh).
 // `sinks` (float32 [H]): exp(sinks[h]) joins head h's denominator once.
+// Compiled a third time with LLMX_SCORE_BIAS=1 a learned bias per distance and head joins every scaled score (common.cuh): a
+// softmax warp's 32 rows and a tile's 64 keys span 95 distances, which it copies to shared memory while it waits for the
+// tile's scores; lane r then reads entry r + 63 - e for key e, 32 neighbouring words a load.
 #include "tc_ptx.cuh"
 
 #define AT_ROWS 128        // query rows per CTA = MMA M
@@ -43,7 +46,9 @@
 #define AT_TILE (2 * AT_PANEL) // bytes of the [128 x 128] query tile
 #define AT_KPANEL (AT_KEYS * 128)   // bytes of one [64 keys x 64 dims] panel of K or V
 #define AT_KTILE (2 * AT_KPANEL)    // bytes of a [64 keys x 128 dims] tile of K or V
-#define AT_SMEM (AT_TILE + 4 * AT_KTILE + 16 * 8 + 64)   // Q, K[2], V[2], barriers
+#define AT_BIAS 96                  // distances between a warp's rows and a tile's keys (95), padded
+#define AT_BARS (16 * 8 + 64)
+#define AT_SMEM (AT_TILE + 4 * AT_KTILE + AT_BARS + (LLMX_SCORE_BIAS ? 4 * AT_BIAS * 4 : 0))   // Q, K[2], V[2], barriers
 
 __device__ int g_at_status = 0;    // 0, or which bounded wait ran out (1..10 below), 20: shared memory not 1024-byte aligned
 __device__ __forceinline__ void at_report(int code) {
@@ -64,9 +69,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ block_table, int table_width, const int* __restrict__ seq_start,
                             const int* __restrict__ seq_past, int H, int G, int window, int keep_first,
                             int mask_chunk, float scale_log2_arg, float sink, const float* __restrict__ sinks,
-                            const ScoreCap cap) {
-#if LLMX_SCORE_CAP
-  constexpr float scale_log2 = 1.0f;           // the capped scores are base-2 logarithms already
+                            const ScoreCap cap, const ScoreBiasArg bias) {
+#if LLMX_SCORE_CAP || LLMX_SCORE_BIAS
+  constexpr float scale_log2 = 1.0f;           // the capped or biased scores are base-2 logarithms already
 #else
   const float scale_log2 = scale_log2_arg;
 #endif
@@ -215,8 +220,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     float m_used = -INFINITY;      // the maximum the exponentials are taken against (may lag the true one)
     float l = 0.f;                 // row sum in units of 2^-m_used
     bool ok = true;
+#if LLMX_SCORE_BIAS
+    float* wbias = reinterpret_cast<float*>(pV0 + 2 * AT_KTILE + AT_BARS) + (warp - 2) * AT_BIAS;
+    const float* brow = bias.table + (size_t)hq * bias.len;
+#endif
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int st = j & 1;
+#if LLMX_SCORE_BIAS
+      __syncwarp();                 // (every lane has read the tile before's)
+      {
+        const int d0 = past + i0 + quad * 32 - (tile_at(j) * AT_KEYS + AT_KEYS - 1);
+#pragma unroll
+        for (int i = 0; i < AT_BIAS; i += 32)
+          wbias[i + lane] = brow[min(max(d0 + i + lane, 0), bias.len - 1)] * LLMX_LOG2E;
+      }
+      __syncwarp();
+#endif
       ok = mbar_wait(s_full0 + 8u * st, (j >> 1) & 1);
       if (!ok && lane == 0) at_report(7);
       ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
@@ -232,6 +251,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #if LLMX_SCORE_CAP
 #pragma unroll
       for (int e = 0; e < AT_KEYS; ++e) sr[e] = __float_as_uint(capped_score_log2(cap, __uint_as_float(sr[e])));
+#endif
+#if LLMX_SCORE_BIAS
+      {
+        const float* wb = wbias + lane + AT_KEYS - 1;
+#pragma unroll
+        for (int e = 0; e < AT_KEYS; ++e)
+          sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2_arg, wb[-e]));
+      }
 #endif
       // Tiles that some row of this CTA sees only in part (the diagonal, a window's edge, rows past the
       // sequence's end) are masked; the others, which is most of them, skip the compares.
@@ -365,15 +392,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 // max_new = most new tokens of a sequence.
 // mask_chunk n > 0: a query sees only the keys of its own chunk of n positions, counted from the sequence's
 // position 0 (no kept first keys then).
-// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it.
-LLMX_API int llmx_attention_prefill_tc_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
+// sinks: null, or float32 [H]; softcap: 0 in the library without LLMX_SCORE_CAP, positive in the one with it;
+// score_bias: float32 [H, bias_len] in the library with LLMX_SCORE_BIAS, null in the others.
+LLMX_API int llmx_attention_prefill_tc_biased(const void* q, void* out, const void* k_cache, const void* v_cache,
                                               long long n_pages, const int* block_table, int table_width,
                                               const int* seq_start, const int* seq_past, int B, int T, int max_new,
                                               int H, int G, int D, int window, int keep_first, int mask_chunk,
                                               float scale, float sink, const float* sinks, float softcap,
-                                              cudaStream_t stream) {
+                                              const float* score_bias, int bias_len, cudaStream_t stream) {
   if (B <= 0 || max_new <= 0 || T <= 0) return 0;
   if ((softcap > 0.f) != (LLMX_SCORE_CAP != 0)) return LLMX_REFUSED(1);
+  if ((score_bias != nullptr) != (LLMX_SCORE_BIAS != 0) || (score_bias && bias_len <= 0)) return LLMX_REFUSED(1);
   if (window <= 0) keep_first = 0;
   if (mask_chunk < 0 || (mask_chunk > 0 && keep_first > 0)) return LLMX_REFUSED(1);
   if (D != AT_D || H <= 0 || G <= 0 || H % G || window < 0 || keep_first < 0 || B > 65535 || (max_new + AT_ROWS - 1) / AT_ROWS > 65535 || n_pages <= 0)
@@ -399,8 +428,19 @@ LLMX_API int llmx_attention_prefill_tc_capped(const void* q, void* out, const vo
   dim3 grid(H, (max_new + AT_ROWS - 1) / AT_ROWS, B);
   launch_pdl(attention_prefill_tc_kernel, grid, dim3(AT_THREADS), smem, stream, mq, mk, mv, (bf16*)out, block_table,
              table_width, seq_start, seq_past, H, G, window, keep_first, mask_chunk, scale * 1.4426950408889634f, sink,
-             sinks, make_score_cap(scale, softcap));
+             sinks, make_score_cap(scale, softcap), make_score_bias(score_bias, bias_len));
   return LLMX_LAUNCH_STATUS();
+}
+
+LLMX_API int llmx_attention_prefill_tc_capped(const void* q, void* out, const void* k_cache, const void* v_cache,
+                                              long long n_pages, const int* block_table, int table_width,
+                                              const int* seq_start, const int* seq_past, int B, int T, int max_new,
+                                              int H, int G, int D, int window, int keep_first, int mask_chunk,
+                                              float scale, float sink, const float* sinks, float softcap,
+                                              cudaStream_t stream) {
+  return llmx_attention_prefill_tc_biased(q, out, k_cache, v_cache, n_pages, block_table, table_width, seq_start, seq_past,
+                                          B, T, max_new, H, G, D, window, keep_first, mask_chunk, scale, sink, sinks,
+                                          softcap, nullptr, 0, stream);
 }
 
 LLMX_API int llmx_attention_prefill_tc_masked(const void* q, void* out, const void* k_cache, const void* v_cache,

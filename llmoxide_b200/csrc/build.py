@@ -43,7 +43,12 @@ LIBRARIES = {
     "attention_decode_capped": (["attention_decode.cu"], ["-DLLMX_SCORE_CAP=1"]),
     "attention_prefill_capped": (["attention_prefill.cu"], ["-DLLMX_SCORE_CAP=1"]),
     "attention_prefill_tc_capped": (["attention_prefill_tc.cu"], ["-DLLMX_SCORE_CAP=1"]),
+    # and once with a learned bias per distance and head on every score
+    "attention_decode_biased": (["attention_decode.cu"], ["-DLLMX_SCORE_BIAS=1"]),
+    "attention_prefill_biased": (["attention_prefill.cu"], ["-DLLMX_SCORE_BIAS=1"]),
+    "attention_prefill_tc_biased": (["attention_prefill_tc.cu"], ["-DLLMX_SCORE_BIAS=1"]),
     "delta_rule": (["delta_rule.cu"], []),
+    "dual_norm": (["dual_norm.cu"], []),
     "gemm_fma": (["gemm_fma.cu"], []),
     "gemm_tc": (["gemm_tc.cu"], []),
     "linear_attention": (["linear_attention.cu"], []),
@@ -52,6 +57,8 @@ LIBRARIES = {
     "moe": (["moe.cu"], []),
     "post_norm": (["post_norm.cu"], []),
     "qk_row_norm": (["qk_row_norm.cu"], []),
+    "qk_unit": (["qk_unit.cu"], []),
+    "state_space": (["state_space.cu"], []),
     "moe_tc": (["moe_tc.cu"], []),
     "short_conv": (["short_conv.cu"], []),
     "stream_mix": (["stream_mix.cu"], []),

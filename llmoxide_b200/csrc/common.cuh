@@ -221,13 +221,35 @@ static inline ScoreCap make_score_cap(float scale, float softcap) {
   return c;
 }
 
+// Learned score biases.  The tiled attention kernels are compiled once more with LLMX_SCORE_BIAS 1 (a third library):
+// table[h * len + min(p - j, len - 1)] joins the scaled score of head h between the query at position p and the key at j.
+// The other builds' kernels take the empty form.
+#ifndef LLMX_SCORE_BIAS
+#define LLMX_SCORE_BIAS 0
+#endif
+struct ScoreBias {
+  const float* table;      // float32 [H, len], natural units
+  int len;
+};
+struct NoScoreBias {};
+#if LLMX_SCORE_BIAS
+typedef ScoreBias ScoreBiasArg;
+static inline ScoreBiasArg make_score_bias(const float* table, int len) { return ScoreBias{table, len}; }
+#else
+typedef NoScoreBias ScoreBiasArg;
+static inline ScoreBiasArg make_score_bias(const float*, int) { return NoScoreBias{}; }
+#endif
+#define LLMX_LOG2E 1.4426950408889634f
+
 // Gated activations of the feed-forwards, act(g) * f(u):
 //   SILU            g sigmoid(g) * u
 //   RELU            max(g, 0) * u
 //   CLAMPED_SWISH   g' sigmoid(slope g') * (u' + shift),  g' = min(g, limit),  u' = clamp(u, -limit, limit)
 //   GELU_TANH       0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u
-enum { LLMX_ACT_SILU = 0, LLMX_ACT_RELU = 1, LLMX_ACT_CLAMPED_SWISH = 2, LLMX_ACT_GELU_TANH = 3 };
-#define LLMX_ACT_LAST LLMX_ACT_GELU_TANH
+//   RELU_SQUARED    max(g, 0)^2 * u
+// A feed-forward without a gate applies the same function with u = 1.
+enum { LLMX_ACT_SILU = 0, LLMX_ACT_RELU = 1, LLMX_ACT_CLAMPED_SWISH = 2, LLMX_ACT_GELU_TANH = 3, LLMX_ACT_RELU_SQUARED = 4 };
+#define LLMX_ACT_LAST LLMX_ACT_RELU_SQUARED
 struct GateAct {
   int kind;
   float slope, limit, shift;
@@ -237,6 +259,7 @@ struct GateAct {
 __device__ __forceinline__ float gated_act(const GateAct a, float g, float u) {
   if (a.kind == LLMX_ACT_SILU) return (g / (1.0f + expf(-g))) * u;
   if (a.kind == LLMX_ACT_RELU) return fmaxf(g, 0.f) * u;
+  if (a.kind == LLMX_ACT_RELU_SQUARED) return fmaxf(g, 0.f) * fmaxf(g, 0.f) * u;
   if (a.kind == LLMX_ACT_GELU_TANH) return (0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)))) * u;
   g = fminf(g, a.limit);
   u = fminf(fmaxf(u, -a.limit), a.limit);
@@ -246,6 +269,7 @@ __device__ __forceinline__ float gated_act(const GateAct a, float g, float u) {
 __device__ __forceinline__ float gated_act_fast(const GateAct a, float g, float u) {
   if (a.kind == LLMX_ACT_SILU) return __fdividef(g, 1.0f + __expf(-g)) * u;
   if (a.kind == LLMX_ACT_RELU) return fmaxf(g, 0.f) * u;
+  if (a.kind == LLMX_ACT_RELU_SQUARED) return fmaxf(g, 0.f) * fmaxf(g, 0.f) * u;
   if (a.kind == LLMX_ACT_GELU_TANH) {       // 0.5 (1 + tanh z) = 1 / (1 + exp(-2z))
     const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return __fdividef(g, 1.0f + __expf(-2.0f * z)) * u;

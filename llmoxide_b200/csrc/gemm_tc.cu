@@ -63,6 +63,7 @@ __host__ __device__ constexpr uint32_t umma_idesc(int n) {
 //         columns brings the two together (the lower lanes finish the even columns, the upper lanes the odd
 //         ones), and no warp waits for another.  A tile of 128 rows gives 64 features:
 //         out[t, n0/2 + 16 * quad + lane % 16] = silu(gate) * up.
+// MODE 3: out[t, n] = act(acc), the activation of a feed-forward without a gate.
 // ---------------------------------------------------------------------------
 #define TC_FUSE_BYTES (64 * 4)                    // row scales
 
@@ -112,7 +113,8 @@ __device__ __forceinline__ void epilogue_tile(uint32_t acc_addr, bool have_acc, 
         const int t = t0 + c + e;
         if (t < T) {
           float r = v[e];
-          if (MODE != 0) r = gated_act_fast(act, r, g[e]);
+          if (MODE == 1) r = gated_act_fast(act, r, g[e]);
+          if (MODE == 3) r = gated_act_fast(act, r, 1.0f);
           out[(size_t)t * ldy + n] = from_f32<TY>(r);
         }
       }
@@ -162,7 +164,7 @@ __device__ __forceinline__ void epilogue_tile_staged(uint32_t acc_addr, const CU
       }
     } else {
 #pragma unroll
-      for (int e = 0; e < ROWS; ++e) buf[e * COLS + col] = from_f32<TY>(v[e]);
+      for (int e = 0; e < ROWS; ++e) buf[e * COLS + col] = from_f32<TY>(MODE == 3 ? gated_act_fast(act, v[e], 1.0f) : v[e]);
     }
     fence_proxy_async();
     asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -183,6 +185,7 @@ __device__ __forceinline__ void epilogue_tile_staged(uint32_t acc_addr, const CU
 // sets, so the epilogue of a unit overlaps the MMAs of the next.
 // MODE 0: Y (bf16 or f32) [T, N] or split partials f32 [n_split][T, N].
 // MODE 1: two accumulators, rows n and n + F of W; act[T, F] = silu(g) * u.
+// MODE 3: Y (bf16) [T, N] = act(product).
 // ---------------------------------------------------------------------------
 template <int BN, int MODE, typename TY>
 __global__ void __launch_bounds__(TC_THREADS)
@@ -330,7 +333,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
   } else {
     // ---------------- epilogue ----------------
     const int quad = warp & 3;          // the quarter of tensor memory this warp may read
-    const int n_limit = MODE == 0 ? N : F;
+    const int n_limit = MODE == 0 || MODE == 3 ? N : F;
     bool waited = false, failed = false;
     const float* row_scale = nullptr;
     if (sc.sumsq) {
@@ -634,7 +637,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
   } else {
     // ---------------- epilogue (both CTAs) ----------------
     const int quad = warp & 3;
-    const int n_limit = MODE == 0 ? N : F;
+    const int n_limit = MODE == 0 || MODE == 3 ? N : F;
     bool failed = false;
     int j = 0, chunk_no = 0;
     for (int u = pair; u < n_units; u += n_pairs, ++j) {
@@ -748,6 +751,7 @@ static int launch(const CUtensorMap& mw, const CUtensorMap& mx, void* Y, int T, 
 // mode 1: W = [gate rows; up rows] with N = 2F; Y = act [T,F] of y_dtype.
 // mode 2: W = blocks of 32 rows, each 16 gate rows then the 16 up rows of the same features (N = 2F, F % 16 == 0);
 //         Y = act [T,F] bf16.
+// mode 3: Y [T,N] bf16 = act(product), act as for a gate with up = 1.
 // The same with row scales applied in the epilogue (see TcScale): in_sumsq [in_parts][in_stride >= T], T <= 64.
 LLMX_API int llmx_gemm_tc_scaled(const void* X, const void* W, void* Y, int y_dtype, int T, int N, int K, long long ldx,
                                  long long ldw, long long ldy, int n_split, long long split_stride, int mode,
@@ -773,8 +777,8 @@ LLMX_API int llmx_gemm_tc_scaled(const void* X, const void* W, void* Y, int y_dt
   }
   if (K <= 0 || (K % 8) || (ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return LLMX_REFUSED(1);
   if (n_split < 1 || (n_split > 1 && (mode != 0 || y_dtype != LLMX_F32))) return LLMX_REFUSED(1);
-  if (mode < 0 || mode > 2 || (mode == 1 && (N % 2)) || (mode == 2 && (N % 32))) return LLMX_REFUSED(1);
-  const int F = mode != 0 ? N / 2 : 0;
+  if (mode < 0 || mode > 3 || (mode == 1 && (N % 2)) || (mode == 2 && (N % 32))) return LLMX_REFUSED(1);
+  const int F = mode == 1 || mode == 2 ? N / 2 : 0;
   int bn = 16;
   while (bn < T && bn < (mode == 1 ? 128 : 256)) bn <<= 1;
   CUtensorMap mw, mx;
@@ -801,6 +805,7 @@ LLMX_API int llmx_gemm_tc_scaled(const void* X, const void* W, void* Y, int y_dt
     }
   }
   if (mode == 2 && y_dtype == LLMX_BF16) { BY_BN(2, bf16) }
+  if (mode == 3 && y_dtype == LLMX_BF16) { BY_BN(3, bf16) }
 #undef BY_BN
 #undef GO
   return LLMX_REFUSED(2);
@@ -892,8 +897,8 @@ LLMX_API int llmx_gemm_tc_pair(const void* X, const void* W, void* Y, int y_dtyp
                                long long split_stride, cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || (K % 8) || (ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return LLMX_REFUSED(1);
-  if (T <= 128 || mode < 0 || mode > 2 || (mode == 1 && (N % 2)) || (mode == 2 && (N % 32))) return LLMX_REFUSED(1);
-  const int F = mode != 0 ? N / 2 : 0;
+  if (T <= 128 || mode < 0 || mode > 3 || (mode == 1 && (N % 2)) || (mode == 2 && (N % 32))) return LLMX_REFUSED(1);
+  const int F = mode == 1 || mode == 2 ? N / 2 : 0;
   const int bn = mode == 1 ? 128 : 256;
   CUtensorMap mw, mx;
   if (make_map(&mw, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, TC_BM, true)) return LLMX_REFUSED(4);
@@ -905,6 +910,7 @@ LLMX_API int llmx_gemm_tc_pair(const void* X, const void* W, void* Y, int y_dtyp
     return launch_pair<256, 0, float>(mw, mx, Y, T, N, K, ldy, F, accumulate, n_split, split_stride, stream);
   if (mode == 1 && y_dtype == LLMX_BF16) return launch_pair<128, 1, bf16>(mw, mx, Y, T, N, K, ldy, F, 0, 1, 0, stream);
   if (mode == 2 && y_dtype == LLMX_BF16) return launch_pair<256, 2, bf16>(mw, mx, Y, T, N, K, ldy, F, 0, 1, 0, stream);
+  if (mode == 3 && y_dtype == LLMX_BF16) return launch_pair<256, 3, bf16>(mw, mx, Y, T, N, K, ldy, F, 0, 1, 0, stream);
   return LLMX_REFUSED(2);
 }
 

@@ -369,10 +369,11 @@ LLMX_API int llmx_moe_sort(const int* ids, const float* pair_weight, int P, int 
 //
 // GATED: rows are tokens' rows of x gathered through perm (token = pair / top); W = [E][2F][K], gate rows then
 //   up rows; out act[place][f] = gated_act(gate, up) (common.cuh), in sorted order.
+// PLAIN: the same rows; W = [E][F][K]; out act[place][f] = the activation of an expert without a gate.
 // else:  rows are act[place]; W = [E][N][K]; out y[choice][token][n] = weight[pair] * sum, float32: one partial
 //   per choice, which whoever adds them to the residual stream sums in the order of the choices.
 // ---------------------------------------------------------------------------
-template <typename TX, typename TW, typename TY, bool GATED>
+template <typename TX, typename TW, typename TY, bool GATED, bool PLAIN>
 __global__ void __launch_bounds__(256)
 moe_grouped_fma_kernel(const TX* __restrict__ X, long long ldx, const TW* __restrict__ W, TY* __restrict__ Y,
                        const int* __restrict__ perm, const int* __restrict__ tiles,
@@ -395,7 +396,7 @@ moe_grouped_fma_kernel(const TX* __restrict__ X, long long ldx, const TW* __rest
   __syncthreads();
   const int pair = row_src[lrow];
   const TX* xrow = nullptr;
-  if (pair >= 0) xrow = GATED ? X + (size_t)(pair / top) * ldx : X + (size_t)(row0 + lrow) * ldx;
+  if (pair >= 0) xrow = GATED || PLAIN ? X + (size_t)(pair / top) * ldx : X + (size_t)(row0 + lrow) * ldx;
   const size_t w_rows = GATED ? 2 * (size_t)N : (size_t)N;
   const TW* We = W + (size_t)e * w_rows * K;
   const int n_load = n0 + lrow;
@@ -450,6 +451,8 @@ moe_grouped_fma_kernel(const TX* __restrict__ X, long long ldx, const TW* __rest
       if (n >= N) continue;
       if constexpr (GATED) {
         Y[(size_t)(row0 + lr) * N + n] = from_f32<TY>(gated_act(act, acc[i][j], acu[i][j]));
+      } else if constexpr (PLAIN) {
+        Y[(size_t)(row0 + lr) * N + n] = from_f32<TY>(gated_act(act, acc[i][j], 1.0f));
       } else {
         const int t = pr / top, choice = pr - t * top;
         Y[((size_t)choice * n_tokens + t) * N + n] = from_f32<TY>(pair_weight[pr] * acc[i][j]);
@@ -458,8 +461,8 @@ moe_grouped_fma_kernel(const TX* __restrict__ X, long long ldx, const TW* __rest
   }
 }
 
-// gated != 0: X = x [n_tokens, K] (row stride ldx), W [E, 2N, K], Y = act [P, N].
-// else:       X = act [P, K], W [E, N, K], Y = float32 [top, n_tokens, N].
+// gated 1: X = x [n_tokens, K] (row stride ldx), W [E, 2N, K], Y = act [P, N]; gated 2: W [E, N, K] without a gate.
+// gated 0:       X = act [P, K], W [E, N, K], Y = float32 [top, n_tokens, N].
 // The tile list must have been made with MOE_TILE rows per tile.
 LLMX_API int llmx_moe_grouped_fma(const void* X, int x_dtype, long long ldx, const void* W, int w_dtype, void* Y,
                                   int y_dtype, const int* perm, const int* tiles, int max_tiles,
@@ -471,17 +474,23 @@ LLMX_API int llmx_moe_grouped_fma(const void* X, int x_dtype, long long ldx, con
   if (N <= 0 || K <= 0 || top <= 0 || max_tiles <= 0 || max_tiles > 65535 || ldx < K) return LLMX_REFUSED(1);
   if (x_dtype != w_dtype) return LLMX_REFUSED(2);
   dim3 grid((N + MOE_TILE - 1) / MOE_TILE, max_tiles);
-#define GO(TX, TY, G)                                                                                          \
-  launch_pdl(moe_grouped_fma_kernel<TX, TX, TY, G>, grid, dim3(256), 0, stream, (const TX*)X, ldx, (const TX*)W, \
+#define GO(TX, TY, G, P)                                                                                       \
+  launch_pdl(moe_grouped_fma_kernel<TX, TX, TY, G, P>, grid, dim3(256), 0, stream, (const TX*)X, ldx, (const TX*)W, \
              (TY*)Y, perm, tiles, pair_weight, top, n_tokens, N, K, act)
   if (gated) {
-    if (x_dtype == LLMX_F32 && y_dtype == LLMX_F32) GO(float, float, true);
-    else if (x_dtype == LLMX_BF16 && y_dtype == LLMX_BF16) GO(bf16, bf16, true);
-    else return LLMX_REFUSED(2);
+    if (gated < 0 || gated > 2) return LLMX_REFUSED(1);
+    const bool plain = gated == 2;
+    if (x_dtype == LLMX_F32 && y_dtype == LLMX_F32) {
+      if (plain) GO(float, float, false, true); else GO(float, float, true, false);
+    } else if (x_dtype == LLMX_BF16 && y_dtype == LLMX_BF16) {
+      if (plain) GO(bf16, bf16, false, true); else GO(bf16, bf16, true, false);
+    } else {
+      return LLMX_REFUSED(2);
+    }
   } else {
     if (y_dtype != LLMX_F32) return LLMX_REFUSED(2);
-    if (x_dtype == LLMX_F32) GO(float, float, false);
-    else if (x_dtype == LLMX_BF16) GO(bf16, float, false);
+    if (x_dtype == LLMX_F32) GO(float, float, false, false);
+    else if (x_dtype == LLMX_BF16) GO(bf16, float, false, false);
     else return LLMX_REFUSED(2);
   }
 #undef GO

@@ -13,6 +13,7 @@
 //
 //   MODE 1 (gate|up): two accumulators, rows n and n + F of the expert's [2F, K]; act[row, n] = gated_act(gate, up) (common.cuh)
 //   MODE 0 (down):    y[dest[row]][n] = weight[row] * acc, float32 (dest = choice * tokens + token, from the sort)
+//   MODE 2 (up):      act[row, n] = the activation of an expert without a gate (gated_act with up = 1)
 //
 // Which expert a unit reads is decided on the device by the kernel before, so every thread waits for that
 // kernel first.  Every wait on an mbarrier is bounded; when one runs out the CTA records it in the library's
@@ -196,6 +197,8 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
             if (r >= n_rows) break;
             if (MODE == 1) {
               Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(gated_act_fast(act, v[i], g[i]));
+            } else if (MODE == 2) {
+              Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(gated_act_fast(act, v[i], 1.0f));
             } else {
               Y[(size_t)tile_dest[r] * N + n] = from_f32<TY>(tile_weight[r] * v[i]);
             }
@@ -254,9 +257,9 @@ static int mt_launch(const CUtensorMap& mw, const CUtensorMap& mx, void* Y, cons
   return LLMX_LAUNCH_STATUS();
 }
 
-// X: bf16 sorted rows [P, K] (row stride ldx); W: bf16 [E, w_rows, K] contiguous, w_rows = 2N when gated (gate rows,
+// X: bf16 sorted rows [P, K] (row stride ldx); W: bf16 [E, w_rows, K] contiguous, w_rows = 2N when gated is 1 (gate rows,
 // then up rows) else N; tiles: int32 [max_tiles, 3] made with tile_rows rows per tile (16, 64 or 128).
-// gated: Y = act bf16 [P, N].  else: Y = float32 rows of N, row dest[place] = sorted_weight[place] * product
+// gated 1: Y = act bf16 [P, N]; gated 2 (experts without a gate): W [E, N, K], Y = act(product) bf16 [P, N].  0: Y = float32 rows of N, row dest[place] = sorted_weight[place] * product
 // (dest and sorted_weight [P] in sorted order, from the sort).
 LLMX_API int llmx_moe_grouped_tc(const void* X, long long ldx, long long P, const void* W, int n_experts, void* Y,
                                  const int* tiles, int max_tiles, int tile_rows, const int* dest,
@@ -268,12 +271,14 @@ LLMX_API int llmx_moe_grouped_tc(const void* X, long long ldx, long long P, cons
   if (N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || max_tiles <= 0 ||
       n_experts <= 0 || (!gated && (!dest || !sorted_weight)))
     return LLMX_REFUSED(1);
-  const int w_rows = gated ? 2 * N : N;
+  if (gated < 0 || gated > 2) return LLMX_REFUSED(1);
+  const int w_rows = gated == 1 ? 2 * N : N;
   CUtensorMap mw, mx;
   if (make_map(&mw, W, (uint64_t)n_experts * w_rows, (uint64_t)K, (uint64_t)K, MT_BM, true)) return LLMX_REFUSED(4);
   if (make_map(&mx, X, (uint64_t)P, (uint64_t)K, (uint64_t)ldx, (uint32_t)tile_rows, false)) return LLMX_REFUSED(4);
 #define GO(BN)                                                                                                      \
-  return gated ? mt_launch<BN, 1, bf16>(mw, mx, Y, tiles, max_tiles, dest, sorted_weight, N, K, w_rows, act, stream) \
+  return gated == 1 ? mt_launch<BN, 1, bf16>(mw, mx, Y, tiles, max_tiles, dest, sorted_weight, N, K, w_rows, act, stream) \
+       : gated == 2 ? mt_launch<BN, 2, bf16>(mw, mx, Y, tiles, max_tiles, dest, sorted_weight, N, K, w_rows, act, stream) \
                : mt_launch<BN, 0, float>(mw, mx, Y, tiles, max_tiles, dest, sorted_weight, N, K, w_rows, act, stream)
   switch (tile_rows) {
     case 16: GO(16);

@@ -124,7 +124,8 @@ def _library(lib_name: str):
 _STATUS_SLOTS = {"gemm_tc": 0, "attention_prefill_tc": 1, "attention_decode": 2, "sampling": 3, "moe_tc": 4,
                  "short_conv": 5, "stream_mix": 6, "moe": 7, "attention": 8, "latent_attention": 9,
                  "attention_prefill_tc_capped": 10, "attention_decode_capped": 11, "qk_row_norm": 12, "delta_rule": 13,
-                 "latent_cache": 14}
+                 "latent_cache": 14, "attention_prefill_tc_biased": 15, "attention_decode_biased": 16, "qk_unit": 17,
+                 "state_space": 18}
 _STATUS_MEANING = {
     "gemm_tc": {1: "the producer's wait for a free stage ran out", 2: "the MMA issuer's wait for a stage's data ran out",
                 3: "the epilogue's wait for an accumulator ran out", 4: "the MMA issuer's wait for a drained accumulator ran out",
@@ -155,9 +156,13 @@ _STATUS_MEANING = {
                    3: "a sequence's rows or slot lie outside the launch's arrays (convolution rows)",
                    4: "a sequence's position or slot lies outside the launch's arrays (single tokens)",
                    5: "a chunk's copy into shared memory never completed"},
+    "qk_unit": {1: "a token's sequence, position or page lies outside the launch's arrays"},
+    "state_space": {1: "a sequence's rows or slot lie outside the launch's arrays (preparation)",
+                    2: "a sequence's rows or slot lie outside the launch's arrays (states)",
+                    3: "a sequence's position or slot lies outside the launch's arrays (single tokens)"},
 }
-for _capped in ("attention_prefill_tc", "attention_decode"):
-    _STATUS_MEANING[_capped + "_capped"] = _STATUS_MEANING[_capped]
+for _tiled in ("attention_prefill_tc", "attention_decode"):
+    _STATUS_MEANING[_tiled + "_capped"] = _STATUS_MEANING[_tiled + "_biased"] = _STATUS_MEANING[_tiled]
 _status_host = None
 
 
@@ -470,6 +475,37 @@ def post_norm_add_norm(h, groups, bias, post_gain, post_center: bool, post_eps: 
            "post_norm_add_norm")
 
 
+def dual_norm(h, groups, bias, gain0, eps: float, out0, gain1=None, out1=None, rows=None, write_h: bool = True) -> None:
+    """h float32 [T, d] += what up to two sublayers owe the stream together, and one or two RMS norms of it that share
+    their root mean square: ``groups``: up to two tensors [T, d] or split partials [S, T, d], added in order; ``bias``
+    float32 [d] or None; out0[r] = norm(h[rows[r]]) * gain0 (every row without ``rows``), out1 likewise with gain1;
+    ``out0`` None: only the sum."""
+    _dev(h, bias, gain0, gain1, out0, out1, rows, *groups)
+    assert h.dtype == torch.float32 and h.dim() == 2 and len(groups) <= 2
+    _contig("h", h)
+    d = h.shape[1]
+    args = []
+    for g in groups:
+        _contig("delta", g)
+        if g.dim() == 2:
+            g = g.unsqueeze(0)
+        assert g.shape[1:] == h.shape, (g.shape, h.shape)
+        args += [_ptr(g), _tag(g), g.shape[0], g.stride(0)]
+    args += [None, F32, 1, 0] * (2 - len(groups))
+    for v in (bias, gain0, gain1):
+        assert v is None or (v.dtype == torch.float32 and v.numel() == d and v.is_contiguous())
+    n_rows = h.shape[0] if rows is None else rows.numel()
+    for o in (out0, out1):
+        if o is not None:
+            _contig("out", o)
+            assert o.shape[0] >= n_rows and o.shape[-1] == d and o.dtype == out0.dtype
+    f = _fn("dual_norm", "llmx_dual_norm",
+            [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_int,
+             c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(h), *args, _ptr(bias), _ptr(rows), n_rows, _ptr(gain0), _ptr(gain1), eps, _ptr(out0), _ptr(out1),
+             _tag(out0) if out0 is not None else F32, d, int(write_h), _stream()), "dual_norm")
+
+
 ADD_SLICE = 512  # columns per CTA of add_gain_sumsq; the same constant as in elementwise.cu
 
 
@@ -530,11 +566,12 @@ def qk_norm_rope_cache(qkv, q_out, k_cache, v_cache, block_table, token_seq, tok
              v_head_dim, int(write_cache), _ptr(bias), _stream()), "qk_norm_rope_cache")
 
 
-GATE_ACTS = {"silu": 0, "relu": 1, "clamped_swish": 2, "gelu_tanh": 3}
+GATE_ACTS = {"silu": 0, "relu": 1, "clamped_swish": 2, "gelu_tanh": 3, "relu_squared": 4}
 
 
 def gate_act_args(activation="silu") -> tuple:
-    """(kind, slope, limit, shift) as the kernels take them.  ``activation``: "silu", "relu", or
+    """(kind, slope, limit, shift) as the kernels take them.  ``activation``: "silu", "relu", "gelu_tanh", "relu_squared"
+    (max(g, 0)^2 * u), or
     ("clamped_swish", slope, limit, shift): min(g, limit) * sigmoid(slope * min(g, limit)) * (clamp(u, +-limit) + shift)."""
     if isinstance(activation, str):
         return GATE_ACTS[activation], 1.0, 0.0, 0.0
@@ -561,6 +598,20 @@ def silu_gate(gu: torch.Tensor, out: torch.Tensor, block: int = 0, activation="s
              _ptr(bias), _stream()), "gate_act")
 
 
+def plain_act(parts: torch.Tensor, out: torch.Tensor, activation) -> None:
+    """The activation of a feed-forward without a gate: out = act(parts.sum(0)), the gated activation with up = 1;
+    parts [S, ...] (partials added in order) or a tensor of out's shape."""
+    _dev(parts, out)
+    _contig("parts", parts), _contig("out", out)
+    if parts.dim() == out.dim():
+        parts = parts.unsqueeze(0)
+    assert parts.shape[1:] == out.shape
+    f = _fn("elementwise", "llmx_plain_act",
+            [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_longlong, c_int, c_float, c_float, c_float, c_void_p])
+    _check(f(_ptr(parts), _tag(parts), parts.shape[0], parts.stride(0), _ptr(out), _tag(out), out.numel(),
+             *gate_act_args(activation), _stream()), "plain_act")
+
+
 def sum_splits(parts: torch.Tensor, out: torch.Tensor) -> None:
     """out = parts.sum(0) with the partials added in order; parts [S, ...]."""
     _dev(parts, out)
@@ -576,10 +627,19 @@ def _check_sinks(sinks, n_heads: int) -> None:
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads and sinks.is_contiguous())
 
 
+def _check_score_bias(score_bias, n_heads: int) -> None:
+    assert score_bias is None or (score_bias.dtype == torch.float32 and score_bias.dim() == 2 and score_bias.is_contiguous()
+                                  and score_bias.shape[0] == n_heads)
+
+
+def _score_bias_args(score_bias) -> tuple:
+    return (None, 0) if score_bias is None else (_ptr(score_bias), score_bias.shape[1])
+
+
 def attention_paged(q, out, k_cache, v_cache, block_table, token_seq, token_pos, n_heads: int,
                     n_kv_heads: int, head_dim: int, window, scale: float, v_head_dim=None, keep_first: int = 0,
                     sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None,
-                    gate=None, softcap: float = 0.0, sinks=None) -> None:
+                    gate=None, softcap: float = 0.0, sinks=None, score_bias=None) -> None:
     """General attention over the paged cache; q [T,H*D] (rows may be the first columns of wider rows), out
     [T,H*Dv].  Under a window the first ``keep_first`` keys of a sequence stay visible.  ``sink`` is added to the
     softmax's denominator (as many keys of score 0 that have no value).  With ``chunk`` n > 0 a query sees only the
@@ -587,8 +647,11 @@ def attention_paged(q, out, k_cache, v_cache, block_table, token_seq, token_pos,
     window) every block of n positions that lies wholly before the window is seen as row b of ``pool_k`` / ``pool_v``
     (paged like the cache, block table ``pool_table``).  ``gate`` float32 [T, >= H] (a view with any row stride):
     head h's output is multiplied by sigmoid(gate[t, h]).  ``softcap`` c > 0: every scaled score s becomes
-    c * tanh(s / c).  ``sinks`` float32 [H]: exp(sinks[h]) joins head h's denominator (no key, no value, not capped)."""
-    _dev(q, out, k_cache, v_cache, block_table, token_seq, token_pos, pool_k, pool_v, pool_table, gate, sinks)
+    c * tanh(s / c).  ``sinks`` float32 [H]: exp(sinks[h]) joins head h's denominator (no key, no value, not capped).
+    ``score_bias`` float32 [H, n]: score_bias[h, min(p - j, n - 1)] joins the scaled score of the key at j (the last entry
+    stands for every longer distance; not beside pooled blocks or a cap)."""
+    _dev(q, out, k_cache, v_cache, block_table, token_seq, token_pos, pool_k, pool_v, pool_table, gate, sinks, score_bias)
+    _check_score_bias(score_bias, n_heads)
     _check_sinks(sinks, n_heads)
     _contig("out", out), _contig("block_table", block_table)
     if pool:
@@ -602,15 +665,16 @@ def attention_paged(q, out, k_cache, v_cache, block_table, token_seq, token_pos,
         raise Unsupported(f"head_dim {head_dim}/{v_head_dim}: the general attention kernel takes sizes up to 256")
     if n_heads % n_kv_heads:
         raise Unsupported(f"{n_heads} heads are not a multiple of {n_kv_heads} kv heads")
-    f = _fn("attention", "llmx_attention_paged_capped",
+    f = _fn("attention", "llmx_attention_paged_biased",
             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
              c_int, c_int, c_int, c_int, c_int, c_longlong, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p,
-             c_void_p, c_void_p, c_void_p, c_longlong, c_float, c_void_p, c_void_p])
+             c_void_p, c_void_p, c_void_p, c_longlong, c_float, c_void_p, c_void_p, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(out), _tag(q), _ptr(k_cache), _ptr(v_cache), _tag(k_cache), _ptr(block_table),
              block_table.shape[1], _ptr(token_seq), _ptr(token_pos), q.shape[0], n_heads, n_kv_heads, head_dim,
              v_head_dim, q.stride(0), int(window or 0), int(keep_first or 0), scale, float(sink or 0.0), int(chunk or 0),
              int(pool or 0), _ptr(pool_k), _ptr(pool_v), _ptr(pool_table), _ptr(gate),
-             gate.stride(0) if gate is not None else 0, float(softcap or 0.0), _ptr(sinks), _stream()), "attention_paged")
+             gate.stride(0) if gate is not None else 0, float(softcap or 0.0), _ptr(sinks), *_score_bias_args(score_bias),
+             _stream()), "attention_paged")
 
 
 def pool_blocks(k_cache, v_cache, block_table, pool_k, pool_v, pool_table, seq_start, seq_past, n_seqs: int,
@@ -862,22 +926,24 @@ def _counters(device, n: int):
     return buf
 
 
-def capped_library(name: str, softcap) -> str:
-    """The library of a tiled attention kernel: its own build where scores are capped (decode: or sinks learned)."""
-    return name + "_capped" if softcap else name
+def capped_library(name: str, softcap, score_bias=None) -> str:
+    """The library of a tiled attention kernel: its own build where scores are capped (decode: or sinks learned), and one
+    where they have a learned bias."""
+    return name + "_biased" if score_bias is not None else name + "_capped" if softcap else name
 
 
 def attention_decode(q, out, k_cache, v_cache, block_table, seq_past, n_heads: int, n_kv_heads: int,
                      head_dim: int, window, scale: float, n_chunks: int = 0, keep_first: int = 0,
                      sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None,
-                     softcap: float = 0.0, sinks=None) -> None:
+                     softcap: float = 0.0, sinks=None, score_bias=None) -> None:
     """One new token per sequence, bfloat16: q, out [B,H*D] in batch order;
     seq_past[b] is the token's position.  Each sequence's keys are split over
     n_chunks CTAs (0: chosen from the batch's shape), which merge inside a
     cluster, or beyond 8 chunks through a float32 workspace.  ``chunk`` n > 0 is
     the chunked mask of ``attention_paged`` (nothing to do with n_chunks); ``pool`` with its second store, ``softcap`` and ``sinks``
-    likewise (capped scores run in a library of their own; no pooled blocks there)."""
-    _dev(q, out, k_cache, v_cache, block_table, seq_past, pool_k, pool_v, pool_table, sinks)
+    likewise (capped scores run in a library of their own; no pooled blocks there), ``score_bias`` too."""
+    _dev(q, out, k_cache, v_cache, block_table, seq_past, pool_k, pool_v, pool_table, sinks, score_bias)
+    _check_score_bias(score_bias, n_heads)
     _check_sinks(sinks, n_heads)
     _contig("q", q), _contig("out", out), _contig("block_table", block_table)
     if pool:
@@ -902,16 +968,17 @@ def attention_decode(q, out, k_cache, v_cache, block_table, seq_past, n_heads: i
         ws = guard.scratch((B * n_heads * n_chunks * (head_dim + 4),), torch.float32, q.device,
                            "decode attention workspace")
         counters = _counters(q.device, B * n_kv_heads * ((group + 7) // 8))
-    f = _fn(capped_library("attention_decode", softcap or sinks is not None), "llmx_attention_decode_capped",
+    f = _fn(capped_library("attention_decode", softcap or sinks is not None, score_bias), "llmx_attention_decode_biased",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
              c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float, c_int, c_int, c_void_p,
-             c_void_p, c_longlong, c_void_p, c_void_p])
+             c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(block_table),
              block_table.shape[1],
              _ptr(seq_past), _ptr(ws), _ptr(counters), B, n_heads, n_kv_heads, head_dim, int(window or 0),
              int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0), _ptr(sinks), float(softcap or 0.0), n_chunks,
              int(pool or 0), _ptr(pool_k),
-             _ptr(pool_v), pool_k.shape[0] if pool else 0, _ptr(pool_table), _stream()), "attention_decode")
+             _ptr(pool_v), pool_k.shape[0] if pool else 0, _ptr(pool_table), *_score_bias_args(score_bias), _stream()),
+           "attention_decode")
 
 
 def attention_decode_status() -> int:
@@ -928,12 +995,14 @@ def attention_prefill_supports(q, k_cache, head_dim: int) -> bool:
 def attention_prefill(q, out, k_cache, v_cache, block_table, seq_start, seq_past, n_seqs: int, max_new: int,
                       n_heads: int, n_kv_heads: int, head_dim: int, window, scale: float, keep_first: int = 0,
                       sink: float = 0.0, chunk: int = 0, pool: int = 0, pool_k=None, pool_v=None, pool_table=None,
-                      softcap: float = 0.0, sinks=None) -> None:
+                      softcap: float = 0.0, sinks=None, score_bias=None) -> None:
     """Prompt attention on the tensor cores, bfloat16, head sizes 64 and 128:
     q, out [T,H*D] packed sequence after sequence.  Under a window the first ``keep_first`` keys stay visible;
     ``chunk`` n > 0 is the chunked mask of ``attention_paged``, ``pool`` with its second store its pooled blocks;
-    ``softcap`` and ``sinks`` as there (capped scores run in a library of their own; no pooled blocks there)."""
-    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, pool_k, pool_v, pool_table, sinks)
+    ``softcap``, ``sinks`` and ``score_bias`` as there (capped or biased scores run in libraries of their own; no pooled
+    blocks there)."""
+    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, pool_k, pool_v, pool_table, sinks, score_bias)
+    _check_score_bias(score_bias, n_heads)
     _check_sinks(sinks, n_heads)
     _contig("q", q), _contig("out", out), _contig("block_table", block_table)
     if pool:
@@ -942,35 +1011,39 @@ def attention_prefill(q, out, k_cache, v_cache, block_table, seq_start, seq_past
         assert pool_k.is_contiguous() and pool_v.is_contiguous() and pool_k.shape[1:] == k_cache.shape[1:]
     if not attention_prefill_supports(q, k_cache, head_dim):
         raise Unsupported(f"the tiled prompt attention takes bfloat16 and head sizes 64 or 128, not {head_dim}")
-    f = _fn(capped_library("attention_prefill", softcap), "llmx_attention_prefill_capped",
+    f = _fn(capped_library("attention_prefill", softcap, score_bias), "llmx_attention_prefill_biased",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
              c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
-             c_void_p])
+             c_void_p, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
              _ptr(seq_start), _ptr(seq_past), n_seqs, max_new, n_heads, n_kv_heads, head_dim, int(window or 0),
              int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0), int(pool or 0), _ptr(pool_k), _ptr(pool_v),
-             _ptr(pool_table), _ptr(sinks), float(softcap or 0.0), _stream()), "attention_prefill")
+             _ptr(pool_table), _ptr(sinks), float(softcap or 0.0), *_score_bias_args(score_bias), _stream()),
+           "attention_prefill")
 
 
 def attention_prefill_tc(q, out, k_cache, v_cache, block_table, seq_start, seq_past, n_seqs: int, max_new: int,
                          n_heads: int, n_kv_heads: int, head_dim: int, window, scale: float, keep_first: int = 0,
-                         sink: float = 0.0, chunk: int = 0, softcap: float = 0.0, sinks=None) -> None:
+                         sink: float = 0.0, chunk: int = 0, softcap: float = 0.0, sinks=None, score_bias=None) -> None:
     """Prompt attention on tcgen05, bfloat16, head size 128: q, out [T,H*128]
     packed sequence after sequence; the cache entry is [n_pages,G,64,128].  ``chunk`` n > 0 is the chunked mask
-    of ``attention_paged``, ``softcap`` and ``sinks`` as there (capped scores run in a library of their own)."""
-    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, sinks)
+    of ``attention_paged``, ``softcap``, ``sinks`` and ``score_bias`` as there (capped or biased scores run in libraries
+    of their own)."""
+    _dev(q, out, k_cache, v_cache, block_table, seq_start, seq_past, sinks, score_bias)
+    _check_score_bias(score_bias, n_heads)
     _check_sinks(sinks, n_heads)
     _contig("q", q), _contig("out", out), _contig("block_table", block_table)
     assert k_cache.is_contiguous() and v_cache.is_contiguous()
     if head_dim != 128 or q.dtype != torch.bfloat16 or k_cache.dtype != torch.bfloat16:
         raise Unsupported("the tcgen05 prompt attention takes bfloat16 and head size 128")
-    f = _fn(capped_library("attention_prefill_tc", softcap), "llmx_attention_prefill_tc_capped",
+    f = _fn(capped_library("attention_prefill_tc", softcap, score_bias), "llmx_attention_prefill_tc_biased",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float, c_void_p])
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_float, c_void_p, c_int,
+             c_void_p])
     _check(f(_ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(block_table),
              block_table.shape[1], _ptr(seq_start), _ptr(seq_past), n_seqs, q.shape[0], max_new, n_heads,
              n_kv_heads, head_dim, int(window or 0), int(keep_first or 0), int(chunk or 0), scale, float(sink or 0.0),
-             _ptr(sinks), float(softcap or 0.0), _stream()), "attention_prefill_tc")
+             _ptr(sinks), float(softcap or 0.0), *_score_bias_args(score_bias), _stream()), "attention_prefill_tc")
 
 
 def attention_prefill_tc_status(reset: bool = True) -> int:
@@ -1043,7 +1116,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_split: int = 
     or float32), or float32 partials [n_split,T,N] of a split reduction, or,
     with ``gated``, [T,N/2] = silu(gate) * up: ``gated=True`` (or 1) for
     w = [gate rows; up rows], ``gated=2`` for w in blocks of 16 gate rows each
-    followed by the 16 up rows of the same features (N/2 a multiple of 16).
+    followed by the 16 up rows of the same features (N/2 a multiple of 16); ``gated=3``: no gate, [T,N] = act(product)
+    (``gate_act_args`` with up = 1).
     ``pair`` runs the CTA-pair kernel (prompt-sized T > 128; it splits too); with
     ``accumulate`` it adds to a float32 ``out`` instead of overwriting it
     (one float32 addition per element, whatever order the tiles finish in).
@@ -1069,8 +1143,9 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_split: int = 
     else:
         assert gate_bias is None
     if gated:
-        assert n_split == 1 and out.shape == (T, N // 2)
-        ldy, stride = N // 2, 0
+        F = N if gated == 3 else N // 2
+        assert n_split == 1 and out.shape == (T, F)
+        ldy, stride = F, 0
     elif n_split > 1:
         assert out.shape == (n_split, T, N) and out.dtype == torch.float32
         ldy, stride = N, out.stride(0)
@@ -1328,6 +1403,113 @@ def delta_decode(proj, offsets, conv_w, taps: int, a_log, dt_bias, q_scale: floa
              _stream()), "delta_decode")
 
 
+def qk_unit_rope_cache(proj, bias, q_out, k_cache, v_cache, block_table, ctx, eps: float, cos, sin, n_rot: int, n_heads: int,
+                       n_kv_heads: int, head_dim: int) -> None:
+    """Attention whose keys are its values: ``proj`` [T, >= (H+G)*D] (or float32 partials [S, T, ..]) holds q heads, then
+    k heads; + ``bias`` (float32 [(H+G)*D] or None).  A key as it then is goes into the value store; q and k are rotated,
+    divided by their root mean square per head and go to ``q_out`` [T, H*D] and the key store."""
+    _dev(proj, bias, q_out, k_cache, v_cache, block_table, cos, sin)
+    for name, t in (("q_out", q_out), ("k_cache", k_cache), ("v_cache", v_cache), ("block_table", block_table)):
+        _contig(name, t)
+    H, G, D = n_heads, n_kv_heads, head_dim
+    n_split, split_stride, row_stride = _split_view(proj)
+    T = q_out.shape[0]
+    assert q_out.shape == (proj.shape[-2], H * D) and q_out.dtype == k_cache.dtype == v_cache.dtype
+    assert k_cache.shape[1:] == (G, PAGE, D) == v_cache.shape[1:]
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == (H + G) * D and bias.is_contiguous())
+    if D > 256:
+        raise Unsupported(f"head_dim {D}: the q/k norm and rotation kernel takes sizes up to 256")
+    f = _fn("qk_unit", "llmx_qk_unit_rope_cache",
+            [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+             c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_void_p])
+    _check(f(_ptr(proj), _tag(proj), n_split, split_stride, row_stride, _ptr(bias), _ptr(q_out), _ptr(k_cache), _ptr(v_cache),
+             _tag(k_cache), _ptr(block_table), block_table.shape[1], _ptr(ctx.token_seq), _ptr(ctx.token_pos), eps, _ptr(cos),
+             _ptr(sin), n_rot, T, H, G, D, ctx.n_seqs, k_cache.shape[0], _stream()), "qk_unit_rope_cache")
+
+
+def gate_rows(out, z) -> None:
+    """out *= sigmoid(z) in place; out [T, n], z [T, n] (a view of wider rows allowed) or float32 partials [S, T, n]."""
+    _dev(out, z)
+    _contig("out", out)
+    n_split, split_stride, row_stride = _split_view(z)
+    assert z.shape[-2:] == out.shape
+    f = _fn("qk_unit", "llmx_gate_rows",
+            [c_void_p, c_int, c_void_p, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_void_p])
+    _check(f(_ptr(out), _tag(out), _ptr(z), _tag(z), n_split, split_stride, row_stride, out.shape[0], out.shape[1], _stream()),
+           "gate_rows")
+
+
+# ---- the state-space recurrence (csrc/state_space.cu) ------------------------------------------------------------------
+
+SS_CHUNK, SS_MAX_TAPS = 64, 16       # the same constants as in state_space.cu
+
+
+def _ss_args(proj, conv_w, conv_b, a_log, dt_bias, skip, state, ring_off, H, G, N, P):
+    _dev(proj, conv_w, conv_b, a_log, dt_bias, skip, state)
+    _contig("state", state), _contig("conv_w", conv_w)
+    taps, C = conv_w.shape
+    assert proj.dtype == conv_w.dtype == state.dtype == torch.float32 and C == H * P + 2 * G * N and state.dim() == 2
+    assert proj.shape[-1] == H * P + C + H and state.shape[1] >= ring_off + taps * C
+    assert conv_b is None or (conv_b.dtype == torch.float32 and conv_b.numel() == C and conv_b.is_contiguous())
+    assert all(v.dtype == torch.float32 and v.numel() == H and v.is_contiguous() for v in (a_log, dt_bias, skip))
+    n_split, split_stride, row_stride = _split_view(proj)
+    return (_ptr(proj), n_split, split_stride, row_stride, _ptr(conv_w), _ptr(conv_b), taps, _ptr(a_log), _ptr(dt_bias),
+            _ptr(skip), _ptr(state), state.stride(0), ring_off, state.shape[0])
+
+
+_SS_ARGTYPES = [c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                c_longlong, c_longlong, c_int]
+
+
+def ss_prompt(proj, conv_w, conv_b, a_log, dt_bias, skip, state, ring_off: int, y, ctx, n_heads: int, n_groups: int,
+              state_size: int, head_dim: int) -> None:
+    """The state-space recurrence over every sequence's tokens of the step: convolution and SiLU on x, B and C, then
+    S <- exp(-exp(A_log) dt) S + dt B x^T, y = (S^T C + D x) silu(z).  ``proj`` float32 [T, n] (or partials) = [z | x | B |
+    C | dt]; ``conv_w`` float32 [taps, C]; ``state`` float32 [slots, n]: S [H, N, P], then from ``ring_off`` the
+    convolution's ring [taps, C].  ``y`` float32 [T, H*P]."""
+    H, G, N, P = n_heads, n_groups, state_size, head_dim
+    args = _ss_args(proj, conv_w, conv_b, a_log, dt_bias, skip, state, ring_off, H, G, N, P)
+    T = y.shape[0]
+    assert y.dtype == torch.float32 and y.shape == (proj.shape[-2], H * P) and y.is_contiguous()
+    pad4 = lambda n: (n + 3) // 4 * 4
+    chunks = T // SS_CHUNK + ctx.n_seqs
+    new = lambda n, what: guard.scratch((n,), torch.float32, y.device, what)
+    xs = new(T * H * pad4(P), "convolved x of the state-space recurrence")
+    bs, cs = (new(T * G * pad4(N), f"convolved {r} of the state-space recurrence") for r in "BC")
+    da = new(2 * T * H, "decays and step sizes of the state-space recurrence")
+    st = new(chunks * H * N * pad4(P), "states of a prompt's chunks")
+    at = new(pad4(chunks * H), "decays over a prompt's chunks")
+    cb = new(chunks * G * SS_CHUNK * SS_CHUNK, "C . B of a prompt's chunks")
+    f = _fn("state_space", "llmx_ss_prompt",
+            _SS_ARGTYPES + [c_void_p] * 8 + [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(*args, _ptr(xs), _ptr(bs), _ptr(cs), _ptr(da), _ptr(st), _ptr(at), _ptr(cb), _ptr(y), _ptr(ctx.seq_start),
+             _ptr(ctx.seq_past), _ptr(ctx.seq_slot), T, ctx.n_seqs, H, G, N, P, _stream()), "ss_prompt")
+    global launch_count
+    launch_count += 3                    # beside the preparation: the chunks' states, the pass over them, the outputs
+
+
+def ss_decode(proj, conv_w, conv_b, a_log, dt_bias, skip, state, ring_off: int, y, ctx, n_heads: int, n_groups: int,
+              state_size: int, head_dim: int) -> None:
+    """The same for a step in which every sequence brings one token."""
+    H, G, N, P = n_heads, n_groups, state_size, head_dim
+    args = _ss_args(proj, conv_w, conv_b, a_log, dt_bias, skip, state, ring_off, H, G, N, P)
+    assert y.dtype == torch.float32 and y.shape == (ctx.n_seqs, H * P) == (proj.shape[-2], H * P) and y.is_contiguous()
+    f = _fn("state_space", "llmx_ss_decode",
+            _SS_ARGTYPES + [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(*args, _ptr(y), _ptr(ctx.seq_past), _ptr(ctx.seq_slot), ctx.n_seqs, H, G, N, P, _stream()), "ss_decode")
+
+
+def ss_norm(y, gain, eps: float, parts: int, out) -> None:
+    """out = y / sqrt(mean(y^2) + eps) * gain, the mean over each of ``parts`` equal runs of a row's columns; y float32
+    [T, n], gain float32 [n]."""
+    _dev(y, gain, out)
+    _contig("y", y), _contig("out", out)
+    T, n = y.shape
+    assert y.dtype == gain.dtype == torch.float32 and gain.numel() == n and out.shape == y.shape and n % parts == 0
+    f = _fn("state_space", "llmx_ss_norm", [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(y), _ptr(gain), eps, _ptr(out), _tag(out), T, n // parts, parts, _stream()), "ss_norm")
+
+
 def gated_norm(o, proj, g_off: int, gain, eps: float, gate: str, per_head: bool, y, n_heads: int,
                v_head_dim: int, gates=None, den_eps: float = 0.0) -> None:
     """y = o / sqrt(mean(o^2) + eps) * gain * gate(proj[:, g_off:]) with the mean over one head's columns
@@ -1447,39 +1629,41 @@ def moe_gather_rows(x, perm, top: int, xs) -> None:
     _check(f(_ptr(x), x.stride(0), _ptr(perm), top, _ptr(xs), perm.numel(), x.shape[1], _stream()), "moe_gather_rows")
 
 
-def moe_grouped_tc(xs, w, y, tiles, tile_rows: int, dest, sorted_weight, gated: bool, activation="silu") -> None:
+def moe_grouped_tc(xs, w, y, tiles, tile_rows: int, dest, sorted_weight, gated: int, activation="silu") -> None:
     """The grouped products on tcgen05.  ``xs`` bfloat16 [P, K] in sorted order; ``gated``: w [E, 2F, K] (gate rows,
-    then up rows), y bfloat16 [P, F]; else w [E, N, K], y float32 [top, T, N] whose row ``dest[place]`` becomes
+    then up rows), y bfloat16 [P, F]; ``gated`` 2 (experts without a gate): w [E, F, K], y = act(product); else w [E, N, K], y float32 [top, T, N] whose row ``dest[place]`` becomes
     ``sorted_weight[place]`` times the product.  ``tiles`` made by ``moe_sort`` with ``tile_rows`` in (16, 64, 128)."""
     _dev(xs, w, y, tiles, dest, sorted_weight)
     _contig("w", w), _contig("y", y)
     assert moe_tc_supports(xs, w) and tile_rows in (16, 64, 128) and (not gated or moe_tc_gated_supports(activation))
+    gated = int(gated)
     K = xs.shape[1]
-    N = w.shape[1] // 2 if gated else w.shape[1]
+    N = w.shape[1] // 2 if gated == 1 else w.shape[1]
     assert w.shape[2] == K and y.dtype == (torch.bfloat16 if gated else torch.float32)
     f = _fn("moe_tc", "llmx_moe_grouped_tc",
             [c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
              c_int, c_int, c_int, c_float, c_float, c_float, c_void_p])
     _check(f(_ptr(xs), xs.stride(0), xs.shape[0], _ptr(w), w.shape[0], _ptr(y), _ptr(tiles), tiles.shape[0], tile_rows,
-             _ptr(dest), _ptr(sorted_weight), N, K, int(gated), *gate_act_args(activation), _stream()), "moe_grouped_tc")
+             _ptr(dest), _ptr(sorted_weight), N, K, gated, *gate_act_args(activation), _stream()), "moe_grouped_tc")
 
 
-def moe_grouped(x, w, y, perm, tiles, pair_weight, top: int, n_tokens: int, gated: bool, activation="silu") -> None:
+def moe_grouped(x, w, y, perm, tiles, pair_weight, top: int, n_tokens: int, gated: int, activation="silu") -> None:
     """Grouped products over the sorted pairs on the FMA units (the float32 path, and sizes the tensor-core kernel
     does not take).  ``gated``: x [T, K] gathered through ``perm``, w [E, 2F, K] (gate rows, then up rows), y [P, F] =
-    silu(gate) * up in sorted order.  Else: x [P, K] in sorted order, w [E, N, K], y float32 [top, T, N] = weight of
+    silu(gate) * up in sorted order; ``gated`` 2: w [E, F, K] without a gate, y = act(product).  Else: x [P, K] in sorted order, w [E, N, K], y float32 [top, T, N] = weight of
     the pair times the product.  ``tiles`` made by ``moe_sort`` with ``MOE_TILE`` rows per tile."""
     _dev(x, w, y, perm, tiles, pair_weight)
     _contig("w", w), _contig("y", y)
     assert x.stride(1) == 1 and x.dtype == w.dtype
+    gated = int(gated)
     K = x.shape[1]
-    N = w.shape[1] // 2 if gated else w.shape[1]
+    N = w.shape[1] // 2 if gated == 1 else w.shape[1]
     assert w.shape[2] == K
     f = _fn("moe", "llmx_moe_grouped_fma",
             [c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
              c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p])
     _check(f(_ptr(x), _tag(x), x.stride(0), _ptr(w), _tag(w), _ptr(y), _tag(y), _ptr(perm), _ptr(tiles), tiles.shape[0],
-             _ptr(pair_weight), top, n_tokens, N, K, int(gated), *gate_act_args(activation), _stream()), "moe_grouped")
+             _ptr(pair_weight), top, n_tokens, N, K, gated, *gate_act_args(activation), _stream()), "moe_grouped")
 
 
 def moe_extras(x, ids, weights, y, n_real: int, shared=None, shared_z=None) -> None:

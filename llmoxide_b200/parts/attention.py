@@ -42,6 +42,13 @@ encoding that pairs neighbouring dimensions is met by reordering the rows of the
 (gains ``q_norm`` [H*D] and ``k_norm`` [G*D]; built without a rotation); beside it ``q_temp`` = (coef, every)
 multiplies the query at position p by 1 + coef ln(floor((p + 1) / every) + 1).  ``softcap`` c: a scaled score s becomes
 c tanh(s / c) before the softmax.
+``qk_norm`` "unit": q and k are divided by their root mean square per head, after the rotation, without a gain; built
+beside ``values`` "keys": there is no value projection, the key as projected (with its bias, before rotation and norm) is
+the value.  ``score_bias`` (tensor [rows, H]; ``bias_max`` m): a learned number per head and distance bucket joins every
+scaled score; a distance below rows // 2 has a row of its own, longer ones share the other rows on a logarithmic scale
+that ends at m (``distance_buckets``).  Tensor ``sink`` [H]: exp(sink_h) joins head h's softmax denominator, a learned
+score without key and value.  Tensor ``gate`` [H*Dv, d]: the concatenated heads are multiplied by sigmoid(W_gate x)
+before the output projection.
 Tensors ``q_bias``, ``k_bias``, ``v_bias``, ``o_bias``: biases of the four
 projections (q, k, v: added where the projected row is read, before norm and
 rotation; o: offered as ``out_bias`` to an arrangement that adds it in its
@@ -50,14 +57,33 @@ norm kernel, else added here).
 
 from __future__ import annotations
 
+from fractions import Fraction
+
 import torch
 
 from .. import kernels
 from ..cache import KVNeed, StateNeed
-from ..errors import Unsupported
+from ..errors import ConfigError, Unsupported
 from .linear import Linear
 from .position import halves_order
 from .registry import register_mixer
+
+
+def distance_buckets(n_distances: int, rows: int, far) -> list:
+    """The bucket of every distance 0 .. n_distances - 1 on a scale of ``rows`` buckets: distance n < rows // 2 has bucket
+    n, a longer one half + floor(ln(n / half) / ln(far / half) (rows - half)), at most rows - 1.  Decided in exact
+    arithmetic: the k-th bucket beyond half starts where n^r half^k >= far^k half^r, r = rows - half."""
+    half = rows // 2
+    r, far = rows - half, Fraction(far)
+    out, k = [], 0
+    for n in range(n_distances):
+        if n < half:
+            out.append(n)
+            continue
+        while k < r - 1 and Fraction(n) ** r * half ** (k + 1) >= far ** (k + 1) * half ** r:
+            k += 1
+        out.append(half + k)
+    return out
 
 
 @register_mixer("gqa_attention")
@@ -95,7 +121,29 @@ class GQAttention:
         if max(self.D, self.Dv) > 256:
             raise Unsupported(f"head sizes {self.D}/{self.Dv}: the attention kernels take sizes up to 256")
         t = spec.tensors
-        if self.own_kv:
+        self.qk_norm = spec.get("qk_norm", "heads")          # what q and k are normed over: each head, or whole rows
+        self.keys_as_values = spec.get("values", "own") == "keys"
+        self.unit_norm = self.qk_norm == "unit"
+        self.qk_bias = self.gate_off = None
+        if self.unit_norm != self.keys_as_values:
+            raise Unsupported("a q/k norm without gains and keys that serve as values are built beside one another")
+        if self.keys_as_values:
+            if not self.own_kv or self.Dv != self.D or self.pool or spec.get("conv_taps") or spec.get("v_mix") or (
+                    getattr(position, "pairing", "halves") != "halves"):
+                raise Unsupported("keys that serve as values are built for a layer with keys of its own, as large as its "
+                                  "values, without pooled blocks, convolution, mixed values and neighbouring pairs")
+            # one matrix product for q, k and the output's gate: rows in that order
+            ws = [weights.pop(t[r].name) for r in ("q", "k", "gate") if r in t]
+            if len({w.dtype for w in ws}) > 1:
+                ws = [w.float() for w in ws]
+            self.qkv = Linear(torch.cat(ws, dim=0), rt)
+            del ws
+            self.q_only = self.qkv
+            if "gate" in t:
+                self.gate_off = (self.H + self.G) * self.D
+            if "q_bias" in t:
+                self.qk_bias = torch.cat([weights.pop(t[r].name).to(torch.float32) for r in ("q_bias", "k_bias")]).contiguous()
+        elif self.own_kv:
             wq, wk, wv = (weights.pop(t[r].name) for r in ("q", "k", "v"))
             if not (wq.dtype == wk.dtype == wv.dtype):
                 wq, wk, wv = wq.float(), wk.float(), wv.float()
@@ -111,7 +159,7 @@ class GQAttention:
         self.o = Linear(weights.pop(t["o"].name), rt, bias=weights.pop(t["o_bias"].name) if "o_bias" in t else None)
         self.out_bias, self.defer_out_bias = self.o.bias, False
         self.qkv_bias = None
-        if "q_bias" in t:
+        if "q_bias" in t and not self.keys_as_values:
             if not self.own_kv:
                 raise Unsupported("projection biases are built for a layer with its own keys and values")
             bq, bk, bv = (weights.pop(t[r].name).to(torch.float32) for r in ("q_bias", "k_bias", "v_bias"))
@@ -119,7 +167,6 @@ class GQAttention:
             bk = halves_order(position, bk.unsqueeze(1), self.G, self.D).squeeze(1)
             self.qkv_bias = torch.cat([bq, bk, bv]).contiguous()
         self.q_gain = self.k_gain = None
-        self.qk_norm = spec.get("qk_norm", "heads")          # what q and k are normed over: each head, or whole rows
         if "q_norm" in t:
             self.q_gain = weights.pop(t["q_norm"].name).to(torch.float32).contiguous()
             if self.own_kv or self.qk_norm == "heads":
@@ -137,6 +184,16 @@ class GQAttention:
         self.position = position
         if getattr(position, "pairing", "halves") == "neighbours" and ("q_norm" in t or spec.get("conv_taps")):
             raise Unsupported("a rotation of neighbouring pairs beside a q/k norm or a short convolution is not built")
+        self.sinks = weights.pop(t["sink"].name).to(torch.float32).contiguous() if "sink" in t else None
+        self.score_bias = None
+        if "score_bias" in t:
+            self.score_bias = self._distance_table(weights.pop(t["score_bias"].name).to(torch.float32), spec["bias_max"])
+        if self.pool and (self.sinks is not None or self.score_bias is not None):
+            raise Unsupported("learned sinks or score biases beside pooled blocks are not built")
+        if self.softcap and self.score_bias is not None:
+            raise Unsupported("a learned score bias beside capped scores is not built")
+        if "gate" in t and not self.keys_as_values:
+            raise Unsupported("an output gate is built beside keys that serve as values")
         self.taps = int(spec.get("conv_taps") or 0)
         self.sink = float(spec.get("sink") or 0.0)
         self.v_mix, self.v_mix_key = spec.get("v_mix"), spec.get("v_mix_key", "v_mix")
@@ -157,6 +214,20 @@ class GQAttention:
         self.staged = bool(self.taps or self.v_mix)
         self.channels = (self.H + self.G) * self.D + self.G * self.Dv
 
+    def _distance_table(self, table, far):
+        """float32 [H, n] from the table's rows: entry min(distance, n - 1) is the bias.  n covers every distance the mask
+        lets through, or reaches the distance from which on the last row applies."""
+        rows, half = table.shape[0], table.shape[0] // 2
+        if rows < 2 or table.shape[1] != self.H or not far > half:
+            raise ConfigError(f"a distance table of shape {tuple(table.shape)} for {self.H} heads and bias_max {far}: it has "
+                              f"at least two rows, a column per head, and bias_max beyond {half}")
+        n = int(-(-Fraction(far) // 1)) + 1
+        reach = self.window if self.window and not self.keep_first else self.chunk
+        if reach:
+            n = min(n, reach)
+        index = torch.tensor(distance_buckets(n, rows, far), device=table.device)
+        return table.index_select(0, index).t().contiguous()
+
     def cache_need(self):
         state = StateNeed((self.taps - 1, self.channels)) if self.taps > 1 else None
         return KVNeed(self.G, self.D, self.cache_window, v_head_dim=None if self.Dv == self.D else self.Dv,
@@ -165,7 +236,7 @@ class GQAttention:
     @property
     def takes_row_scales(self) -> bool:
         """Its first products (q|k|v) can apply a norm's row scales in their epilogue."""
-        return (self.qkv is None or self.qkv.takes_row_scales) and self.q_only.takes_row_scales
+        return (self.qkv is None or self.qkv.takes_row_scales) and self.q_only.takes_row_scales and not self.keys_as_values
 
     def libraries(self) -> set:
         libs = {"elementwise"} | self.q_only.libraries() | self.o.libraries()
@@ -175,12 +246,14 @@ class GQAttention:
             libs.add("attention")           # the blocks' means are made there
         if self.row_norm:
             libs.add("qk_row_norm")
+        if self.keys_as_values:
+            libs.add("qk_unit")
         if not self.plain:
             return libs | {"attention"}
         if self.rt.dtype == "bfloat16" and self.rt.tensor_cores:
             tc = self.D == 128 and not self.pool      # (pooled blocks: the mma.sync kernel, at both head sizes)
-            cap = lambda name: kernels.capped_library(name, self.softcap)
-            libs |= {cap("attention_decode"),
+            cap = lambda name, sinks=None: kernels.capped_library(name, self.softcap or sinks is not None, self.score_bias)
+            libs |= {cap("attention_decode", self.sinks),
                      cap("attention_prefill_tc") if tc else cap("attention_prefill") if self.D in (64, 128) else "attention"}
         else:
             libs.add("attention")
@@ -214,6 +287,13 @@ class GQAttention:
                                     n_rot, v_first, self.v_lambda, mode, H, G, D, Dv, inline_state=inline)
             if not inline:
                 kernels.conv_state_update(qkv, view.state, self.taps, ctx)
+        elif self.keys_as_values:
+            if not writes_cache:
+                raise Unsupported("a layer whose keys are its values owns its cache entry")
+            proj = self.qkv(x, splits_ok=True)
+            q = torch.empty((T, H * D), dtype=self.rt.act_dtype, device=dev)
+            kernels.qk_unit_rope_cache(proj, self.qk_bias, q, view.k, view.v, block_table, ctx, self.eps, cos, sin, n_rot,
+                                       H, G, D)
         elif self.row_norm:
             proj = self.qkv(x, splits_ok=True) if writes_cache else self.q_only(x, splits_ok=True)
             q = torch.empty((T, H * D), dtype=self.rt.act_dtype, device=dev)
@@ -240,7 +320,9 @@ class GQAttention:
                                 ctx.seq_start, ctx.seq_past, ctx.n_seqs, T, G, D, Dv, self.pool)
         out = torch.empty((T, H * Dv), dtype=self.rt.act_dtype, device=dev)
         self.attend(q, out, view, block_table, ctx)
-        if self.out_bias is None and residual is not None and self.o.add_into(out, residual):
+        if self.gate_off is not None:
+            kernels.gate_rows(out, proj[..., self.gate_off :])
+        if (self.out_bias is None or self.defer_out_bias) and residual is not None and self.o.add_into(out, residual):
             return None
         return self.o(out, splits_ok=True, add_bias=not self.defer_out_bias)
 
@@ -257,6 +339,10 @@ class GQAttention:
                       pool_table=ctx.block_tables[view.pool_group]) if self.pool else {}
         if self.softcap:
             extra["softcap"] = self.softcap
+        if self.sinks is not None:
+            extra["sinks"] = self.sinks
+        if self.score_bias is not None:
+            extra["score_bias"] = self.score_bias
         if fast and ctx.is_decode:
             kernels.attention_decode(q, out, view.k, view.v, block_table, ctx.seq_past, H, G, D, self.window,
                                      self.scale, keep_first=self.keep_first, sink=self.sink, chunk=self.chunk, **extra)

@@ -5,8 +5,8 @@ h += mixer(norm(h)); h += feed_forward(norm(h)).
 
 The residual stream stays float32.  Each residual add is fused into the norm
 that follows it, so a block hands its last delta on as ``pending`` instead of
-adding it itself.  ``parallel`` is the block with one norm whose output both
-sublayers read: h += mixer(norm(h)) + feed_forward(norm(h)).  A mixer or feed-forward with ``adds_to_residual`` is given the
+adding it itself.  ``parallel`` is the block whose sublayers read the same stream: h += mixer(norm(h)) +
+feed_forward(norm(h)) with one norm (``shared``), or with a norm for each (``mixer``, ``feed_forward``).  A mixer or feed-forward with ``adds_to_residual`` is given the
 stream (``residual=h``) and may add its result there itself, in the kernel of its
 last product; it then returns None, and the norm that follows has nothing to add.
 ``sandwich`` norms a sublayer's result as well as its input: h += norm_b(mixer(norm_a(h))), then the same around
@@ -29,7 +29,7 @@ from .. import kernels
 from ..cache import StateNeed
 from ..errors import Unsupported
 from .linear import Linear
-from .norm import stream_rows
+from .norm import Joined, stream_rows
 from .registry import (ARRANGEMENTS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, lookup, register_arrangement)
 
 
@@ -83,6 +83,9 @@ class PreNormBlock:
 def _summed(delta):
     """A delta as one tensor: split partials [S,T,d] are added in order."""
     from .norm import WeightedSum
+    if isinstance(delta, Joined):
+        total = sum(_summed(t).float() for t in delta.terms)
+        return total if delta.bias is None else total + delta.bias
     if isinstance(delta, WeightedSum):
         return sum(w * _summed(t).float() for t, w in delta.terms)
     if delta.dim() == 2:
@@ -117,26 +120,63 @@ def build_block(spec, weights: dict, rt):
 class ParallelBlock:
     """A single norm feeds mixer and feed-forward: x = norm(h); h += mixer(x) + feed_forward(x).  The mixer's
     result joins the float32 stream at once (nothing else reads the stream before the next layer's norm, and the
-    feed-forward reads x); the feed-forward's is handed on as the pending delta, which the next norm adds."""
+    feed-forward reads x); the feed-forward's is handed on as the pending delta, which the next norm adds.
+
+    With a norm for each sublayer (``mixer`` and ``feed_forward`` instead of ``shared``) one kernel adds what the block
+    before owes and makes the rows of both norms; both results are owed to the next block together (``parts.norm.Joined``),
+    save what a sublayer's last product has added to the stream itself."""
 
     def __init__(self, spec, weights: dict, rt):
         position = None
         if spec.position is not None:
             position = rt_shared_position(spec.position, weights, rt)
-        self.norm = build_part(NORMS, "norm", spec.norms["shared"], weights, rt)
+        self.norm = self.mixer_norm = self.ff_norm = None
+        if "shared" in spec.norms:
+            self.norm = build_part(NORMS, "norm", spec.norms["shared"], weights, rt)
+        else:
+            self.mixer_norm = build_part(NORMS, "norm", spec.norms["mixer"], weights, rt)
+            if "feed_forward" in spec.norms:
+                self.ff_norm = build_part(NORMS, "norm", spec.norms["feed_forward"], weights, rt)
         self.mixer = lookup(MIXERS, "mixer", spec.mixer.kind)(spec.mixer, position, weights, rt)
         self.feed_forward = build_part(FEED_FORWARDS, "feed-forward", spec.feed_forward, weights, rt)
+        if self.norm is None and getattr(self.mixer, "out_bias", None) is not None:
+            self.mixer.defer_out_bias = True         # joins with the results, in the next block's norm kernel
 
     def cache_need(self):
         return self.mixer.cache_need()
 
     def libraries(self) -> set:
-        libs = set()
-        for part in (self.norm, self.mixer, self.feed_forward):
-            libs |= getattr(part, "libraries", set)()
+        libs = {"dual_norm"} if self.norm is None else set()
+        for part in (self.norm, self.mixer_norm, self.ff_norm, self.mixer, self.feed_forward):
+            if part is not None:
+                libs |= getattr(part, "libraries", set)()
         return libs
 
+    def _forward_two_norms(self, h, pending, ctx, view, writes_cache):
+        probe = getattr(ctx, "probe", None)
+        if self.ff_norm is not None:
+            x, u = self.mixer_norm.add_forward_pair(h, pending, self.ff_norm)
+        else:
+            x, u = self.mixer_norm.add_forward(h, None if pending is None else Joined.of(pending)), None
+        if probe:
+            probe("resid_in", h), probe("attn_norm", x)
+
+        def run(part, *args):
+            if probe is None and getattr(part, "adds_to_residual", False):
+                return part.forward(*args, residual=h)
+            return part.forward(*args)
+
+        a = run(self.mixer, x, ctx, view, writes_cache)
+        out = run(self.feed_forward, u, ctx) if u is not None else None
+        if probe:
+            probe("attn_output", _summed(a))
+            if out is not None:
+                probe("ffn_out", _summed(out))
+        return Joined([a, out], getattr(self.mixer, "out_bias", None))
+
     def forward(self, h, pending, ctx, view, writes_cache=True):
+        if self.norm is None:
+            return self._forward_two_norms(h, pending, ctx, view, writes_cache)
         probe = getattr(ctx, "probe", None)
         x = self.norm.add_forward(h, pending)
         if probe:

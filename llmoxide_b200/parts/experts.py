@@ -1,5 +1,6 @@
 """Routed experts as a feed-forward: every token uses ``top`` of ``n_experts``
-small gated layers, down(act(gate x) * (up x)), weighted by the router.
+small gated layers, down(act(gate x) * (up x)), weighted by the router; with
+``gated`` false the layers are down(act(up x)) (tensors ``up<e>``, ``down<e>``).
 
 Router logits z = W_r x are float32 (the router's matrix is kept in float32;
 x may be the compute dtype's rounding), plus the tensor ``router_bias`` when
@@ -20,7 +21,9 @@ identity experts: they have no tensors and their output is the input itself
 ``act_up_shift``).  A shared expert (``shared_size``; tensors ``shared_gate``,
 ``shared_up``, ``shared_down``, ``shared_sg`` [1, d]; its limit ``shared_limit``)
 runs for every token and is added times sigmoid(shared_sg . x), or as it is
-when there is no ``shared_sg``.
+when there is no ``shared_sg``.  Without gates the shared expert has none
+either (``shared_up``, ``shared_down``); its product writes its partials behind
+the choices', or adds to the residual stream itself where it can.
 
 The step's (token, choice) pairs are ordered by expert on the device and the
 two products run grouped over that order (csrc/moe.cu), so nothing is read
@@ -63,6 +66,7 @@ class RoutedExperts:
             name, float(spec.get("act_slope", 1.0)), float(limit), float(spec.get("act_up_shift", 0.0)))
         self.activation = act(spec.get("act_limit", 0.0))
         self.rt = rt
+        self.gated = bool(spec.get("gated", True))
         self.E, self.top, self.F = spec["n_experts"], spec["top"], spec["intermediate_size"]
         self.n_identity = int(spec.get("n_identity") or 0)
         self.E_all = self.E + self.n_identity         # what the router chooses among
@@ -91,7 +95,15 @@ class RoutedExperts:
         self.router_bias = (weights.pop(t["router_bias"].name).to(torch.float32).contiguous()
                             if "router_bias" in t else None)
         self.shared, self.shared_gated = None, "shared_sg" in t
-        if spec.get("shared_size"):
+        if spec.get("shared_size") and not self.gated:
+            if self.shared_gated:
+                raise Unsupported("a gate on a shared expert is built for gated experts")
+            from ..config.spec import PartSpec
+            from .feed_forward import PlainMLP
+            self.shared = PlainMLP(PartSpec("mlp", dict(
+                hidden_size=spec["hidden_size"], intermediate_size=int(spec["shared_size"]), activation=self.activation),
+                dict(up=t["shared_up"], down=t["shared_down"])), weights, rt)
+        elif spec.get("shared_size"):
             if self.shared_gated:
                 # the shared expert's gate reads the same rows as the router: its vector is one more row of that matrix
                 self.router = torch.cat([self.router, weights.pop(t["shared_sg"].name).to(torch.float32).reshape(1, -1)],
@@ -104,9 +116,12 @@ class RoutedExperts:
                 activation=act(spec.get("shared_limit", spec.get("act_limit", 0.0)))),
                 dict(gate=t["shared_gate"], up=t["shared_up"], down=t["shared_down"])), weights, rt)
         dt = rt.act_dtype
-        gate_up = [torch.cat([weights.pop(t[f"gate{e}"].name), weights.pop(t[f"up{e}"].name)], dim=0).to(dt)
-                   for e in range(self.E)]
-        self.gate_up = torch.stack(gate_up).contiguous()             # [E, 2F, d]: gate rows, then up rows
+        if self.n_identity and not self.gated:
+            raise Unsupported("identity experts are built beside gated experts")
+        gate_up = [torch.cat([weights.pop(t[r + str(e)].name) for r in (("gate", "up") if self.gated else ("up",))],
+                             dim=0).to(dt) for e in range(self.E)]
+        # [E, 2F, d]: gate rows, then up rows; without gates [E, F, d]
+        self.gate_up = torch.stack(gate_up).contiguous()
         del gate_up
         self.down = torch.stack([weights.pop(t[f"down{e}"].name).to(dt) for e in range(self.E)]).contiguous()  # [E, d, F]
 
@@ -125,6 +140,11 @@ class RoutedExperts:
         the weights), wide ones for prompts."""
         per_expert = n_pairs / self.E
         return 16 if per_expert <= 16 else 64 if per_expert <= 96 else 128
+
+    @property
+    def adds_to_residual(self) -> bool:
+        """A shared expert without a gate adds to the stream itself where its product can; the rest is returned."""
+        return self.shared is not None and not self.gated
 
     def forward(self, x, ctx, residual=None):
         T, dev = x.shape[0], x.device
@@ -147,22 +167,33 @@ class RoutedExperts:
         tiles = torch.empty((kernels.moe_max_tiles(P, self.E_all, rows), 3), dtype=torch.int32, device=dev)
         act = torch.empty((P, self.F), dtype=self.rt.act_dtype, device=dev)
         d = self.down.shape[1]
-        y = torch.empty((self.top + (1 if self.shared else 0), T, d), dtype=torch.float32, device=dev)
+        extra, shared_act = (1 if self.shared else 0), None
+        if self.shared and not self.gated:
+            # added to the stream by its last product, or as partials behind the choices'
+            shared_act = self.shared.activate(x)
+            if residual is not None and self.shared.down.add_into(shared_act, residual):
+                extra, shared_act = 0, None
+            else:
+                extra = self.shared.down.partials(T)
+        y = torch.empty((self.top + extra, T, d), dtype=torch.float32, device=dev)
+        mode = 1 if self.gated else 2
         if fast:
             dest = torch.empty((P,), dtype=torch.int32, device=dev)
             sorted_w = torch.empty((P,), dtype=torch.float32, device=dev)
             kernels.moe_sort(ids, self.E_all, perm, tiles, rows, pair_w, dest, sorted_w, n_tiled=self.E)
             xs = torch.empty((P, x.shape[1]), dtype=torch.bfloat16, device=dev)
             kernels.moe_gather_rows(x, perm, self.top, xs)
-            kernels.moe_grouped_tc(xs, self.gate_up, act, tiles, rows, dest, sorted_w, gated=True,
+            kernels.moe_grouped_tc(xs, self.gate_up, act, tiles, rows, dest, sorted_w, gated=mode,
                                    activation=self.activation)
             kernels.moe_grouped_tc(act, self.down, y, tiles, rows, dest, sorted_w, gated=False)
         else:
             kernels.moe_sort(ids, self.E_all, perm, tiles, rows, n_tiled=self.E)
-            kernels.moe_grouped(x, self.gate_up, act, perm, tiles, pair_w, self.top, T, gated=True,
+            kernels.moe_grouped(x, self.gate_up, act, perm, tiles, pair_w, self.top, T, gated=mode,
                                 activation=self.activation)
             kernels.moe_grouped(act, self.down, y, perm, tiles, pair_w, self.top, T, gated=False)
-        if self.n_identity or self.shared:
+        if shared_act is not None:
+            self.shared.down.into(shared_act, y[self.top :])
+        elif self.n_identity or (self.shared and self.gated):
             # an identity expert's output is the token's own row times the weight; the shared expert's result is
             # weighted by its gate: both join y in one launch
             shared = self.shared.forward(x, ctx) if self.shared else None

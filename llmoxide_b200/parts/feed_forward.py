@@ -96,3 +96,40 @@ class GatedMLP:
         if self.out_bias is None and residual is not None and self.down.add_into(act, residual):
             return None
         return self.down(act, splits_ok=True, add_bias=not self.defer_out_bias)
+
+
+@register_feed_forward("mlp")
+class PlainMLP:
+    """A feed-forward without a gate: down(act(up x)), ``activation`` as for the gated one with up = 1 ("relu_squared":
+    max(z, 0)^2)."""
+
+    def __init__(self, spec, weights: dict, rt):
+        self.activation = spec.get("activation", "relu")
+        if self.activation not in kernels.GATE_ACTS or self.activation == "clamped_swish":
+            raise Unsupported(f"mlp activation {self.activation!r}: built are silu, relu, gelu_tanh, relu_squared")
+        self.rt, self.F = rt, spec["intermediate_size"]
+        t = spec.tensors
+        self.up, self.down = Linear(weights.pop(t["up"].name), rt), Linear(weights.pop(t["down"].name), rt)
+
+    def libraries(self) -> set:
+        return {"elementwise"} | self.up.libraries() | self.down.libraries()
+
+    adds_to_residual = True      # forward() takes ``residual`` and may return None: "already added"
+
+    def activate(self, x):
+        """act(up x)."""
+        tc = self.up._tc
+        # a step of few tokens streams the matrix: split over K where that keeps more SMs at it, the activation then sums
+        # the partials; otherwise it is the product's epilogue
+        if (tc is not None and x.dtype == torch.bfloat16 and kernels.gemm_tc_supports(x, tc.weight)
+                and self.rt.act_dtype == torch.bfloat16 and tc.splits(x.shape[0]) == 1):
+            return tc.activated(x, self.rt.act_dtype, self.activation)
+        act = torch.empty((x.shape[0], self.F), dtype=self.rt.act_dtype, device=x.device)
+        kernels.plain_act(self.up(x, out_dtype=torch.float32, splits_ok=True), act, self.activation)
+        return act
+
+    def forward(self, x, ctx, residual=None):
+        act = self.activate(x)
+        if residual is not None and self.down.add_into(act, residual):
+            return None
+        return self.down(act, splits_ok=True)

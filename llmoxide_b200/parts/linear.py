@@ -56,6 +56,18 @@ class Linear:
         self._tc.add_into(x, residual)
         return True
 
+    def partials(self, n_tokens: int) -> int:
+        """How many float32 partials ``into`` makes for a step of that many tokens."""
+        return self._tc.splits(n_tokens) if self._tc is not None else 1
+
+    def into(self, x, out) -> None:
+        """The product without its bias as ``partials(T)`` float32 partials into ``out`` [partials, T, out]."""
+        if self._tc is not None and not isinstance(x, RowScaled) and x.dtype == torch.bfloat16:
+            self._tc.into(x, out)
+        else:
+            assert out.shape[0] == 1
+            kernels.gemm_fma(x, self.weight, out[0])
+
     @property
     def takes_row_scales(self) -> bool:
         return self._tc is not None

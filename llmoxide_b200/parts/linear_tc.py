@@ -83,6 +83,26 @@ class TensorCoreLinear:
         """residual += x W^T."""
         kernels.gemm_tc(x, self.weight, residual, pair=True, accumulate=True)
 
+    def splits(self, n_tokens: int) -> int:
+        return (choose_splits(self.N, self.K, n_tokens, self.n_sm) if n_tokens <= 64 else
+                choose_prompt_splits(self.N, self.K, n_tokens, self.n_sm))
+
+    def into(self, x, out) -> None:
+        """Partials of the product into ``out`` float32 [splits(T), T, N]."""
+        T, s = x.shape[0], out.shape[0]
+        assert s == self.splits(T) and out.dtype == torch.float32 and out.is_contiguous()
+        if not kernels.gemm_tc_supports(x, self.weight):
+            out[1:].zero_()
+            kernels.gemm_fma(x, self.weight, out[0])
+            return
+        kernels.gemm_tc(x, self.weight, out if s > 1 else out[0], n_split=s, pair=T > PAIR_MIN_TOKENS)
+
+    def activated(self, x, out_dtype, activation):
+        """act(x W^T) for a feed-forward without a gate, the activation in the product's epilogue."""
+        out = scratch((x.shape[0], self.N), out_dtype, x.device, "output of the activated matrix product")
+        kernels.gemm_tc(x, self.weight, out, gated=3, pair=x.shape[0] > PAIR_MIN_TOKENS, activation=activation)
+        return out
+
     def __call__(self, x, out_dtype, splits_ok):
         x, scale = self._unpack(x)
         T = x.shape[0]
@@ -91,10 +111,7 @@ class TensorCoreLinear:
             out = torch.empty((T, self.N), dtype=out_dtype, device=x.device)
             kernels.gemm_fma(x, self.weight, out)
             return out
-        s = 1
-        if splits_ok:
-            s = (choose_splits(self.N, self.K, T, self.n_sm) if T <= 64 else
-                 choose_prompt_splits(self.N, self.K, T, self.n_sm))
+        s = self.splits(T) if splits_ok else 1
         if s > 1:
             out = scratch((s, T, self.N), torch.float32, x.device, "split partials of a matrix product")
             kernels.gemm_tc(x, self.weight, out, n_split=s, scale=scale, pair=T > PAIR_MIN_TOKENS)

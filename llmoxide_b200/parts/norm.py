@@ -21,6 +21,11 @@ whose sublayers read the stream itself (``post_norm``) there is no norm on the
 other side: ``stream_rows`` adds what is owed and returns the stream's rows in
 the compute dtype, by the same kernel.
 
+Two sublayers that read the same stream through norms of their own hand over a
+``Joined``: both results (and the first one's output bias), which the next
+kernel adds together.  ``RMSNorm.add_forward_pair`` then makes the rows of both
+norms of the next such block in that one pass (csrc/dual_norm.cu).
+
 ``gain_offset`` (parameter of ``rms_norm``): the gain is the stored weight plus
 this number, for weights stored as their distance from one."""
 
@@ -49,6 +54,20 @@ class WeightedSum:
 
     def __init__(self, terms):
         self.terms = list(terms)          # [(delta, weight)], at most two
+
+
+class Joined:
+    """What two sublayers side by side owe the residual stream: the sum of their results (each [T,d] or partials
+    [S,T,d]; at most two) and a bias."""
+
+    __slots__ = ("terms", "bias")
+
+    def __init__(self, terms, bias=None):
+        self.terms, self.bias = [t for t in terms if t is not None], bias
+
+    @staticmethod
+    def of(delta) -> "Joined":
+        return delta if isinstance(delta, Joined) else Joined([delta])
 
 
 class PostNormed:
@@ -171,6 +190,16 @@ class RMSNorm:
         kernels.stream_mix_norm(h, d, mix, write, self.read if out is not None else None, self.gain, self.eps, out,
                                 rows=rows, write_h=write_h)
 
+    def add_forward_pair(self, h, delta, other):
+        """h += ``delta`` (None, a tensor, partials or a ``Joined``); (norm(h) * gain, norm(h) * the other norm's gain),
+        the root mean square taken once (both norms have the same eps)."""
+        assert self.eps == other.eps and self.size == other.size
+        d = Joined.of(delta)
+        a = torch.empty((h.shape[0], self.size), dtype=self.rt.act_dtype, device=h.device)
+        b = torch.empty_like(a)
+        kernels.dual_norm(h, d.terms, d.bias, self.gain, self.eps, a, other.gain, b)
+        return a, b
+
     ROW_SCALE_MAX_TOKENS = 64      # what the products' epilogues take
 
     def add(self, h, delta) -> None:
@@ -178,6 +207,8 @@ class RMSNorm:
         if isinstance(delta, (PostNormed, WeightedSum)):
             kernels._library("post_norm")
             return _general_add_norm(h, delta, None, False, 0.0, None, None, True)
+        if isinstance(delta, Joined):
+            return kernels.dual_norm(h, delta.terms, delta.bias, None, self.eps, None)
         if h.dim() == 2 and isinstance(delta, StreamUpdate):
             h = h.unsqueeze(0)       # one copy, with connection weights of its own
         if h.dim() == 3:
@@ -189,6 +220,11 @@ class RMSNorm:
     def add_forward(self, h, delta, rows=None, write_h=True, out_dtype=None, row_scales_ok=False):
         """With ``row_scales_ok`` the caller's next products apply the norm's scale themselves; for a step of
         few tokens the result is then ``RowScaled`` (the norm in two halves, see ``parts.row_scaled``)."""
+        if isinstance(delta, Joined):
+            n = h.shape[0] if rows is None else rows.numel()
+            out = torch.empty((n, self.size), dtype=out_dtype or self.rt.act_dtype, device=h.device)
+            kernels.dual_norm(h, delta.terms, delta.bias, self.gain, self.eps, out, rows=rows, write_h=write_h)
+            return out
         if isinstance(delta, (PostNormed, WeightedSum)):
             n = h.shape[0] if rows is None else rows.numel()
             out = torch.empty((n, self.size), dtype=out_dtype or self.rt.act_dtype, device=h.device)
