@@ -11,6 +11,7 @@ B200.  A "step" is one decode step of a batch of 8 sequences from depth 2048
     python bench.py --design fusasun    # the Fusasun decoder beside the Tifapel decoder's attention layers, two sizes
     python bench.py --design soputar    # the Soputar decoder beside the Tifapel decoder's attention and retention layers and
                                         # the Fusasun decoder's latent layers, two sizes
+    python bench.py --design gebasun    # the Gebasun decoder beside the Tifapel decoder's retention and attention layers, two sizes
 
 ``value`` is device-timed (CUDA events around K steps queued back to back);
 ``e2e`` is the same metric through ``Session.generate`` with host token ids in
@@ -199,7 +200,7 @@ def main() -> int:
                          "one replayed decode step, when each kernel's dependency resolved")
     ap.add_argument("--cpu-baseline", action="store_true",
                     help="instead of the benchmark: time the plain implementation of tests/ on the CPU (tiny configurations)")
-    ap.add_argument("--design", choices=["tifapel", "voserax", "ninenex", "fusasun", "soputar"], default=None,
+    ap.add_argument("--design", choices=["tifapel", "voserax", "ninenex", "fusasun", "soputar", "gebasun"], default=None,
                     help="instead of the benchmark: prefill and decode rates of that design at layer sizes of a real "
                          "model (random weights), beside the dense Qwen3 decoder at equal sizes, with every kernel's "
                          "time per step (one JSON line of its own; the default workload is untouched)")
@@ -509,6 +510,19 @@ def soputar_layers(n_layers, heads, kv_heads, dim, kv_rank, ff):
     return out
 
 
+def gebasun_layers(n_layers, heads, kv_heads, dim, window, ssm_heads, ssm_dim, state, groups, experts, top, ff):
+    """Layers in the order state-space recurrence, attention with distance biases, state-space recurrence, rotated
+    attention with kept first tokens and an output gate; every layer with experts and a shared expert."""
+    moe = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top), shared=dict(ff=ff))
+    ssm = dict(type="mamba2", mlp=moe, mixer=dict(heads=ssm_heads, vdim=ssm_dim, state=state, groups=groups, conv=4,
+                                                  norm_groups=groups))
+    att = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5)
+    biased = dict(type="attention", mlp=moe, mixer=dict(att, mask=dict(size=window), bias_max=2 * window, bias_rows=32))
+    rotated = dict(type="attention_2", mlp=moe, mixer=dict(att, mask=dict(size=window, keep_first=4),
+                                                           rot=dict(dims=dim // 2, base=10000.0)))
+    return [json.loads(json.dumps((ssm, biased, ssm, rotated)[i % 4])) for i in range(n_layers)]
+
+
 def design_bench(args) -> int:
     """``--design tifapel``: prefill and decode rates of the Tifapel decoder at layer sizes that resemble a real model's (width 2048,
     16 heads of 128 on 4 key/value heads, a window of 1024 that keeps 4 tokens, 16 experts of 1024 of which a
@@ -534,7 +548,11 @@ def design_bench(args) -> int:
     ``--design soputar``: the same measurement of the Soputar decoder (attention with capped scores, the gated delta
     rule, latent attention over a cache of latents, attention on borrowed keys and values; dense feed-forwards) at two
     sizes, beside the Tifapel decoder with attention and retention layers in turn and the Fusasun decoder's latent
-    layers, all without a window that binds, with experts of the same active width."""
+    layers, all without a window that binds, with experts of the same active width.
+
+    ``--design gebasun``: the same measurement of the Gebasun decoder (the state-space recurrence of Mamba-2, attention
+    with distance biases, rotated attention with an output gate; experts without gates and a shared expert) at two
+    sizes, beside the Tifapel decoder with retention layers whose states are as large and windowed attention in turn."""
     import numpy as np
     import torch
 
@@ -616,6 +634,30 @@ def design_bench(args) -> int:
                               bf16_tflops=pk["bf16_tflops"], data="synthetic: seeded uniform token ids, random weights",
                               runs=runs)))
         return 0
+    if args.design == "gebasun":
+        runs = []
+        for width, heads, kv, dim, window, sh, sd, state, groups, E, top, ff in (
+                (2048, 16, 4, 128, 1024, 64, 64, 128, 2, 16, 2, 1024), (1024, 16, 8, 64, 512, 32, 64, 64, 1, 8, 2, 512)):
+            moe = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=E, top=top, scale=1.0))
+            decay = [1.0 - 2.0 ** -(3 + 7 * h / max(1, heads - 1)) for h in range(heads)]
+            # as many state elements and value columns as the state-space layers
+            ret = dict(type="retention", mlp=moe, mixer=dict(heads=heads, dim=state, vdim=sh * sd // heads, decay=decay))
+            att = dict(type="attention", mlp=moe, mixer=dict(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5,
+                                                             mask=dict(size=window, keep_first=4)))
+            models = {
+                "gebasun": dict(architecture="Gebasun", vocab=vocab, width=width, norm=dict(eps=1e-6),
+                                layers=gebasun_layers(L, heads, kv, dim, window, sh, sd, state, groups, E, top, ff)),
+                "tifapel": dict(architecture="Tifapel", vocab=vocab, width=width, norm=dict(eps=1e-6),
+                                layers=[json.loads(json.dumps(att if i % 2 else ret)) for i in range(L)]),
+            }
+            res = _design_models(args, models, vocab, T, B, depth, rng)
+            runs.append(dict(sizes=dict(width=width, heads=heads, kv_heads=kv, head_dim=dim, window=window, ssm_heads=sh,
+                                        ssm_head_dim=sd, state=state, groups=groups, conv=4, experts=E, top=top,
+                                        expert_ff=ff, shared_ff=ff, vocab=vocab), **res))
+        print(json.dumps(dict(design="gebasun", unit="tokens/s", dtype="bf16", layers=L, peaks=pk_src, hbm_gbs=pk["hbm_gbs"],
+                              bf16_tflops=pk["bf16_tflops"], data="synthetic: seeded uniform token ids, random weights",
+                              runs=runs)))
+        return 0
     if args.design == "ninenex":
         runs = []
         for width, heads, kv, dim, window, E, top, ff in ((2048, 16, 4, 128, 1024, 16, 2, 1024),
@@ -679,15 +721,18 @@ def _design_models(args, models, vocab, T, B, depth, rng) -> dict:
             f = raw_fn(lib, name, argtypes)
 
             def call(*a):
-                tag = name.replace("llmx_", "").replace("_capped", "")      # (the entry that also takes a cap's arguments)
+                # (the entries that also take a cap's and a bias's arguments)
+                tag = name.replace("llmx_", "").replace("_capped", "").replace("_biased", "")
                 if lib.endswith("_capped"):
                     tag += " (capped scores)"
+                elif lib.endswith("_biased"):
+                    tag += " (distance biases)"
                 if name.startswith("llmx_gemm_tc") and len(a) > 6:
                     tag += f" N{a[5]} K{a[6]}"
                 elif name == "llmx_gemm_fma":
                     tag += f" N{a[7]} K{a[8]}"
                 elif name == "llmx_moe_grouped_tc":
-                    tag += " gate|up" if a[13] else " down"
+                    tag += " gate|up" if a[13] == 1 else " up" if a[13] else " down"
                 elif name == "llmx_stream_mix_norm":
                     tag += " update+norm" if a[7] and a[14] else " norm" if a[14] else " update"
                 e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
