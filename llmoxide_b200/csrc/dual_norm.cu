@@ -53,7 +53,9 @@ __device__ __forceinline__ void dn_add_group(float4 (&v)[NC], const TD* p, int n
   }
 }
 
-template <typename TO, int NC>
+// DEEP: a step of few rows and many partials (a decode step): their loads are batched and the gains fetched ahead of the
+// wait; otherwise few registers, so that several rows share an SM.
+template <typename TO, int NC, bool DEEP>
 __global__ void __launch_bounds__(512)
 dual_norm_kernel(float* __restrict__ h, const DnGroup ga, const DnGroup gb, const float* __restrict__ bias,
                  const int* __restrict__ rows, const float* __restrict__ gain0, const float* __restrict__ gain1, float eps,
@@ -63,13 +65,13 @@ dual_norm_kernel(float* __restrict__ h, const DnGroup ga, const DnGroup gb, cons
   const int r = blockIdx.x;
   const int t = rows ? rows[r] : r;                     // a step input, not a result of the kernel before
   float* hrow = h + (size_t)t * d;
-  constexpr int J = NC == 1 ? 8 : NC == 2 ? 4 : 2;
+  constexpr int J = !DEEP ? (NC == 1 ? 2 : 1) : NC == 1 ? 8 : NC == 2 ? 4 : 2;
   float4 v[NC], g0[NC], g1[NC];
   int col[NC];
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     col[c] = (c * blockDim.x + threadIdx.x) * 4;
-    const bool live = col[c] < d;
+    const bool live = DEEP && col[c] < d;
     g0[c] = live && out0 ? dn_load4(gain0 + col[c]) : make_float4(0.f, 0.f, 0.f, 0.f);       // weights: ahead of the wait
     g1[c] = live && out1 ? dn_load4(gain1 + col[c]) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
@@ -101,6 +103,10 @@ dual_norm_kernel(float* __restrict__ h, const DnGroup ga, const DnGroup gb, cons
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     if (col[c] >= d) continue;
+    if (!DEEP) {
+      g0[c] = dn_load4(gain0 + col[c]);
+      if (out1) g1[c] = dn_load4(gain1 + col[c]);
+    }
     const float4 n = make_float4(v[c].x * rs, v[c].y * rs, v[c].z * rs, v[c].w * rs);
     dn_store4(out0 + (size_t)r * d + col[c], make_float4(n.x * g0[c].x, n.y * g0[c].y, n.z * g0[c].z, n.w * g0[c].w));
     if (out1) dn_store4(out1 + (size_t)r * d + col[c], make_float4(n.x * g1[c].x, n.y * g1[c].y, n.z * g1[c].z, n.w * g1[c].w));
@@ -171,7 +177,11 @@ LLMX_API int llmx_dual_norm(float* h, const void* a, int dtype_a, int n_a, long 
     const int nc = vecs <= 512 ? 1 : vecs <= 1024 ? 2 : 4;
     int threads = ((vecs + nc - 1) / nc + 31) / 32 * 32;
     if (threads < 64) threads = 64;
-#define GO(TO, NC) launch_pdl(dual_norm_kernel<TO, NC>, dim3(n_rows), dim3(threads), 0, stream, ARGS(TO))
+#define GO(TO, NC)                                                                                                \
+  do {                                                                                                            \
+    if (n_rows <= 64) launch_pdl(dual_norm_kernel<TO, NC, true>, dim3(n_rows), dim3(threads), 0, stream, ARGS(TO)); \
+    else launch_pdl(dual_norm_kernel<TO, NC, false>, dim3(n_rows), dim3(threads), 0, stream, ARGS(TO));           \
+  } while (0)
     if (out_bf16) {
       if (nc == 1) GO(bf16, 1); else if (nc == 2) GO(bf16, 2); else GO(bf16, 4);
     } else {

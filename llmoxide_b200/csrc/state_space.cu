@@ -23,7 +23,7 @@
 //   ss_pass    walks a sequence's chunks in order: leaves every chunk its E and the sequence its new state; moves the ring
 //   ss_out     per (chunk, head): the outputs, times silu(z)
 //   ss_norm    the norm
-// The products run on the FMA units from tiles in shared memory, 4 x 4 results a thread: the recurrence is float32 by the
+// The products run on the FMA units from tiles in shared memory, 8 x 8 results a thread: the recurrence is float32 by the
 // design, which the tensor cores' formats are not.  Single tokens: ss_decode, one CTA per (sequence, head), S read and
 // written once; then ss_norm.
 //
@@ -36,7 +36,7 @@
 #define SS_MAX_TAPS 16
 #define SS_LDM 68                // row stride of the masked 64 x 64 matrix in shared memory: 16-byte stores meet no bank twice
 
-__device__ __forceinline__ float ss_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float ss_silu(float x) { return __fdividef(x, 1.0f + expf(-x)); }   // (quotient within 2 ulp)
 __device__ __forceinline__ float ss_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float4 ss_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ void ss_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
@@ -69,9 +69,10 @@ __device__ __forceinline__ int ss_find_seq(const int* seq_start, int n_seqs, int
 
 // ---------------------------------------------------------------------------
 // One thread per channel and run of SS_RUN tokens of one sequence.  xs [T][H][Pp], bs and cs [T][G][Np], da [H][T] (a, dt).
-// TAPS > 0: compiled for that many taps, the run's rows asked for together; 0: any number.
+// TAPS > 0: compiled for that many taps, the run's rows asked for together; 0: any number.  SPLIT: the projection comes as
+// partials.
 // ---------------------------------------------------------------------------
-template <int TAPS>
+template <int TAPS, bool SPLIT>
 __global__ void __launch_bounds__(128)
 ss_prep_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ conv_w, const float* __restrict__ conv_b,
                const float* __restrict__ a_log, const float* __restrict__ dt_bias, const float* __restrict__ state,
@@ -90,6 +91,7 @@ ss_prep_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ con
     return;
   }
   const int n = min(SS_RUN, n_new - first);
+  auto proj_at = [&](int t, int c) { return SPLIT ? proj.at(t, c) : proj.p[(size_t)t * proj.row_stride + c]; };
   const int taps = TAPS > 0 ? TAPS : dm.taps;
   pdl_wait();
   if (c >= C + dm.H) return;
@@ -99,7 +101,7 @@ ss_prep_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ con
     const int col = dm.inner() + C + h;
     float z[SS_RUN];
 #pragma unroll
-    for (int i = 0; i < SS_RUN; ++i) z[i] = i < n ? proj.at(row0 + first + i, col) : 0.f;
+    for (int i = 0; i < SS_RUN; ++i) z[i] = i < n ? proj_at(row0 + first + i, col) : 0.f;
 #pragma unroll
     for (int i = 0; i < SS_RUN; ++i)
       if (i < n) {
@@ -111,7 +113,7 @@ ss_prep_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ con
   const float* ring = state + (size_t)sl * slot_stride + ring_off;
   const int col = dm.inner() + c;
   auto u_at = [&](int i) {                                            // the projected row i tokens into the sequence's new ones
-    if (i >= 0) return proj.at(row0 + i, col);
+    if (i >= 0) return proj_at(row0 + i, col);
     return p0 + i >= 0 ? ring[(size_t)((p0 + i) % taps) * C + c] : 0.f;
   };
   float y[SS_RUN];
@@ -160,23 +162,39 @@ ss_prep_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ con
 }
 
 // ---------------------------------------------------------------------------
-// acc[r][c] += sum_k A[k][i0 + r] B[k][j0 + c]: K rows of 64 results in shared memory, 256 threads, 4 x 4 each.  A warp
-// covers 16 rows x 32 columns, so that a row of A costs it one 64-byte and a row of B one 128-byte read.
+// acc[r][c] += sum_k A[k][row r] B[k][col c]: K rows of 64 results in shared memory, 64 threads, 8 x 8 results each, so that
+// the four 16-byte reads a thread makes per k (512 bytes a warp each, 128 a cycle) last as long as its 64 multiply-adds.
+// A thread's rows are i0 .. i0+3 and i0+32 .. i0+35, its columns j0 .. j0+3 and j0+32 .. j0+35: neighbouring lanes read
+// neighbouring 16 bytes.
 // ---------------------------------------------------------------------------
-__device__ __forceinline__ int ss_row0() { return ((threadIdx.x >> 6) * 4 + ((threadIdx.x & 31) >> 3)) * 4; }
-__device__ __forceinline__ int ss_col0() { return (((threadIdx.x >> 5) & 1) * 8 + (threadIdx.x & 7)) * 4; }
-__device__ __forceinline__ void ss_product(float (&acc)[4][4], const float* A, int lda, const float* B, int ldb, int K) {
+#define SS_THREADS 64
+__device__ __forceinline__ int ss_row0() { return (threadIdx.x >> 3) * 4; }
+__device__ __forceinline__ int ss_col0() { return (threadIdx.x & 7) * 4; }
+__device__ __forceinline__ void ss_product(float (&acc)[8][8], const float* A, int lda, const float* B, int ldb, int K) {
   const float* ap = A + ss_row0();
   const float* bp = B + ss_col0();
-#pragma unroll 8
+#pragma unroll 4
   for (int k = 0; k < K; ++k) {
-    const float4 a = ss_load4(ap + (size_t)k * lda), b = ss_load4(bp + (size_t)k * ldb);
-    const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+    const float4 a0 = ss_load4(ap + k * lda), a1 = ss_load4(ap + k * lda + 32);
+    const float4 b0 = ss_load4(bp + k * ldb), b1 = ss_load4(bp + k * ldb + 32);
+    const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+    const float bv[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
 #pragma unroll
-    for (int r = 0; r < 4; ++r)
+    for (int r = 0; r < 8; ++r)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) acc[r][c] = fmaf(av[r], bv[c], acc[r][c]);
+      for (int c = 0; c < 8; ++c) acc[r][c] = fmaf(av[r], bv[c], acc[r][c]);
   }
+}
+__device__ __forceinline__ int ss_row(int i0, int r) { return i0 + (r & 3) + ((r & 4) << 3); }   // the r-th of a thread's rows
+__device__ __forceinline__ void ss_copy16(float* dst, const float* src, bool live) {             // 16 bytes, or zeros
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src),
+               "r"(live ? 16 : 0)
+               : "memory");
+}
+__device__ __forceinline__ void ss_copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void ss_copy_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
 // The chunk of a slot: its sequence, first token, number of tokens (0: none) and number within the sequence.
@@ -196,7 +214,7 @@ __device__ __forceinline__ SsChunk ss_chunk_of(const int* seq_start, int n_seqs,
 
 // st [slots][H][N][Pp]: the chunk's own part of its last state; at [slots][H]: gamma of its last token; cb [slots][G][64][64]:
 // C_i . B_j at row j, column i.
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(SS_THREADS)
 ss_chunk_kernel(const float* __restrict__ xs, const float* __restrict__ bs, const float* __restrict__ cs,
                 const float2* __restrict__ da, float* __restrict__ st, float* __restrict__ at, float* __restrict__ cb,
                 const int* __restrict__ seq_start, int n_seqs, int n_tokens, const SsDims dm) {
@@ -209,11 +227,11 @@ ss_chunk_kernel(const float* __restrict__ xs, const float* __restrict__ bs, cons
   if (ck.n <= 0) return;                               // (uniform)
   const int Np = dm.Np(), Pp = dm.Pp();
   const int p_tiles = (Pp + 63) >> 6, tiles = ((dm.N + 63) >> 6) * p_tiles;
-  float acc[4][4];
+  float acc[8][8];
 #pragma unroll
-  for (int r = 0; r < 4; ++r)
+  for (int r = 0; r < 8; ++r)
 #pragma unroll
-    for (int c = 0; c < 4; ++c) acc[r][c] = 0.f;
+    for (int c = 0; c < 8; ++c) acc[r][c] = 0.f;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   const int i0 = ss_row0(), j0 = ss_col0();
   pdl_wait();
@@ -221,16 +239,23 @@ ss_chunk_kernel(const float* __restrict__ xs, const float* __restrict__ bs, cons
     const int h = blockIdx.y / tiles, tl = blockIdx.y - h * tiles;
     const int n0 = (tl / p_tiles) * 64, c0 = (tl % p_tiles) * 64;
     const int g = h / (dm.H / dm.G);
-    // sixteen columns' quarter of a token's row per thread: both tiles are asked for before the weights are made
-    const int j = tid >> 2, q = (tid & 3) * 4;
-    float4 bv[4], xv[4];
-    const float* brow = bs + ((size_t)(ck.t0 + j) * dm.G + g) * Np + n0;
-    const float* xrow = xs + ((size_t)(ck.t0 + j) * dm.H + h) * Pp + c0;
+    // 16 lanes a row: x goes straight to shared memory, B through registers, where it takes its token's weight
+    const int lr = tid >> 4, lc = (tid & 15) * 4;
+    const float* brow = bs + ((size_t)ck.t0 * dm.G + g) * Np + n0 + lc;
+    const float* xrow = xs + ((size_t)ck.t0 * dm.H + h) * Pp + c0 + lc;
+    const bool b_live = n0 + lc < Np, x_live = c0 + lc < Pp;
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      const int c = q + 16 * m;
-      bv[m] = j < ck.n && n0 + c < Np ? ss_load4(brow + c) : zero;
-      xv[m] = j < ck.n && c0 + c < Pp ? ss_load4(xrow + c) : zero;
+    for (int m = 0; m < 16; ++m) {
+      const int j = lr + 4 * m;
+      const bool live = x_live && j < ck.n;
+      ss_copy16(Bs + j * 64 + lc, live ? xrow + (size_t)j * dm.H * Pp : xs, live);
+    }
+    ss_copy_commit();
+    float4 bv[16];
+#pragma unroll
+    for (int m = 0; m < 16; ++m) {
+      const int j = lr + 4 * m;
+      bv[m] = b_live && j < ck.n ? ss_load4(brow + (size_t)j * dm.G * Np) : zero;
     }
     if (tid < 32) {
       // w_j = (a_(j+1) .. a_last) dt_j, two tokens a lane, by a suffix product over the warp
@@ -250,48 +275,55 @@ ss_chunk_kernel(const float* __restrict__ xs, const float* __restrict__ bs, cons
       if (tid == 0 && tl == 0) at[(size_t)slot * dm.H + h] = v;
     }
     __syncthreads();
-    const float w = ws[j];
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      ss_store4(As + j * 64 + q + 16 * m, make_float4(bv[m].x * w, bv[m].y * w, bv[m].z * w, bv[m].w * w));
-      ss_store4(Bs + j * 64 + q + 16 * m, xv[m]);
+    for (int m = 0; m < 16; ++m) {
+      const int j = lr + 4 * m;
+      const float w = ws[j];
+      ss_store4(As + j * 64 + lc, make_float4(bv[m].x * w, bv[m].y * w, bv[m].z * w, bv[m].w * w));
     }
+    ss_copy_wait<0>();
     __syncthreads();
-    ss_product(acc, As, 64, Bs, 64, (ck.n + 7) & ~7);   // (rows past the chunk's tokens are zero)
-    float* dst = st + (((size_t)slot * dm.H + h) * dm.N + n0 + i0) * Pp + c0 + j0;
-    if (c0 + j0 < Pp)
+    ss_product(acc, As, 64, Bs, 64, (ck.n + 3) & ~3);   // (rows past the chunk's tokens are zero)
+    float* dst = st + ((size_t)slot * dm.H + h) * dm.N * Pp + c0 + j0;
 #pragma unroll
-      for (int r = 0; r < 4; ++r)
-        if (n0 + i0 + r < dm.N) ss_store4(dst + (size_t)r * Pp, make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]));
+    for (int r = 0; r < 8; ++r) {
+      const int n = n0 + ss_row(i0, r);
+      if (n >= dm.N) continue;
+      if (c0 + j0 < Pp) ss_store4(dst + (size_t)n * Pp, make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]));
+      if (c0 + j0 + 32 < Pp) ss_store4(dst + (size_t)n * Pp + 32, make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]));
+    }
     return;
   }
   // ---- C_i . B_j of a group: both operands are turned so that a row of shared memory holds one dim of all tokens
   const int g = blockIdx.y - dm.H * tiles;
-  const int i = tid & 63, q = (tid >> 6) * 4;
-  for (int kb = 0; kb < Np; kb += 64) {
-    const float* crow = cs + ((size_t)(ck.t0 + i) * dm.G + g) * Np + kb;
-    const float* brow = bs + ((size_t)(ck.t0 + i) * dm.G + g) * Np + kb;
-    float4 cv[4], bv[4];
+  const float* crow = cs + ((size_t)(ck.t0 + tid) * dm.G + g) * Np;
+  const float* brow = bs + ((size_t)(ck.t0 + tid) * dm.G + g) * Np;
+  const bool live = tid < ck.n;
+  for (int kb = 0; kb < Np; kb += 32) {
+    float4 cv[8], bv[8];
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      const bool live = i < ck.n && kb + q + 16 * m < Np;
-      cv[m] = live ? ss_load4(crow + q + 16 * m) : zero;
-      bv[m] = live ? ss_load4(brow + q + 16 * m) : zero;
+    for (int m = 0; m < 8; ++m) {
+      cv[m] = live && kb + 4 * m < Np ? ss_load4(crow + kb + 4 * m) : zero;
+      bv[m] = live && kb + 4 * m < Np ? ss_load4(brow + kb + 4 * m) : zero;
     }
     __syncthreads();                                   // (the tiles of the block before have been read)
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      float* ap = As + (q + 16 * m) * 64 + i;
-      float* bp = Bs + (q + 16 * m) * 64 + i;
+    for (int m = 0; m < 8; ++m) {
+      float* ap = As + 4 * m * 64 + tid;
+      float* bp = Bs + 4 * m * 64 + tid;
       ap[0] = cv[m].x, ap[64] = cv[m].y, ap[128] = cv[m].z, ap[192] = cv[m].w;
       bp[0] = bv[m].x, bp[64] = bv[m].y, bp[128] = bv[m].z, bp[192] = bv[m].w;
     }
     __syncthreads();
-    ss_product(acc, As, 64, Bs, 64, min(64, Np - kb));
+    ss_product(acc, As, 64, Bs, 64, min(32, Np - kb));
   }
   float* dst = cb + ((size_t)slot * dm.G + g) * 4096;
 #pragma unroll
-  for (int c = 0; c < 4; ++c) ss_store4(dst + (j0 + c) * 64 + i0, make_float4(acc[0][c], acc[1][c], acc[2][c], acc[3][c]));
+  for (int c = 0; c < 8; ++c) {
+    float* row = dst + ss_row(j0, c) * 64 + i0;
+    ss_store4(row, make_float4(acc[0][c], acc[1][c], acc[2][c], acc[3][c]));
+    ss_store4(row + 32, make_float4(acc[4][c], acc[5][c], acc[6][c], acc[7][c]));
+  }
 }
 
 // Every four elements of a sequence's state, one thread: E_0 is the stored state, E_(c+1) = at_c E_c + st_c; st_c becomes
@@ -356,15 +388,14 @@ ss_pass_kernel(const SsProj proj, const SsDims dm, float* __restrict__ st, const
 }
 
 // y [T][inner] = (recurrence's output + D x) silu(z), 64 tokens x 64 columns of a head per CTA.
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(SS_THREADS)
 ss_out_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ xs, const float* __restrict__ cs,
               const float2* __restrict__ da, const float* __restrict__ st, const float* __restrict__ cb,
               const float* __restrict__ skip, float* __restrict__ y, const int* __restrict__ seq_start, int n_seqs,
               int n_tokens) {
-  __shared__ __align__(16) float Ms[64 * SS_LDM];      // row j: L_ij (C_i . B_j) dt_j over i
-  __shared__ __align__(16) float As[32 * 64];
-  __shared__ __align__(16) float Bs[32 * 64];
-  __shared__ float a_s[SS_CHUNK], dt_s[SS_CHUNK], gamma[SS_CHUNK];
+  __shared__ __align__(16) float Ms[64 * SS_LDM];      // row j: L_ij (C_i . B_j) dt_j over i; before that the turned C
+  __shared__ __align__(16) float Bs[2][32 * 64];       // rows of E, then of x
+  __shared__ float a_s[SS_CHUNK], gamma[SS_CHUNK];
   pdl_launch_dependents();
   const int tid = threadIdx.x, slot = blockIdx.x;
   const SsChunk ck = ss_chunk_of(seq_start, n_seqs, n_tokens, slot);
@@ -374,121 +405,133 @@ ss_out_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ xs, 
   const int g = h / (dm.H / dm.G);
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   pdl_wait();
-  if (tid < SS_CHUNK) {
-    const float2 e = tid < ck.n ? da[(size_t)h * n_tokens + ck.t0 + tid] : make_float2(1.f, 0.f);
-    a_s[tid] = e.x, dt_s[tid] = e.y;
-  }
-  // phase 1's tiles: C turned (a thread takes one token's dims), E as it lies
-  const int ai = tid & 63, aq = (tid >> 6) * 4;        // token, dims aq .. aq+3 and 16 further
-  const int br = tid >> 3, bc = (tid & 7) * 4;         // row of E or x, columns bc .. bc+3 and 32 further
-  const float* crow = cs + ((size_t)(ck.t0 + ai) * dm.G + g) * Np;
-  const float* e_base = st + ((size_t)slot * dm.H + h) * dm.N * Pp + c0;
-  const float* x_base = xs + ((size_t)ck.t0 * dm.H + h) * Pp + c0;
-  float4 av[2], bv[2];
-  auto fetch_state = [&](int kb) {
+  const int lr = tid >> 4, lc = (tid & 15) * 4;        // a row of E or x: 16 lanes
+  const bool col_live = c0 + lc < Pp;
+  const float* e_base = st + ((size_t)slot * dm.H + h) * dm.N * Pp + c0 + lc;
+  const float* x_base = xs + ((size_t)ck.t0 * dm.H + h) * Pp + c0 + lc;
+  const float* crow = cs + ((size_t)(ck.t0 + tid) * dm.G + g) * Np;
+  const int e_steps = (dm.N + 31) >> 5, steps = e_steps + ((ck.n + 31) >> 5);
+  auto copy_rows = [&](int step) {                      // 32 rows of E, then of x, into one of two buffers
+    float* dst = Bs[step & 1] + lc;
 #pragma unroll
-    for (int m = 0; m < 2; ++m) {
-      av[m] = ai < ck.n && kb + aq + 16 * m < Np ? ss_load4(crow + kb + aq + 16 * m) : zero;
-      bv[m] = kb + br < dm.N && c0 + bc + 32 * m < Pp ? ss_load4(e_base + (size_t)(kb + br) * Pp + bc + 32 * m) : zero;
+    for (int m = 0; m < 8; ++m) {
+      const int r = lr + 4 * m, k = (step < e_steps ? step : step - e_steps) * 32 + r;
+      const bool live = col_live && (step < e_steps ? k < dm.N : k < ck.n);
+      const float* src = step < e_steps ? e_base + (size_t)k * Pp : x_base + (size_t)k * dm.H * Pp;
+      ss_copy16(dst + r * 64, live ? src : xs, live);
     }
+    ss_copy_commit();
   };
-  auto fetch_x = [&](int jb) {
+  float4 cv[8];
+  auto fetch_c = [&](int kb) {
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
-      bv[m] = jb + br < ck.n && c0 + bc + 32 * m < Pp ? ss_load4(x_base + (size_t)(jb + br) * dm.H * Pp + bc + 32 * m) : zero;
+    for (int m = 0; m < 8; ++m) cv[m] = tid < ck.n && kb + 4 * m < Np ? ss_load4(crow + kb + 4 * m) : zero;
   };
-  fetch_state(0);
-  __syncthreads();
-  {
-    // L_ij by multiplying a along i, a quarter of the column per thread; what lies above the diagonal is zero
-    const int j = tid & 63, q = tid >> 6, i_lo = 16 * q;
-    const float* cbj = cb + (((size_t)slot * dm.G + g) * 64 + j) * 64 + i_lo;
-    float4 d[4];
+  copy_rows(0);
+  fetch_c(0);
+  const float2 own = tid < ck.n ? da[(size_t)h * n_tokens + ck.t0 + tid] : make_float2(1.f, 0.f);    // this token's a and dt
+  a_s[tid] = own.x;
+  float acc[8][8];
 #pragma unroll
-    for (int m = 0; m < 4; ++m) d[m] = i_lo + 15 >= j ? ss_load4(cbj + 4 * m) : zero;
-    float L = 1.f;
-    for (int i = j + 1; i < i_lo; ++i) L *= a_s[i];
-    const float dt = dt_s[j];
+  for (int r = 0; r < 8; ++r)
 #pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      float o[4] = {d[m].x, d[m].y, d[m].z, d[m].w};
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = i_lo + 4 * m + e;
-        if (i > j) L *= a_s[i];
-        o[e] = i >= j ? o[e] * L * dt : 0.f;
-      }
-      ss_store4(Ms + j * SS_LDM + i_lo + 4 * m, make_float4(o[0], o[1], o[2], o[3]));
-    }
-    if (tid < 32) {                                    // gamma, two tokens a lane, by a prefix product over the warp
-      const float a0 = a_s[2 * tid], a1 = a_s[2 * tid + 1];
-      float v = a0 * a1;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float u = __shfl_up_sync(0xffffffffu, v, o);
-        if (tid >= o) v *= u;
-      }
-      float before = __shfl_up_sync(0xffffffffu, v, 1);
-      if (tid == 0) before = 1.f;
-      gamma[2 * tid] = before * a0;
-      gamma[2 * tid + 1] = before * a0 * a1;
-    }
-  }
-  __syncthreads();
-  float acc[4][4];
-#pragma unroll
-  for (int r = 0; r < 4; ++r)
-#pragma unroll
-    for (int c = 0; c < 4; ++c) acc[r][c] = 0.f;
-  const float ga = gamma[ai];
-  for (int kb = 0; kb < Np; kb += 32) {
-#pragma unroll
-    for (int m = 0; m < 2; ++m) {
-      float* ap = As + (aq + 16 * m) * 64 + ai;
-      ap[0] = av[m].x * ga, ap[64] = av[m].y * ga, ap[128] = av[m].z * ga, ap[192] = av[m].w * ga;
-      ss_store4(Bs + br * 64 + bc + 32 * m, bv[m]);
-    }
-    __syncthreads();
-    if (kb + 32 < Np) fetch_state(kb + 32);
-    else fetch_x(0);
-    ss_product(acc, As, 64, Bs, 64, min(32, Np - kb));
-    __syncthreads();
-  }
+    for (int c = 0; c < 8; ++c) acc[r][c] = 0.f;
   const int i0 = ss_row0(), j0 = ss_col0();
-  const int row_end = ((tid >> 6) + 1) * 16;           // the warp's rows end here: later tokens do not reach them
-  for (int jb = 0; jb < ck.n; jb += 32) {
+  // ---- E^T C_i
+  for (int s = 0; s < e_steps; ++s) {
+    float* As = Ms + (s & 1) * 32 * 64;
 #pragma unroll
-    for (int m = 0; m < 2; ++m) ss_store4(Bs + br * 64 + bc + 32 * m, bv[m]);
+    for (int m = 0; m < 8; ++m) {                      // C turned: a row of shared memory holds one dim of all tokens
+      float* ap = As + 4 * m * 64 + tid;
+      ap[0] = cv[m].x, ap[64] = cv[m].y, ap[128] = cv[m].z, ap[192] = cv[m].w;
+    }
+    ss_copy_wait<0>();
+    __syncthreads();                                   // (and every thread is done with the tiles of the step before)
+    copy_rows(s + 1);
+    if (s + 1 < e_steps) fetch_c((s + 1) * 32);
+    ss_product(acc, As, 64, Bs[s & 1], 64, min(32, Np - s * 32));
+  }
+  __syncthreads();                                     // the turned C has been read: its place takes the masked matrix
+  if (tid < 32) {                                      // gamma, two tokens a lane, by a prefix product over the warp
+    const float a0 = a_s[2 * tid], a1 = a_s[2 * tid + 1];
+    float v = a0 * a1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float u = __shfl_up_sync(0xffffffffu, v, o);
+      if (tid >= o) v *= u;
+    }
+    float before = __shfl_up_sync(0xffffffffu, v, 1);
+    if (tid == 0) before = 1.f;
+    gamma[2 * tid] = before * a0;
+    gamma[2 * tid + 1] = before * a0 * a1;
+  }
+  {
+    // L_ij by multiplying a along i, a thread a column j; what lies above the diagonal is zero
+    const float* cbj = cb + (((size_t)slot * dm.G + g) * 64 + tid) * 64;
+    float L = own.y;                                   // (dt_j rides on it)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      float4 d[4];
+#pragma unroll
+      for (int m = 0; m < 4; ++m) d[m] = 16 * q + 15 >= tid ? ss_load4(cbj + 16 * q + 4 * m) : zero;
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        float o[4] = {d[m].x, d[m].y, d[m].z, d[m].w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = 16 * q + 4 * m + e;
+          if (i > tid) L *= a_s[i];
+          o[e] = i >= tid ? o[e] * L : 0.f;
+        }
+        ss_store4(Ms + tid * SS_LDM + 16 * q + 4 * m, make_float4(o[0], o[1], o[2], o[3]));
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int r = 0; r < 8; ++r) {
+    const float ga = gamma[ss_row(i0, r)];
+#pragma unroll
+    for (int c = 0; c < 8; ++c) acc[r][c] *= ga;
+  }
+  // ---- + sum over the chunk's own tokens
+  for (int s = e_steps; s < steps; ++s) {
+    ss_copy_wait<0>();
     __syncthreads();
-    if (jb + 32 < ck.n) fetch_x(jb + 32);
-    ss_product(acc, Ms + jb * SS_LDM, SS_LDM, Bs, 64, min(32, max(0, row_end - jb)));
-    __syncthreads();
+    if (s + 1 < steps) copy_rows(s + 1);
+    const int jb = (s - e_steps) * 32;
+    ss_product(acc, Ms + jb * SS_LDM, SS_LDM, Bs[s & 1], 64, min(32, ck.n - jb));
   }
   // ---- + D x, times silu(z)
-  const int inner = dm.inner(), p = c0 + j0;
-  if (p >= dm.P) return;
+  const int inner = dm.inner();
   const float dsk = skip[h];
   const bool vec = (dm.P & 3) == 0 && (proj.row_stride & 3) == 0 && (proj.split_stride & 3) == 0;
 #pragma unroll
-  for (int r = 0; r < 4; ++r) {
-    const int i = i0 + r;
-    if (i >= ck.n) break;
+  for (int r = 0; r < 8; ++r) {
+    const int i = ss_row(i0, r);
+    if (i >= ck.n) continue;
     const size_t t = (size_t)(ck.t0 + i);
-    const float4 x = ss_load4(xs + (t * dm.H + h) * Pp + p);
-    float v[4] = {fmaf(dsk, x.x, acc[r][0]), fmaf(dsk, x.y, acc[r][1]), fmaf(dsk, x.z, acc[r][2]), fmaf(dsk, x.w, acc[r][3])};
-    float* dst = y + t * inner + (size_t)h * dm.P + p;
-    if (vec) {
-      const float* zp = proj.p + t * proj.row_stride + h * dm.P + p;
-      float4 z = ss_load4(zp);
-      for (int s = 1; s < proj.n_split; ++s) {
-        const float4 u = ss_load4(zp + (size_t)s * proj.split_stride);
-        z.x += u.x, z.y += u.y, z.z += u.z, z.w += u.w;
-      }
-      ss_store4(dst, make_float4(v[0] * ss_silu(z.x), v[1] * ss_silu(z.y), v[2] * ss_silu(z.z), v[3] * ss_silu(z.w)));
-    } else {
 #pragma unroll
-      for (int c = 0; c < 4; ++c)
-        if (p + c < dm.P) dst[c] = v[c] * ss_silu(proj.at(t, h * dm.P + p + c));
+    for (int half = 0; half < 2; ++half) {
+      const int p = c0 + j0 + 32 * half;
+      if (p >= dm.P) continue;
+      const float4 x = ss_load4(xs + (t * dm.H + h) * Pp + p);
+      const float* ar = acc[r] + 4 * half;
+      float v[4] = {fmaf(dsk, x.x, ar[0]), fmaf(dsk, x.y, ar[1]), fmaf(dsk, x.z, ar[2]), fmaf(dsk, x.w, ar[3])};
+      float* dst = y + t * inner + (size_t)h * dm.P + p;
+      if (vec) {
+        const float* zp = proj.p + t * proj.row_stride + h * dm.P + p;
+        float4 z = ss_load4(zp);
+        for (int q = 1; q < proj.n_split; ++q) {
+          const float4 u = ss_load4(zp + (size_t)q * proj.split_stride);
+          z.x += u.x, z.y += u.y, z.z += u.z, z.w += u.w;
+        }
+        ss_store4(dst, make_float4(v[0] * ss_silu(z.x), v[1] * ss_silu(z.y), v[2] * ss_silu(z.z), v[3] * ss_silu(z.w)));
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (p + c < dm.P) dst[c] = v[c] * ss_silu(proj.at(t, h * dm.P + p + c));
+      }
     }
   }
 }
@@ -550,7 +593,7 @@ __device__ __forceinline__ void ss_loadv(const float* p, float (&o)[V]) {
 }
 
 template <int V>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 4)
 ss_decode_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ conv_w, const float* __restrict__ conv_b,
                  const float* __restrict__ a_log, const float* __restrict__ dt_bias, const float* __restrict__ skip,
                  float* __restrict__ state, size_t slot_stride, size_t ring_off, float* __restrict__ y,
@@ -663,8 +706,13 @@ LLMX_API int llmx_ss_prompt(const float* proj, int n_split, long long split_stri
   const int runs = n_tokens / SS_RUN + n_seqs, chunks = n_tokens / SS_CHUNK + n_seqs;
   if ((long long)H * p_tiles * n_tiles + G > 65535) return LLMX_REFUSED(3);
   const dim3 pgrid(runs, (C + H + 127) / 128);
-#define PREP(TAPS)                                                                                                       \
-  launch_pdl(ss_prep_kernel<TAPS>, pgrid, dim3(128), 0, stream, pr, dm, conv_w, conv_b, a_log, dt_bias, (const float*)state, \
+#define PREP(TAPS)                       \
+  do {                                    \
+    if (n_split > 1) PREP2(TAPS, true);   \
+    else PREP2(TAPS, false);              \
+  } while (0)
+#define PREP2(TAPS, SPLIT)                                                                                               \
+  launch_pdl(ss_prep_kernel<TAPS, SPLIT>, pgrid, dim3(128), 0, stream, pr, dm, conv_w, conv_b, a_log, dt_bias, (const float*)state, \
              (size_t)slot_stride, (size_t)ring_off, xs, bs, cs, (float2*)da, seq_start, seq_past, seq_slot, n_seqs,      \
              n_tokens, n_slots)
   switch (taps) {
@@ -674,13 +722,14 @@ LLMX_API int llmx_ss_prompt(const float* proj, int n_split, long long split_stri
     default: PREP(0); break;
   }
 #undef PREP
-  launch_pdl(ss_chunk_kernel, dim3(chunks, H * p_tiles * n_tiles + G), dim3(256), 0, stream, (const float*)xs,
+#undef PREP2
+  launch_pdl(ss_chunk_kernel, dim3(chunks, H * p_tiles * n_tiles + G), dim3(SS_THREADS), 0, stream, (const float*)xs,
              (const float*)bs, (const float*)cs, (const float2*)da, st, at, cb, seq_start, n_seqs, n_tokens, dm);
   const long long quads = (long long)H * N * (dm.Pp() / 4);
   const int state_blocks = (int)((quads + 255) / 256), ring_blocks = taps > 1 ? (C + 255) / 256 : 0;
   launch_pdl(ss_pass_kernel, dim3(state_blocks + ring_blocks, n_seqs), dim3(256), 0, stream, pr, dm, st, (const float*)at,
              state, (size_t)slot_stride, (size_t)ring_off, seq_start, seq_past, seq_slot, n_tokens, n_slots, state_blocks);
-  launch_pdl(ss_out_kernel, dim3(chunks, H * p_tiles), dim3(256), 0, stream, pr, dm, (const float*)xs, (const float*)cs,
+  launch_pdl(ss_out_kernel, dim3(chunks, H * p_tiles), dim3(SS_THREADS), 0, stream, pr, dm, (const float*)xs, (const float*)cs,
              (const float2*)da, (const float*)st, (const float*)cb, skip, y, seq_start, n_seqs, n_tokens);
   return LLMX_LAUNCH_STATUS();
 }

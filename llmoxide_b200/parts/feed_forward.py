@@ -122,7 +122,7 @@ class PlainMLP:
         # a step of few tokens streams the matrix: split over K where that keeps more SMs at it, the activation then sums
         # the partials; otherwise it is the product's epilogue
         if (tc is not None and x.dtype == torch.bfloat16 and kernels.gemm_tc_supports(x, tc.weight)
-                and self.rt.act_dtype == torch.bfloat16 and tc.splits(x.shape[0]) == 1):
+                and self.rt.act_dtype == torch.bfloat16 and (x.shape[0] > 64 or tc.splits(x.shape[0]) == 1)):
             return tc.activated(x, self.rt.act_dtype, self.activation)
         act = torch.empty((x.shape[0], self.F), dtype=self.rt.act_dtype, device=x.device)
         kernels.plain_act(self.up(x, out_dtype=torch.float32, splits_ok=True), act, self.activation)

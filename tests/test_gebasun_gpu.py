@@ -302,7 +302,7 @@ def test_one_token_seen_to_the_edge_of_the_window_and_not_beyond(tmp_path, kind,
             eng.release(slot)
             outs.append(np.concatenate([a] + b))
         want = plain.forward(cfg, w, toks).numpy()
-        assert ru.rel_err(outs[0], want) < (F32_TOL if dtype == "float32" else 3e-2), mark
+        assert ru.rel_err(outs[0], want) < (F32_TOL if dtype == "float32" else 8e-2), mark
         diff = np.abs(outs[0] - outs[1]).max(axis=1) / np.abs(want).max()
         seen = np.zeros(len(toks), bool)
         seen[mark : mark + window] = True

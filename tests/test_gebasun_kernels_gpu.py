@@ -123,10 +123,6 @@ def test_unit_norm_rotation_and_keys_stored_twice(H, G, D, rot, n_split, extra, 
     x = row.reshape(T, H + G, D)
     turned = x
     if rot:
-        full = torch.zeros((int(pos.max()) + 1, H + G, D), dtype=F)        # the plain rotation takes positions 0, 1, ..
-        for i, p in enumerate(pos):
-            full = full.clone()
-            full[p] = x[i]
         # positions of different sequences may coincide: turn them one at a time
         turned = torch.stack([plain.rotate_halves(torch.cat([torch.zeros((int(p), H + G, D), dtype=F), x[i : i + 1]]), rot,
                                                   base)[-1] for i, p in enumerate(pos)])
@@ -141,7 +137,8 @@ def test_unit_norm_rotation_and_keys_stored_twice(H, G, D, rot, n_split, extra, 
     q = torch.empty((T, H * D), dtype=dtype, device=DEV)
     ctx = _ctx(past, counts)
     kernels.qk_unit_rope_cache(pd, _f32(bias), q, kc, vc, table, ctx, eps, cos, sin, rot, H, G, D)
-    tol = 3e-6 if dtype == torch.float32 else 6e-3
+    # (angles are float32 products of position and frequency: up to 200 radians here)
+    tol = 2e-5 if dtype == torch.float32 else 6e-3
     assert _rel(q.float().reshape(T, H, D), unit[:, :H]) < tol
     at = 0
     for b, (p, n) in enumerate(zip(past, counts)):
