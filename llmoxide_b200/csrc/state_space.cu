@@ -170,19 +170,28 @@ ss_prep_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ con
 #define SS_THREADS 64
 __device__ __forceinline__ int ss_row0() { return (threadIdx.x >> 3) * 4; }
 __device__ __forceinline__ int ss_col0() { return (threadIdx.x & 7) * 4; }
+// Two multiply-adds in one instruction, each rounded like fmaf: (d.x, d.y) += a * (b.x, b.y).
+__device__ __forceinline__ void ss_fma2(float& dx, float& dy, float a, float bx, float by) {
+  asm("{\n.reg .b64 va, vb, vd;\nmov.b64 va, {%2, %2};\nmov.b64 vb, {%3, %4};\nmov.b64 vd, {%0, %1};\n"
+      "fma.rn.f32x2 vd, va, vb, vd;\nmov.b64 {%0, %1}, vd;\n}"
+      : "+f"(dx), "+f"(dy)
+      : "f"(a), "f"(bx), "f"(by));
+}
+// LOW false: only the rows from 32 on (a triangle's lower half has nothing above).
+template <int UNROLL, bool LOW = true>
 __device__ __forceinline__ void ss_product(float (&acc)[8][8], const float* A, int lda, const float* B, int ldb, int K) {
   const float* ap = A + ss_row0();
   const float* bp = B + ss_col0();
-#pragma unroll 4
+#pragma unroll UNROLL
   for (int k = 0; k < K; ++k) {
-    const float4 a0 = ss_load4(ap + k * lda), a1 = ss_load4(ap + k * lda + 32);
+    const float4 a0 = LOW ? ss_load4(ap + k * lda) : make_float4(0.f, 0.f, 0.f, 0.f), a1 = ss_load4(ap + k * lda + 32);
     const float4 b0 = ss_load4(bp + k * ldb), b1 = ss_load4(bp + k * ldb + 32);
     const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
     const float bv[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
 #pragma unroll
-    for (int r = 0; r < 8; ++r)
+    for (int r = LOW ? 0 : 4; r < 8; ++r)
 #pragma unroll
-      for (int c = 0; c < 8; ++c) acc[r][c] = fmaf(av[r], bv[c], acc[r][c]);
+      for (int c = 0; c < 8; c += 2) ss_fma2(acc[r][c], acc[r][c + 1], av[r], bv[c], bv[c + 1]);
   }
 }
 __device__ __forceinline__ int ss_row(int i0, int r) { return i0 + (r & 3) + ((r & 4) << 3); }   // the r-th of a thread's rows
@@ -283,7 +292,7 @@ ss_chunk_kernel(const float* __restrict__ xs, const float* __restrict__ bs, cons
     }
     ss_copy_wait<0>();
     __syncthreads();
-    ss_product(acc, As, 64, Bs, 64, (ck.n + 3) & ~3);   // (rows past the chunk's tokens are zero)
+    ss_product<4>(acc, As, 64, Bs, 64, (ck.n + 3) & ~3);   // (rows past the chunk's tokens are zero)
     float* dst = st + ((size_t)slot * dm.H + h) * dm.N * Pp + c0 + j0;
 #pragma unroll
     for (int r = 0; r < 8; ++r) {
@@ -315,7 +324,7 @@ ss_chunk_kernel(const float* __restrict__ xs, const float* __restrict__ bs, cons
       bp[0] = bv[m].x, bp[64] = bv[m].y, bp[128] = bv[m].z, bp[192] = bv[m].w;
     }
     __syncthreads();
-    ss_product(acc, As, 64, Bs, 64, min(32, Np - kb));
+    ss_product<4>(acc, As, 64, Bs, 64, min(32, Np - kb));
   }
   float* dst = cb + ((size_t)slot * dm.G + g) * 4096;
 #pragma unroll
@@ -449,7 +458,7 @@ ss_out_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ xs, 
     __syncthreads();                                   // (and every thread is done with the tiles of the step before)
     copy_rows(s + 1);
     if (s + 1 < e_steps) fetch_c((s + 1) * 32);
-    ss_product(acc, As, 64, Bs[s & 1], 64, min(32, Np - s * 32));
+    ss_product<2>(acc, As, 64, Bs[s & 1], 64, min(32, Np - s * 32));
   }
   __syncthreads();                                     // the turned C has been read: its place takes the masked matrix
   if (tid < 32) {                                      // gamma, two tokens a lane, by a prefix product over the warp
@@ -500,7 +509,8 @@ ss_out_kernel(const SsProj proj, const SsDims dm, const float* __restrict__ xs, 
     __syncthreads();
     if (s + 1 < steps) copy_rows(s + 1);
     const int jb = (s - e_steps) * 32;
-    ss_product(acc, Ms + jb * SS_LDM, SS_LDM, Bs[s & 1], 64, min(32, ck.n - jb));
+    if (jb == 0) ss_product<2>(acc, Ms, SS_LDM, Bs[s & 1], 64, min(32, ck.n));
+    else ss_product<2, false>(acc, Ms + jb * SS_LDM, SS_LDM, Bs[s & 1], 64, ck.n - jb);      // (they reach rows 32.. only)
   }
   // ---- + D x, times silu(z)
   const int inner = dm.inner();
