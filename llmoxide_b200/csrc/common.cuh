@@ -246,10 +246,11 @@ static inline ScoreBiasArg make_score_bias(const float*, int) { return NoScoreBi
 //   RELU            max(g, 0) * u
 //   CLAMPED_SWISH   g' sigmoid(slope g') * (u' + shift),  g' = min(g, limit),  u' = clamp(u, -limit, limit)
 //   GELU_TANH       0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u
-//   RELU_SQUARED    max(g, 0)^2 * u
-// A feed-forward without a gate applies the same function with u = 1.
+// A feed-forward without a gate applies act(g) alone (plain_act below), where there is one more kind:
+//   RELU_SQUARED    max(g, 0)^2
 enum { LLMX_ACT_SILU = 0, LLMX_ACT_RELU = 1, LLMX_ACT_CLAMPED_SWISH = 2, LLMX_ACT_GELU_TANH = 3, LLMX_ACT_RELU_SQUARED = 4 };
-#define LLMX_ACT_LAST LLMX_ACT_RELU_SQUARED
+#define LLMX_ACT_LAST LLMX_ACT_GELU_TANH            // the last kind that takes a gate
+#define LLMX_ACT_LAST_PLAIN LLMX_ACT_RELU_SQUARED
 struct GateAct {
   int kind;
   float slope, limit, shift;
@@ -259,7 +260,6 @@ struct GateAct {
 __device__ __forceinline__ float gated_act(const GateAct a, float g, float u) {
   if (a.kind == LLMX_ACT_SILU) return (g / (1.0f + expf(-g))) * u;
   if (a.kind == LLMX_ACT_RELU) return fmaxf(g, 0.f) * u;
-  if (a.kind == LLMX_ACT_RELU_SQUARED) return fmaxf(g, 0.f) * fmaxf(g, 0.f) * u;
   if (a.kind == LLMX_ACT_GELU_TANH) return (0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)))) * u;
   g = fminf(g, a.limit);
   u = fminf(fmaxf(u, -a.limit), a.limit);
@@ -269,7 +269,6 @@ __device__ __forceinline__ float gated_act(const GateAct a, float g, float u) {
 __device__ __forceinline__ float gated_act_fast(const GateAct a, float g, float u) {
   if (a.kind == LLMX_ACT_SILU) return __fdividef(g, 1.0f + __expf(-g)) * u;
   if (a.kind == LLMX_ACT_RELU) return fmaxf(g, 0.f) * u;
-  if (a.kind == LLMX_ACT_RELU_SQUARED) return fmaxf(g, 0.f) * fmaxf(g, 0.f) * u;
   if (a.kind == LLMX_ACT_GELU_TANH) {       // 0.5 (1 + tanh z) = 1 / (1 + exp(-2z))
     const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return __fdividef(g, 1.0f + __expf(-2.0f * z)) * u;
@@ -277,6 +276,15 @@ __device__ __forceinline__ float gated_act_fast(const GateAct a, float g, float 
   g = fminf(g, a.limit);
   u = fminf(fmaxf(u, -a.limit), a.limit);
   return __fdividef(g, 1.0f + __expf(-a.slope * g)) * (u + a.shift);
+}
+
+__device__ __forceinline__ float plain_act(const GateAct a, float x) {
+  const float r = fmaxf(x, 0.f);
+  return a.kind == LLMX_ACT_RELU_SQUARED ? r * r : gated_act(a, x, 1.0f);
+}
+__device__ __forceinline__ float plain_act_fast(const GateAct a, float x) {
+  const float r = fmaxf(x, 0.f);
+  return a.kind == LLMX_ACT_RELU_SQUARED ? r * r : gated_act_fast(a, x, 1.0f);
 }
 
 // Butterfly reductions: every lane ends with the same value, and the order of

@@ -754,7 +754,7 @@ LLMX_API int llmx_silu_gate(const void* gu, int in_dtype, int n_split, long long
 }
 
 // ---------------------------------------------------------------------------
-// The activation of a feed-forward without a gate: act[i] = gated_act(sum_s in[s][i], 1), in float32.
+// The activation of a feed-forward without a gate: act[i] = plain_act(sum_s in[s][i]), in float32.
 // ---------------------------------------------------------------------------
 template <typename TI, typename TO>
 __global__ void plain_act_kernel(const TI* __restrict__ in, int n_split, size_t split_stride, TO* __restrict__ act, size_t n,
@@ -762,13 +762,13 @@ __global__ void plain_act_kernel(const TI* __restrict__ in, int n_split, size_t 
   pdl_launch_dependents();
   pdl_wait();
   for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
-    act[i] = from_f32<TO>(gated_act(kind, split_value(in, i, n_split, split_stride), 1.0f));
+    act[i] = from_f32<TO>(plain_act(kind, split_value(in, i, n_split, split_stride)));
 }
 
 LLMX_API int llmx_plain_act(const void* in, int in_dtype, int n_split, long long split_stride, void* act, int out_dtype,
                             long long n, int act_kind, float slope, float limit, float shift, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (n_split < 1 || act_kind < LLMX_ACT_SILU || act_kind > LLMX_ACT_LAST) return LLMX_REFUSED(1);
+  if (n_split < 1 || act_kind < LLMX_ACT_SILU || act_kind > LLMX_ACT_LAST_PLAIN) return LLMX_REFUSED(1);
   const GateAct kind = {act_kind, slope, limit, shift};
   const long long want = (n + 255) / 256;
   const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);

@@ -114,7 +114,7 @@ __device__ __forceinline__ void epilogue_tile(uint32_t acc_addr, bool have_acc, 
         if (t < T) {
           float r = v[e];
           if (MODE == 1) r = gated_act_fast(act, r, g[e]);
-          if (MODE == 3) r = gated_act_fast(act, r, 1.0f);
+          if (MODE == 3) r = plain_act_fast(act, r);
           out[(size_t)t * ldy + n] = from_f32<TY>(r);
         }
       }
@@ -164,7 +164,7 @@ __device__ __forceinline__ void epilogue_tile_staged(uint32_t acc_addr, const CU
       }
     } else {
 #pragma unroll
-      for (int e = 0; e < ROWS; ++e) buf[e * COLS + col] = from_f32<TY>(MODE == 3 ? gated_act_fast(act, v[e], 1.0f) : v[e]);
+      for (int e = 0; e < ROWS; ++e) buf[e * COLS + col] = from_f32<TY>(MODE == 3 ? plain_act_fast(act, v[e]) : v[e]);
     }
     fence_proxy_async();
     asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -696,7 +696,7 @@ static int sm_count() {
 // set otherwise; kinds in common.cuh.
 static thread_local GateAct t_gate_act = {LLMX_ACT_SILU, 1.f, 0.f, 0.f, nullptr};
 LLMX_API int llmx_gemm_tc_gate_act(int kind, float slope, float limit, float shift) {
-  if (kind < LLMX_ACT_SILU || kind > LLMX_ACT_LAST) return LLMX_REFUSED(1);
+  if (kind < LLMX_ACT_SILU || kind > LLMX_ACT_LAST_PLAIN) return LLMX_REFUSED(1);
   t_gate_act = GateAct{kind, slope, limit, shift, t_gate_act.bias};
   return 0;
 }
@@ -751,7 +751,7 @@ static int launch(const CUtensorMap& mw, const CUtensorMap& mx, void* Y, int T, 
 // mode 1: W = [gate rows; up rows] with N = 2F; Y = act [T,F] of y_dtype.
 // mode 2: W = blocks of 32 rows, each 16 gate rows then the 16 up rows of the same features (N = 2F, F % 16 == 0);
 //         Y = act [T,F] bf16.
-// mode 3: Y [T,N] bf16 = act(product), act as for a gate with up = 1.
+// mode 3: Y [T,N] bf16 = act(product), without a gate.
 // The same with row scales applied in the epilogue (see TcScale): in_sumsq [in_parts][in_stride >= T], T <= 64.
 LLMX_API int llmx_gemm_tc_scaled(const void* X, const void* W, void* Y, int y_dtype, int T, int N, int K, long long ldx,
                                  long long ldw, long long ldy, int n_split, long long split_stride, int mode,
@@ -778,6 +778,7 @@ LLMX_API int llmx_gemm_tc_scaled(const void* X, const void* W, void* Y, int y_dt
   if (K <= 0 || (K % 8) || (ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return LLMX_REFUSED(1);
   if (n_split < 1 || (n_split > 1 && (mode != 0 || y_dtype != LLMX_F32))) return LLMX_REFUSED(1);
   if (mode < 0 || mode > 3 || (mode == 1 && (N % 2)) || (mode == 2 && (N % 32))) return LLMX_REFUSED(1);
+  if ((mode == 1 || mode == 2) && t_gate_act.kind > LLMX_ACT_LAST) return LLMX_REFUSED(1);
   const int F = mode == 1 || mode == 2 ? N / 2 : 0;
   int bn = 16;
   while (bn < T && bn < (mode == 1 ? 128 : 256)) bn <<= 1;
@@ -898,6 +899,7 @@ LLMX_API int llmx_gemm_tc_pair(const void* X, const void* W, void* Y, int y_dtyp
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || (K % 8) || (ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return LLMX_REFUSED(1);
   if (T <= 128 || mode < 0 || mode > 3 || (mode == 1 && (N % 2)) || (mode == 2 && (N % 32))) return LLMX_REFUSED(1);
+  if ((mode == 1 || mode == 2) && t_gate_act.kind > LLMX_ACT_LAST) return LLMX_REFUSED(1);
   const int F = mode == 1 || mode == 2 ? N / 2 : 0;
   const int bn = mode == 1 ? 128 : 256;
   CUtensorMap mw, mx;

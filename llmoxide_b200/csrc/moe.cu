@@ -452,7 +452,7 @@ moe_grouped_fma_kernel(const TX* __restrict__ X, long long ldx, const TW* __rest
       if constexpr (GATED) {
         Y[(size_t)(row0 + lr) * N + n] = from_f32<TY>(gated_act(act, acc[i][j], acu[i][j]));
       } else if constexpr (PLAIN) {
-        Y[(size_t)(row0 + lr) * N + n] = from_f32<TY>(gated_act(act, acc[i][j], 1.0f));
+        Y[(size_t)(row0 + lr) * N + n] = from_f32<TY>(plain_act(act, acc[i][j]));
       } else {
         const int t = pr / top, choice = pr - t * top;
         Y[((size_t)choice * n_tokens + t) * N + n] = from_f32<TY>(pair_weight[pr] * acc[i][j]);
@@ -469,7 +469,7 @@ LLMX_API int llmx_moe_grouped_fma(const void* X, int x_dtype, long long ldx, con
                                   const float* pair_weight, int top, int n_tokens, int N, int K, int gated,
                                   int act_kind, float slope, float limit, float shift, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (act_kind < LLMX_ACT_SILU || act_kind > LLMX_ACT_LAST) return LLMX_REFUSED(1);
+  if (act_kind < LLMX_ACT_SILU || act_kind > (gated == 2 ? LLMX_ACT_LAST_PLAIN : LLMX_ACT_LAST)) return LLMX_REFUSED(1);
   const GateAct act = {act_kind, slope, limit, shift};
   if (N <= 0 || K <= 0 || top <= 0 || max_tiles <= 0 || max_tiles > 65535 || ldx < K) return LLMX_REFUSED(1);
   if (x_dtype != w_dtype) return LLMX_REFUSED(2);

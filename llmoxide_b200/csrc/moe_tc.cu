@@ -13,7 +13,7 @@
 //
 //   MODE 1 (gate|up): two accumulators, rows n and n + F of the expert's [2F, K]; act[row, n] = gated_act(gate, up) (common.cuh)
 //   MODE 0 (down):    y[dest[row]][n] = weight[row] * acc, float32 (dest = choice * tokens + token, from the sort)
-//   MODE 2 (up):      act[row, n] = the activation of an expert without a gate (gated_act with up = 1)
+//   MODE 2 (up):      act[row, n] = the activation of an expert without a gate (plain_act)
 //
 // Which expert a unit reads is decided on the device by the kernel before, so every thread waits for that
 // kernel first.  Every wait on an mbarrier is bounded; when one runs out the CTA records it in the library's
@@ -198,7 +198,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
             if (MODE == 1) {
               Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(gated_act_fast(act, v[i], g[i]));
             } else if (MODE == 2) {
-              Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(gated_act_fast(act, v[i], 1.0f));
+              Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(plain_act_fast(act, v[i]));
             } else {
               Y[(size_t)tile_dest[r] * N + n] = from_f32<TY>(tile_weight[r] * v[i]);
             }
@@ -266,7 +266,7 @@ LLMX_API int llmx_moe_grouped_tc(const void* X, long long ldx, long long P, cons
                                  const float* sorted_weight, int N, int K, int gated, int act_kind, float slope, float limit,
                                  float shift, cudaStream_t stream) {
   if (P <= 0) return 0;
-  if (act_kind < LLMX_ACT_SILU || act_kind > LLMX_ACT_LAST) return LLMX_REFUSED(1);
+  if (act_kind < LLMX_ACT_SILU || act_kind > (gated == 2 ? LLMX_ACT_LAST_PLAIN : LLMX_ACT_LAST)) return LLMX_REFUSED(1);
   const GateAct act = {act_kind, slope, limit, shift};
   if (N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || max_tiles <= 0 ||
       n_experts <= 0 || (!gated && (!dest || !sorted_weight)))

@@ -566,15 +566,16 @@ def qk_norm_rope_cache(qkv, q_out, k_cache, v_cache, block_table, token_seq, tok
              v_head_dim, int(write_cache), _ptr(bias), _stream()), "qk_norm_rope_cache")
 
 
-GATE_ACTS = {"silu": 0, "relu": 1, "clamped_swish": 2, "gelu_tanh": 3, "relu_squared": 4}
+GATE_ACTS = {"silu": 0, "relu": 1, "clamped_swish": 2, "gelu_tanh": 3}
+PLAIN_ACTS = {"silu": 0, "relu": 1, "gelu_tanh": 3, "relu_squared": 4}       # of a feed-forward without a gate
 
 
 def gate_act_args(activation="silu") -> tuple:
-    """(kind, slope, limit, shift) as the kernels take them.  ``activation``: "silu", "relu", "gelu_tanh", "relu_squared"
-    (max(g, 0)^2 * u), or
+    """(kind, slope, limit, shift) as the kernels take them.  ``activation``: "silu", "relu", "gelu_tanh", without a gate
+    "relu_squared" (max(z, 0)^2), or
     ("clamped_swish", slope, limit, shift): min(g, limit) * sigmoid(slope * min(g, limit)) * (clamp(u, +-limit) + shift)."""
     if isinstance(activation, str):
-        return GATE_ACTS[activation], 1.0, 0.0, 0.0
+        return {**GATE_ACTS, **PLAIN_ACTS}[activation], 1.0, 0.0, 0.0
     name, slope, limit, shift = activation
     return GATE_ACTS[name], float(slope), float(limit), float(shift)
 
@@ -599,7 +600,7 @@ def silu_gate(gu: torch.Tensor, out: torch.Tensor, block: int = 0, activation="s
 
 
 def plain_act(parts: torch.Tensor, out: torch.Tensor, activation) -> None:
-    """The activation of a feed-forward without a gate: out = act(parts.sum(0)), the gated activation with up = 1;
+    """The activation of a feed-forward without a gate (``PLAIN_ACTS``): out = act(parts.sum(0));
     parts [S, ...] (partials added in order) or a tensor of out's shape."""
     _dev(parts, out)
     _contig("parts", parts), _contig("out", out)
@@ -1117,7 +1118,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_split: int = 
     with ``gated``, [T,N/2] = silu(gate) * up: ``gated=True`` (or 1) for
     w = [gate rows; up rows], ``gated=2`` for w in blocks of 16 gate rows each
     followed by the 16 up rows of the same features (N/2 a multiple of 16); ``gated=3``: no gate, [T,N] = act(product)
-    (``gate_act_args`` with up = 1).
+    (``PLAIN_ACTS``).
     ``pair`` runs the CTA-pair kernel (prompt-sized T > 128; it splits too); with
     ``accumulate`` it adds to a float32 ``out`` instead of overwriting it
     (one float32 addition per element, whatever order the tiles finish in).
@@ -1132,7 +1133,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_split: int = 
     N = w.shape[0]
     assert w.shape[1] == K and out.is_contiguous()
     if gated:
-        if not gemm_tc_gated_supports(activation):
+        if activation not in PLAIN_ACTS if gated == 3 else not gemm_tc_gated_supports(activation):
             raise Unsupported(f"the tensor-core product has no epilogue for the activation {activation!r}")
         _set_tc_gate_act(activation)
         if gate_bias is not None:
@@ -1635,8 +1636,8 @@ def moe_grouped_tc(xs, w, y, tiles, tile_rows: int, dest, sorted_weight, gated: 
     ``sorted_weight[place]`` times the product.  ``tiles`` made by ``moe_sort`` with ``tile_rows`` in (16, 64, 128)."""
     _dev(xs, w, y, tiles, dest, sorted_weight)
     _contig("w", w), _contig("y", y)
-    assert moe_tc_supports(xs, w) and tile_rows in (16, 64, 128) and (not gated or moe_tc_gated_supports(activation))
     gated = int(gated)
+    assert moe_tc_supports(xs, w) and tile_rows in (16, 64, 128) and (not gated or (activation in PLAIN_ACTS if gated == 2 else moe_tc_gated_supports(activation)))
     K = xs.shape[1]
     N = w.shape[1] // 2 if gated == 1 else w.shape[1]
     assert w.shape[2] == K and y.dtype == (torch.bfloat16 if gated else torch.float32)

@@ -60,13 +60,14 @@ class NoFeedForward:
 class RoutedExperts:
     def __init__(self, spec, weights: dict, rt):
         name = spec.get("activation", "silu")
-        if name not in kernels.GATE_ACTS:
-            raise Unsupported(f"routed_experts activation {name!r}: built are {sorted(kernels.GATE_ACTS)}")
+        self.gated = bool(spec.get("gated", True))
+        acts = kernels.GATE_ACTS if self.gated else kernels.PLAIN_ACTS
+        if name not in acts:
+            raise Unsupported(f"routed_experts activation {name!r}: built are {sorted(acts)}")
         act = lambda limit: name if name != "clamped_swish" else (
             name, float(spec.get("act_slope", 1.0)), float(limit), float(spec.get("act_up_shift", 0.0)))
         self.activation = act(spec.get("act_limit", 0.0))
         self.rt = rt
-        self.gated = bool(spec.get("gated", True))
         self.E, self.top, self.F = spec["n_experts"], spec["top"], spec["intermediate_size"]
         self.n_identity = int(spec.get("n_identity") or 0)
         self.E_all = self.E + self.n_identity         # what the router chooses among
@@ -127,7 +128,7 @@ class RoutedExperts:
 
         # bfloat16 with sizes the TMA takes: the grouped products run on tcgen05 (csrc/moe_tc.cu)
         self.tensor_cores = bool(rt.tensor_cores and dt == torch.bfloat16 and self.gate_up.shape[2] % 8 == 0
-                                 and self.F % 8 == 0 and kernels.moe_tc_gated_supports(self.activation))
+                                 and self.F % 8 == 0 and (not self.gated or kernels.moe_tc_gated_supports(self.activation)))
 
     def libraries(self) -> set:
         libs = {"moe", "elementwise"} | ({"moe_tc"} if self.tensor_cores else set())

@@ -100,13 +100,13 @@ class GatedMLP:
 
 @register_feed_forward("mlp")
 class PlainMLP:
-    """A feed-forward without a gate: down(act(up x)), ``activation`` as for the gated one with up = 1 ("relu_squared":
+    """A feed-forward without a gate: down(act(up x)), ``activation`` one of ``kernels.PLAIN_ACTS`` ("relu_squared":
     max(z, 0)^2)."""
 
     def __init__(self, spec, weights: dict, rt):
         self.activation = spec.get("activation", "relu")
-        if self.activation not in kernels.GATE_ACTS or self.activation == "clamped_swish":
-            raise Unsupported(f"mlp activation {self.activation!r}: built are silu, relu, gelu_tanh, relu_squared")
+        if self.activation not in kernels.PLAIN_ACTS:
+            raise Unsupported(f"mlp activation {self.activation!r}: built are {sorted(kernels.PLAIN_ACTS)}")
         self.rt, self.F = rt, spec["intermediate_size"]
         t = spec.tensors
         self.up, self.down = Linear(weights.pop(t["up"].name), rt), Linear(weights.pop(t["down"].name), rt)
