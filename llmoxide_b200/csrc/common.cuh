@@ -282,9 +282,19 @@ __device__ __forceinline__ float plain_act(const GateAct a, float x) {
   const float r = fmaxf(x, 0.f);
   return a.kind == LLMX_ACT_RELU_SQUARED ? r * r : gated_act(a, x, 1.0f);
 }
-__device__ __forceinline__ float plain_act_fast(const GateAct a, float x) {
-  const float r = fmaxf(x, 0.f);
-  return a.kind == LLMX_ACT_RELU_SQUARED ? r * r : gated_act_fast(a, x, 1.0f);
+// A whole array of an epilogue at once: the kind is looked at once, not once an element.
+template <int N>
+__device__ __forceinline__ void plain_act_fast(const GateAct a, float (&x)[N]) {
+  if (a.kind == LLMX_ACT_RELU_SQUARED) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float r = fmaxf(x[i], 0.f);
+      x[i] = r * r;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) x[i] = gated_act_fast(a, x[i], 1.0f);
+  }
 }
 
 // Butterfly reductions: every lane ends with the same value, and the order of

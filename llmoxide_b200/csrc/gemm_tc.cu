@@ -108,13 +108,13 @@ __device__ __forceinline__ void epilogue_tile(uint32_t acc_addr, bool have_acc, 
           out[(size_t)t * ldy + n] = from_f32<TY>(gated_act_fast(act, gate, up));
       }
     } else if (store && n < n_limit) {
+      if (MODE == 3) plain_act_fast(act, v);
 #pragma unroll
       for (int e = 0; e < 16; ++e) {
         const int t = t0 + c + e;
         if (t < T) {
           float r = v[e];
           if (MODE == 1) r = gated_act_fast(act, r, g[e]);
-          if (MODE == 3) r = plain_act_fast(act, r);
           out[(size_t)t * ldy + n] = from_f32<TY>(r);
         }
       }
@@ -163,8 +163,9 @@ __device__ __forceinline__ void epilogue_tile_staged(uint32_t acc_addr, const CU
         buf[(e + (upper ? 1 : 0)) * COLS + col] = from_f32<TY>(gated_act_fast(act, gate, up));
       }
     } else {
+      if (MODE == 3) plain_act_fast(act, v);
 #pragma unroll
-      for (int e = 0; e < ROWS; ++e) buf[e * COLS + col] = from_f32<TY>(MODE == 3 ? plain_act_fast(act, v[e]) : v[e]);
+      for (int e = 0; e < ROWS; ++e) buf[e * COLS + col] = from_f32<TY>(v[e]);
     }
     fence_proxy_async();
     asm volatile("bar.sync 1, 128;" ::: "memory");

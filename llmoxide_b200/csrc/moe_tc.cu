@@ -190,6 +190,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
         float v[16], g[16];
         tmem_ld16(acc_addr + (uint32_t)c, v);
         if (MODE == 1) tmem_ld16(acc_addr + (uint32_t)(BN + c), g);
+        if (MODE == 2) plain_act_fast(act, v);
         if (n < N) {
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
@@ -198,7 +199,7 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
             if (MODE == 1) {
               Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(gated_act_fast(act, v[i], g[i]));
             } else if (MODE == 2) {
-              Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(plain_act_fast(act, v[i]));
+              Y[(size_t)(row0 + r) * N + n] = from_f32<TY>(v[i]);
             } else {
               Y[(size_t)tile_dest[r] * N + n] = from_f32<TY>(tile_weight[r] * v[i]);
             }
