@@ -111,7 +111,7 @@ def window_mask(T, size, keep_first=0):
 
 
 def attend(q, k, v, scale, visible, sink, bias=None):
-    """One head: q, k [T, D], v [T, Dv]; ``bias`` [T, T] joins the scaled scores; exp(sink) joins the denominator."""
+    """One head: q, k [T, D], v [T, Dv]; ``bias`` [T, T] is added to the scaled scores, exp(sink) to the sum of weights."""
     s = (q @ k.T) * scale
     if bias is not None:
         s = s + bias
@@ -175,7 +175,7 @@ def state_space(x, B, C, dt, A_log, D_skip, state=None):
 
 
 def gate_then_norm(y, z, weight, parts, eps):
-    """y * silu(z), every one of ``parts`` equal runs of columns divided by its own root mean square, times ``weight``."""
+    """y * silu(z), an RMS norm over each of ``parts`` equal runs of columns, times ``weight``."""
     g = y * silu(z)
     T, n = g.shape
     return unit_rms(g.reshape(T, parts, n // parts), eps).reshape(T, n) * weight

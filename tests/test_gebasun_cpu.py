@@ -192,7 +192,7 @@ def test_convolution_meets_the_current_token_with_its_last_tap():
     assert plain.causal_conv(u, w, torch.tensor([0.5], dtype=F))[:, 0].tolist() == [5.5, 53.5, 530.5]
 
 
-def test_gate_comes_before_a_norm_in_parts():
+def test_norm_in_parts_takes_the_gated_rows():
     y = torch.tensor([[3.0, 4.0, 1.0, 1.0]], dtype=F)
     z = torch.full((1, 4), 50.0, dtype=F)                 # silu(50) = 50
     got = plain.gate_then_norm(y, z, torch.tensor([1.0, 1.0, 2.0, 2.0], dtype=F), 2, 1e-12)
